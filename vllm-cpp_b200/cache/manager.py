@@ -12,6 +12,10 @@ window) form a group with pages and tables of its own.  A request holds one tabl
 per group.  A group with a window gives pages back as soon as the window has
 passed them: a query at position p reads keys j with p - window < j <= p, so once
 a request holds ``n`` tokens no later query reads a key at or below n - window.
+A group whose rows stand for ``stride`` tokens each (PagedKVSpec.stride) hands out pages
+for n // stride rows; its pool is sized so that whatever fits a group of one row per
+token fits it too.  A windowed group that such rows are made from (``keep_block``)
+keeps the tokens of the block that is not complete yet.
 Layers that declare a StateSpec get one slot per live request in a tensor of
 their own; the slot is zeroed when the request is admitted.  A request always
 gets a slot id, even if no layer has state.
@@ -92,7 +96,7 @@ class CacheManager:
         if isinstance(spec, PagedKVSpec):
             g = next((i for i, pg in enumerate(self.paged) if pg.spec == spec), None)
             if g is None:
-                self.paged.append(PagedGroup(spec, [], BlockPool(self.num_pages)))
+                self.paged.append(PagedGroup(spec, [], BlockPool(self.group_pages(spec, self.num_pages, self.max_num_seqs))))
                 g = len(self.paged) - 1
             self.paged[g].layers.append(layer)
             return ("paged", g, len(self.paged[g].layers) - 1)
@@ -105,18 +109,33 @@ class CacheManager:
             return ("state", g, len(self.state[g].layers) - 1)
         raise TypeError(f"cache layer {layer}: unknown cache need {spec!r}")
 
+    @staticmethod
+    def group_pages(spec: PagedKVSpec, num_pages: int, max_num_seqs: int) -> int:
+        """Pages of the group's pool in a cache of ``num_pages`` pages of one row per token.  With a stride s, requests of
+        n_1, n_2, ... tokens that fit those pages hold at most sum(n_i) / s rows, and every request may leave one page
+        partly filled: ceil(num_pages / s) + max_num_seqs pages hold them in any mixture."""
+        return num_pages if spec.stride == 1 else cdiv(num_pages, spec.stride) + max_num_seqs
+
     # ---------------------------------------------------------------- device
     @staticmethod
     def bytes_per_page(cache_specs: List[object], page_size: int, dtype: torch.dtype) -> int:
-        """Device bytes that one page id costs over all paged cache layers."""
+        """Device bytes that one page of tokens costs over all paged cache layers (a group of one row per ``stride``
+        tokens costs a page's stride-th part; ``fixed_bytes`` has the rest)."""
         el = torch.empty((), dtype=dtype).element_size()
-        return sum(s.planes * s.num_kv_heads * page_size * s.head_dim * el
+        return sum(cdiv(s.planes * s.num_kv_heads * page_size * s.head_dim * el, s.stride)
                    for s in flatten_specs(cache_specs) if isinstance(s, PagedKVSpec))
+
+    @staticmethod
+    def fixed_bytes(cache_specs: List[object], page_size: int, max_num_seqs: int, dtype: torch.dtype) -> int:
+        """Device bytes of the pages that strided groups have beyond their share of the page count (group_pages)."""
+        el = torch.empty((), dtype=dtype).element_size()
+        return sum((max_num_seqs + 1) * s.planes * s.num_kv_heads * page_size * s.head_dim * el
+                   for s in flatten_specs(cache_specs) if isinstance(s, PagedKVSpec) and s.stride > 1)
 
     def _allocate_device(self) -> None:
         for g in self.paged:
             s = g.spec
-            g.pages = torch.zeros((len(g.layers), self.num_pages, s.planes, s.num_kv_heads, self.page_size * s.head_dim),
+            g.pages = torch.zeros((len(g.layers), g.pool.num_blocks, s.planes, s.num_kv_heads, self.page_size * s.head_dim),
                                   dtype=self.dtype, device=self.device)
         for g in self.state:
             g.slots = torch.zeros((len(g.layers), self.max_num_seqs) + tuple(g.spec.shape),
@@ -159,8 +178,12 @@ class CacheManager:
     def pages_needed(self, req_id, n_new: int) -> List[int]:
         """Pages each group must still hand out before ``n_new`` more tokens fit."""
         rc = self.requests[req_id]
-        want = cdiv(rc.num_tokens + n_new, self.page_size)
-        return [max(0, want - len(t)) for t in rc.tables]
+        n = rc.num_tokens + n_new
+        return [max(0, cdiv(n // g.spec.stride, self.page_size) - len(t)) for g, t in zip(self.paged, rc.tables)]
+
+    def _room(self, g: PagedGroup, pages: int) -> int:
+        """Most tokens a request may hold with ``pages`` pages of the group."""
+        return (pages * self.page_size + 1) * g.spec.stride - 1
 
     def can_append(self, req_id, n_new: int) -> bool:
         return all(g.pool.can_allocate(n) for g, n in zip(self.paged, self.pages_needed(req_id, n_new)))
@@ -170,10 +193,9 @@ class CacheManager:
         if not self.paged:
             return 1 << 30
         if req_id is None:
-            return self.num_free_pages() * self.page_size
+            return min(self._room(g, g.pool.num_free) for g in self.paged)
         rc = self.requests[req_id]
-        return min((len(t) + g.pool.num_free) * self.page_size for g, t in zip(self.paged, rc.tables)) \
-            - rc.num_tokens
+        return min(self._room(g, len(t) + g.pool.num_free) for g, t in zip(self.paged, rc.tables)) - rc.num_tokens
 
     def reserve(self, req_id, n_new: int) -> None:
         """Give the request pages for its next ``n_new`` tokens in every group, or none at all."""
@@ -182,7 +204,7 @@ class CacheManager:
         for g, n in zip(self.paged, need):
             if not g.pool.can_allocate(n):
                 raise OutOfPages(f"request {req_id!r} needs {n} more pages for {n_new} tokens; "
-                                 f"{g.pool.num_free} of {self.num_pages} are free")
+                                 f"{g.pool.num_free} of {g.pool.num_blocks} are free")
         for gi, (g, table, n) in enumerate(zip(self.paged, rc.tables, need)):
             for _ in range(n):
                 page = g.pool.acquire()
@@ -194,14 +216,17 @@ class CacheManager:
         """The request now holds ``n_new`` more tokens; give back what windows have passed."""
         rc = self.requests[req_id]
         rc.num_tokens += n_new
-        if rc.tables and rc.num_tokens > min(len(t) for t in rc.tables) * self.page_size:
+        if any(rc.num_tokens > self._room(g, len(t)) for g, t in zip(self.paged, rc.tables)):
             raise PageError(f"request {req_id!r} holds {rc.num_tokens} tokens but pages for fewer")
         for gi, g in enumerate(self.paged):
             w = g.spec.window
             if w <= 0:
                 continue
-            # keys at positions <= num_tokens - w are never read again
-            dead_blocks = max(0, (rc.num_tokens - w + 1) // self.page_size)
+            # keys at positions <= num_tokens - w are never read again, unless a block's summary is still to be made of them
+            dead = rc.num_tokens - w + 1
+            if g.spec.keep_block > 1:
+                dead = min(dead, rc.num_tokens // g.spec.keep_block * g.spec.keep_block)
+            dead_blocks = max(0, dead // self.page_size)
             table = rc.tables[gi]
             for b in range(rc.released[gi], min(dead_blocks, len(table))):
                 g.pool.release(table[b])
@@ -242,5 +267,5 @@ class CacheManager:
         return self.requests[req_id].slot
 
     def num_free_pages(self) -> int:
-        """Free pages of the scarcest group."""
-        return min((g.pool.num_free for g in self.paged), default=self.num_pages)
+        """Free pages of the scarcest group of one row per token (a group with a stride counts rows of another kind)."""
+        return min((g.pool.num_free for g in self.paged if g.spec.stride == 1), default=self.num_pages)

@@ -311,9 +311,10 @@ VCB_EXPORT int vcb_cast_rows(const float* x, const void* delta, float mult, void
 }
 
 // ------------------------------------------------------- gated activation
-// out[t, i] = silu(gu[t, i]) * gu[t, inter + i],  silu(z) = z / (1 + exp(-z))
-// (src/kernels/activation.cu:8-10,34-39), evaluated in float with expf.
-template <typename T>
+// out[t, i] = act(gu[t, i]) * gu[t, inter + i],  act GATE_SILU: z / (1 + exp(-z))
+// (src/kernels/activation.cu:8-10,34-39), evaluated in float with expf; GATE_RELU: max(z, 0).
+enum { GATE_SILU = 0, GATE_RELU = 1 };
+template <typename T, int ACT>
 __global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, int inter) {
     pdl_start();
     const int t = blockIdx.y;
@@ -322,7 +323,7 @@ __global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, i
     T* o = out + (size_t)t * inter;
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < inter; i += gridDim.x * blockDim.x) {
         const float z = to_f32<T>(g[i]);
-        const float s = z / (1.0f + expf(-z));
+        const float s = ACT == GATE_RELU ? fmaxf(z, 0.0f) : z / (1.0f + expf(-z));
         o[i] = from_f32<T>(s * to_f32<T>(u[i]));
     }
 }
@@ -331,7 +332,7 @@ __global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, i
 // and round so that eight loads are in flight before the first is used.  The result is rounded to
 // bfloat16, so the exponential and the division are the fast ones (a few units in the last place of a
 // float); the 32-bit path above uses expf and a true division.
-template <typename IDX>
+template <typename IDX, int ACT>
 __global__ void silu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out,
                                        int inter, IDX n_vec) {
     pdl_start();
@@ -362,7 +363,8 @@ __global__ void silu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __n
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const float2 g = __bfloat1622float2(g2[e]), u = __bfloat1622float2(u2[e]);
-                const float a = __fdividef(g.x, 1.0f + __expf(-g.x)), b = __fdividef(g.y, 1.0f + __expf(-g.y));
+                const float a = ACT == GATE_RELU ? fmaxf(g.x, 0.0f) : __fdividef(g.x, 1.0f + __expf(-g.x));
+                const float b = ACT == GATE_RELU ? fmaxf(g.y, 0.0f) : __fdividef(g.y, 1.0f + __expf(-g.y));
                 o2[e] = __floats2bfloat162_rn(a * u.x, b * u.y);
             }
             *reinterpret_cast<uint4*>(out + dst[k]) = o4;
@@ -370,18 +372,18 @@ __global__ void silu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __n
     }
 }
 
-VCB_EXPORT int vcb_silu_mul(const void* gu, void* out, int n_tokens, int inter, int dtype, void* stream) {
+template <int ACT>
+static int launch_gate_mul(const void* gu, void* out, int n_tokens, int inter, int dtype, cudaStream_t s) {
     if (n_tokens <= 0) return 0;
-    cudaStream_t s = (cudaStream_t)stream;
     if (dtype == VCB_BF16 && inter % 8 == 0 && ((((uintptr_t)gu | (uintptr_t)out) & 15) == 0)) {
         const size_t n_vec = (size_t)n_tokens * (inter >> 3);
         size_t blocks = (n_vec + 1023) / 1024;
         if (blocks > vcb_sm_count() * 16) blocks = vcb_sm_count() * 16;
         if (n_vec < (1u << 30))
-            vcb_launch(silu_mul_bf16x8_kernel<unsigned>, (int)blocks, 256, 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out,
+            vcb_launch(silu_mul_bf16x8_kernel<unsigned, ACT>, (int)blocks, 256, 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out,
                        inter, (unsigned)n_vec);
         else
-            vcb_launch(silu_mul_bf16x8_kernel<size_t>, (int)blocks, 256, 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out,
+            vcb_launch(silu_mul_bf16x8_kernel<size_t, ACT>, (int)blocks, 256, 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out,
                        inter, n_vec);
         return vcb_last_error();
     }
@@ -390,9 +392,9 @@ VCB_EXPORT int vcb_silu_mul(const void* gu, void* out, int n_tokens, int inter, 
     if (bx > 64) bx = 64;
     dim3 grid(bx, n_tokens);
     if (dtype == VCB_F32)
-        vcb_launch(silu_mul_kernel<float>, grid, threads, 0, s, (const float*)gu, (float*)out, inter);
+        vcb_launch(silu_mul_kernel<float, ACT>, grid, threads, 0, s, (const float*)gu, (float*)out, inter);
     else if (dtype == VCB_BF16)
-        vcb_launch(silu_mul_kernel<__nv_bfloat16>, grid, threads, 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, inter);
+        vcb_launch(silu_mul_kernel<__nv_bfloat16, ACT>, grid, threads, 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, inter);
     else
         return VCB_ERR_BAD_ARG;
     return vcb_last_error();
@@ -499,6 +501,14 @@ VCB_EXPORT int vcb_clamped_swish_mul(const void* gu, const float* bias, void* ou
     else
         return VCB_ERR_BAD_ARG;
     return vcb_last_error();
+}
+
+VCB_EXPORT int vcb_silu_mul(const void* gu, void* out, int n_tokens, int inter, int dtype, void* stream) {
+    return launch_gate_mul<GATE_SILU>(gu, out, n_tokens, inter, dtype, (cudaStream_t)stream);
+}
+
+VCB_EXPORT int vcb_relu_mul(const void* gu, void* out, int n_tokens, int inter, int dtype, void* stream) {
+    return launch_gate_mul<GATE_RELU>(gu, out, n_tokens, inter, dtype, (cudaStream_t)stream);
 }
 
 // ------------------------------------- q/k/v bias + rotary + cache write

@@ -14,10 +14,9 @@
 //
 // States, decays and their logarithms, softplus and exponentials, gates, unit norms and every sum are float whatever the
 // type T of the projections is.  The reference has no recurrent mixer (src/layers/attention.cpp is its only mixer).
-#include "common.cuh"
+#include "short_conv.cuh"
 
-#define CONV_MAX_TAPS 8
-#define CONV_SEG 32            // tokens a thread walks; at least CONV_MAX_TAPS - 1, so that only a request's first segment reads the state
+#define CONV_MAX_TAPS 64       // up to 8 in registers (short_conv.cuh), more from memory
 
 __device__ __forceinline__ float gr_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float gr_silu(float z) { return z / (1.0f + expf(-z)); }
@@ -34,84 +33,125 @@ struct ConvArgs {
     const float* bias;          // [C] or null: added to the sum
     float* state;               // slot s, row j (0 .. J - 2), channel c at state[s * slot_stride + j * C + c]
     long long slot_stride;
-    float* out;                 // [n, C] float, row stride ldo
+    void* out;                  // [n, C] of TO, row stride ldo
     long long ldo;
     const int* q_start;
     const int* state_slots;
     int C, J, act;
 };
 
-// Grid (segments of the longest portion, requests, tiles of 128 channels); a thread per channel.
-template <typename T>
+// Grid (segments of the longest portion, requests, tiles of 128 * VW channels); a thread per VW channels and segment.
+template <typename T, typename TO, int MAXJ, int SEG, int VW>
 __global__ void __launch_bounds__(128) causal_conv_kernel(ConvArgs a) {
-    const int c = blockIdx.z * 128 + threadIdx.x;
-    float w[CONV_MAX_TAPS];
-    const int J = a.J;
-    const bool live = c < a.C;
+    const int c = (blockIdx.z * 128 + threadIdx.x) * VW;
+    const bool there = c < a.C;
+    float taps[MAXJ][VW], pb[VW], cb[VW];
+    if (there) {
+        conv_taps<MAXJ, VW>(a.w + (size_t)c * a.J, a.J, VW, taps);
 #pragma unroll
-    for (int j = 0; j < CONV_MAX_TAPS; ++j) w[j] = (live && j < J) ? a.w[(size_t)c * J + j] : 0.0f;
-    const float pb = (live && a.pre_bias) ? a.pre_bias[c] : 0.0f, cb = (live && a.bias) ? a.bias[c] : 0.0f;
+        for (int e = 0; e < VW; ++e) {
+            pb[e] = a.pre_bias ? a.pre_bias[c + e] : 0.0f;
+            cb[e] = a.bias ? a.bias[c + e] : 0.0f;
+        }
+    }
     pdl_start();
     const int r = blockIdx.y;
     const int row0 = a.q_start[r], len = a.q_start[r + 1] - row0;
-    const int seg0 = blockIdx.x * CONV_SEG;
-    if (seg0 >= len || !live) return;
+    const int seg0 = blockIdx.x * SEG;
+    if (seg0 >= len || !there) return;
     const T* x = (const T*)a.x + (size_t)row0 * a.ldx + c;
     float* st = a.state + (size_t)a.state_slots[r] * a.slot_stride + c;
-    // win[j]: the input J - 1 - j places before the current token, oldest first
-    float win[CONV_MAX_TAPS - 1], old[CONV_MAX_TAPS - 1];
+    float h[MAXJ - 1 + SEG][VW];
+    conv_window<T, MAXJ, SEG, VW>(x, a.ldx, st, a.C, pb, a.J, seg0, len, VW, h);
+    TO* out = (TO*)a.out + (size_t)(row0 + seg0) * a.ldo + c;
 #pragma unroll
-    for (int j = 0; j < CONV_MAX_TAPS - 1; ++j) {
-        win[j] = old[j] = 0.0f;
-        if (j < J - 1) {
-            const int li = seg0 - (J - 1) + j;
-            win[j] = li >= 0 ? to_f32<T>(x[(size_t)li * a.ldx]) + pb : st[(size_t)(J - 1 + li) * a.C];
-            old[j] = win[j];
+    for (int t = 0; t < SEG; ++t) {
+        if (seg0 + t >= len) break;
+        float y[VW];
+#pragma unroll
+        for (int e = 0; e < VW; ++e) {
+            y[e] = cb[e];
+#pragma unroll
+            for (int m = 0; m < MAXJ; ++m) y[e] = fmaf(taps[m][e], h[t + m][e], y[e]);
+            if (a.act) y[e] = gr_silu(y[e]);
         }
+        TO* dst = out + (size_t)t * a.ldo;
+        if constexpr (VW == 2 && sizeof(TO) == 2) *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(y[0], y[1]);
+        else if constexpr (VW == 2) *reinterpret_cast<float2*>(dst) = make_float2(y[0], y[1]);
+        else dst[0] = from_f32<TO>(y[0]);
     }
-    const int end = min(seg0 + CONV_SEG, len);
-    float* out = a.out + (size_t)row0 * a.ldo + c;
-    for (int t = seg0; t < end; ++t) {
-        const float cur = to_f32<T>(x[(size_t)t * a.ldx]) + pb;
-        float acc = cb;
-#pragma unroll
-        for (int j = 0; j < CONV_MAX_TAPS - 1; ++j)
-            if (j < J - 1) acc = fmaf(w[j], win[j], acc);
-        acc = fmaf(w[J - 1], cur, acc);
-        out[(size_t)t * a.ldo] = a.act ? gr_silu(acc) : acc;
-#pragma unroll
-        for (int j = 0; j < CONV_MAX_TAPS - 2; ++j) win[j] = win[j + 1];
-        if (J >= 2) {
-#pragma unroll
-            for (int j = 0; j < CONV_MAX_TAPS - 1; ++j)
-                if (j == J - 2) win[j] = cur;
+    if (seg0 == 0) conv_keep<T, VW>(x, a.ldx, st, a.C, pb, a.J, len, VW);
+}
+
+// More taps than the registers hold, read from memory one by one.
+template <typename T, typename TO>
+__global__ void __launch_bounds__(128) causal_conv_long_kernel(ConvArgs a) {
+    constexpr int SEG = CONV_MAX_TAPS;
+    const int c = blockIdx.z * 128 + threadIdx.x;
+    pdl_start();
+    const int r = blockIdx.y;
+    const int row0 = a.q_start[r], len = a.q_start[r + 1] - row0;
+    const int seg0 = blockIdx.x * SEG;
+    if (seg0 >= len || c >= a.C) return;
+    const float pb[1] = {a.pre_bias ? a.pre_bias[c] : 0.0f}, cb = a.bias ? a.bias[c] : 0.0f;
+    const T* x = (const T*)a.x + (size_t)row0 * a.ldx + c;
+    float* st = a.state + (size_t)a.state_slots[r] * a.slot_stride + c;
+    TO* out = (TO*)a.out + (size_t)row0 * a.ldo + c;
+    for (int li = seg0; li < min(seg0 + SEG, len); ++li) {
+        float y = cb;
+        for (int j = 0; j < a.J; ++j) {
+            const int s = li - (a.J - 1) + j;
+            y = fmaf(a.w[(size_t)c * a.J + j], s >= 0 ? to_f32<T>(x[(size_t)s * a.ldx]) + pb[0] : st[(size_t)(a.J - 1 + s) * a.C], y);
         }
+        out[(size_t)li * a.ldo] = from_f32<TO>(a.act ? gr_silu(y) : y);
     }
-    if (seg0 == 0) {
-        // this thread alone reads and writes the channel's state: what it read is in old[]
-#pragma unroll
-        for (int j = 0; j < CONV_MAX_TAPS - 1; ++j) {
-            if (j >= J - 1) break;
-            const int li = len - (J - 1) + j;
-            st[(size_t)j * a.C] = li >= 0 ? to_f32<T>(x[(size_t)li * a.ldx]) + pb : old[J - 1 + li];
-        }
+    if (seg0 == 0) conv_keep<T, 1>(x, a.ldx, st, a.C, pb, a.J, len, 1);
+}
+
+template <typename T, typename TO, int MAXJ, int SEG>
+static void launch_conv(const ConvArgs& a, int n_reqs, int max_q_len, bool pairs, cudaStream_t s) {
+    dim3 grid((max_q_len + SEG - 1) / SEG, n_reqs, (a.C + (pairs ? 255 : 127)) / (pairs ? 256 : 128));
+    if (pairs) vcb_launch(causal_conv_kernel<T, TO, MAXJ, SEG, 2>, grid, 128, 0, s, a);
+    else vcb_launch(causal_conv_kernel<T, TO, MAXJ, SEG, 1>, grid, 128, 0, s, a);
+}
+
+template <typename T, typename TO>
+static int launch_conv_any(const ConvArgs& a, int n_reqs, int max_q_len, cudaStream_t s) {
+    const bool pairs = !(a.C & 1) && !(a.ldx & 1) && !(a.ldo & 1) && !((uintptr_t)a.x & (2 * sizeof(T) - 1)) && !((uintptr_t)a.out & (2 * sizeof(TO) - 1));
+    if (a.J > 8) {
+        dim3 grid((max_q_len + CONV_MAX_TAPS - 1) / CONV_MAX_TAPS, n_reqs, (a.C + 127) / 128);
+        vcb_launch(causal_conv_long_kernel<T, TO>, grid, 128, 0, s, a);
+    } else if (max_q_len == 1) {
+        if (a.J <= 4) launch_conv<T, TO, 4, 1>(a, n_reqs, 1, pairs, s);
+        else launch_conv<T, TO, 8, 1>(a, n_reqs, 1, pairs, s);
+    } else {
+        if (a.J <= 4) launch_conv<T, TO, 4, 16>(a, n_reqs, max_q_len, pairs, s);
+        else launch_conv<T, TO, 8, 16>(a, n_reqs, max_q_len, pairs, s);
     }
+    return vcb_last_error();
+}
+
+// out_f32: the result in float whatever the type of x is, else in x's type.
+VCB_EXPORT int vcb_causal_conv_as(const void* x, long long ldx, const float* pre_bias, const float* w, const float* bias,
+                                  float* state, long long slot_stride, void* out, long long ldo, int out_f32, const int* q_start,
+                                  const int* state_slots, int n_reqs, int max_q_len, int C, int J, int act, int dtype, void* stream) {
+    if (n_reqs <= 0 || max_q_len <= 0) return 0;
+    if (!x || !w || (!state && J > 1) || !out || C <= 0 || J <= 0 || J > CONV_MAX_TAPS || n_reqs > 65535) return VCB_ERR_BAD_ARG;
+    ConvArgs a{x, ldx, pre_bias, w, bias, state, slot_stride, out, ldo, q_start, state_slots, C, J, act};
+    if ((C + 127) / 128 > 65535) return VCB_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == VCB_F32) return launch_conv_any<float, float>(a, n_reqs, max_q_len, s);
+    if (dtype != VCB_BF16) return VCB_ERR_BAD_ARG;
+    return out_f32 ? launch_conv_any<__nv_bfloat16, float>(a, n_reqs, max_q_len, s)
+                   : launch_conv_any<__nv_bfloat16, __nv_bfloat16>(a, n_reqs, max_q_len, s);
 }
 
 VCB_EXPORT int vcb_causal_conv(const void* x, long long ldx, const float* pre_bias, const float* w, const float* bias,
                                float* state, long long slot_stride, float* out, long long ldo, const int* q_start,
                                const int* state_slots, int n_reqs, int max_q_len, int C, int J, int act, int dtype,
                                void* stream) {
-    if (n_reqs <= 0 || max_q_len <= 0) return 0;
-    if (!x || !w || (!state && J > 1) || !out || C <= 0 || J <= 0 || J > CONV_MAX_TAPS || n_reqs > 65535) return VCB_ERR_BAD_ARG;
-    ConvArgs a{x, ldx, pre_bias, w, bias, state, slot_stride, out, ldo, q_start, state_slots, C, J, act};
-    dim3 grid((max_q_len + CONV_SEG - 1) / CONV_SEG, n_reqs, (C + 127) / 128);
-    if (grid.z > 65535) return VCB_ERR_UNSUPPORTED;
-    cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == VCB_F32) vcb_launch(causal_conv_kernel<float>, grid, 128, 0, s, a);
-    else if (dtype == VCB_BF16) vcb_launch(causal_conv_kernel<__nv_bfloat16>, grid, 128, 0, s, a);
-    else return VCB_ERR_BAD_ARG;
-    return vcb_last_error();
+    return vcb_causal_conv_as(x, ldx, pre_bias, w, bias, state, slot_stride, out, ldo, 1, q_start, state_slots, n_reqs, max_q_len, C, J, act,
+                              dtype, stream);
 }
 
 // ------------------------------------------------------------------------------- gates of the recurrent unit

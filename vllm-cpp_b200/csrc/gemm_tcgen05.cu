@@ -82,9 +82,11 @@ struct GemmArgs {
     int ldr, sumsq_ld;
     // Gated feed-forward (swapped products on a gated tile image only): > 0 = the number of gate features.
     // Tile t holds gate rows 64 t .. and, in its upper half, the matching up rows;
-    // out[token, 64 t + r] = silu(gate) * up.
-    int gated;
+    // out[token, 64 t + r] = act(gate) * up, act 0: silu, 1: relu.
+    int gated, gated_act;
 };
+
+__device__ __forceinline__ float gate_activation(int act, float z) { return act == 1 ? fmaxf(z, 0.0f) : z / (1.0f + expf(-z)); }
 
 // The segments of one CTA's run of (tile, slab) units.
 struct Segments {
@@ -377,7 +379,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
                             const float f = a.scale_sumsq ? rstd_s[j] : 1.0f;
                             const float z = v[g8 + e] * f, u = xch[r * 8 + e] * f;
                             reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)j * a.ldc + feature] =
-                                __float2bfloat16_rn(z / (1.0f + expf(-z)) * u);
+                                __float2bfloat16_rn(gate_activation(a.gated_act, z) * u);
                         }
                     }
                     asm volatile("bar.sync 1, 128;" ::: "memory");   // the halves are read before the next group overwrites them
@@ -479,7 +481,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
                                 const float z = (is_gate ? __uint_as_float(lo[e]) : from_gate[e * 64 + half_row]) * f;
                                 const float u = (is_gate ? from_up[e * 64 + half_row] : __uint_as_float(hi[e])) * f;
                                 reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)j * a.ldc + feature] =
-                                    __float2bfloat16_rn(z / (1.0f + expf(-z)) * u);
+                                    __float2bfloat16_rn(gate_activation(a.gated_act, z) * u);
                             }
                         }
                         asm volatile("bar.sync 1, 128;" ::: "memory");   // read before the next round overwrites
@@ -731,13 +733,14 @@ VCB_EXPORT int vcb_tile_weights(const void* w, int rows, int k, int ld, int gate
 //       residual += result; out (bfloat16) = residual * gain; sumsq_out = partial sums over the features
 //       of residual^2 for every token.
 //   gated > 0: p_tiled is a gated image (vcb_tile_weights) of a [2 gated, k] matrix, rows_p = 2 gated;
-//       out (bfloat16, [rows_q][>= gated]) = silu(gate) * up.
-VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused(const void* p, int rows_p, int ldp, const void* p_tiled, const void* q,
+//       out (bfloat16, [rows_q][>= gated]) = act(gate) * up with gated_act 0: silu, 1: relu.
+VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused_act(const void* p, int rows_p, int ldp, const void* p_tiled, const void* q,
                                            int rows_q, int ldq, int k, void* out, int ldc, int out_f32, int swapped,
                                            int bn, int max_ctas, float* partial, int* tickets, int n_tickets,
                                            int* status, const float* scale_sumsq, int scale_parts, int scale_ld,
                                            int scale_width, float scale_eps, float* residual, int ldr,
-                                           const float* gain, float* sumsq_out, int sumsq_ld, int gated, void* stream) {
+                                           const float* gain, float* sumsq_out, int sumsq_ld, int gated, int gated_act,
+                                           void* stream) {
     if (rows_p <= 0 || rows_q <= 0) return 0;
     if (k <= 0 || max_ctas < 1 || !status || !partial || !tickets) return VCB_ERR_BAD_ARG;
     // TMA needs 16-byte aligned bases and row strides
@@ -745,7 +748,7 @@ VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused(const void* p, int rows_p, int ldp, c
     if (!p_tiled && ((ldp % 8) || ((uintptr_t)p & 15))) return VCB_ERR_UNSUPPORTED;
     if (bn != 16 && bn != 32 && bn != 64 && bn != 128 && bn != 256) return VCB_ERR_BAD_ARG;
     if (gated) {
-        if (gated < 0 || rows_p != 2 * gated || !p_tiled || !swapped || rows_q > bn || bn > 128 || out_f32 || residual ||
+        if (gated < 0 || gated_act < 0 || gated_act > 1 || rows_p != 2 * gated || !p_tiled || !swapped || rows_q > bn || bn > 128 || out_f32 || residual ||
             ldc < gated)
             return VCB_ERR_BAD_ARG;
         rows_p = 128 * ((gated + 63) / 64);       // rows of the image
@@ -771,7 +774,7 @@ VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused(const void* p, int rows_p, int ldp, c
     GemmArgs a{out, partial, tickets, status, (const uint8_t*)p_tiled, ldc, out_f32, swapped, rows_p, rows_q,
                k_slabs, tiles_p, per, (int)total,
                scale_sumsq, scale_parts, scale_ld, scale_sumsq ? 1.0f / (float)scale_width : 0.0f, scale_eps,
-               residual, gain, sumsq_out, ldr, sumsq_ld, gated};
+               residual, gain, sumsq_out, ldr, sumsq_ld, gated, gated_act};
     cudaStream_t s = (cudaStream_t)stream;
     switch (bn) {
         case 16: return launch<16, 6>(mp, mq, a, ctas, s);
@@ -780,6 +783,18 @@ VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused(const void* p, int rows_p, int ldp, c
         case 128: return launch<128, 6>(mp, mq, a, ctas, s);
         default: return launch<256, 4>(mp, mq, a, ctas, s);
     }
+}
+
+// The same with silu in the gated form.
+VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused(const void* p, int rows_p, int ldp, const void* p_tiled, const void* q,
+                                           int rows_q, int ldq, int k, void* out, int ldc, int out_f32, int swapped,
+                                           int bn, int max_ctas, float* partial, int* tickets, int n_tickets,
+                                           int* status, const float* scale_sumsq, int scale_parts, int scale_ld,
+                                           int scale_width, float scale_eps, float* residual, int ldr,
+                                           const float* gain, float* sumsq_out, int sumsq_ld, int gated, void* stream) {
+    return vcb_gemm_bf16_tcgen05_fused_act(p, rows_p, ldp, p_tiled, q, rows_q, ldq, k, out, ldc, out_f32, swapped, bn, max_ctas,
+                                           partial, tickets, n_tickets, status, scale_sumsq, scale_parts, scale_ld, scale_width,
+                                           scale_eps, residual, ldr, gain, sumsq_out, sumsq_ld, gated, 0, stream);
 }
 
 VCB_EXPORT int vcb_gemm_bf16_tcgen05(const void* p, int rows_p, int ldp, const void* p_tiled, const void* q, int rows_q,

@@ -1,0 +1,431 @@
+// A generalised delta rule per head on a matrix S of key channels by value channels: the token decays S per key channel,
+// removes, at a rate per key channel, what S held under the token's unit key, and adds the outer product of the plain key and
+// the value; both terms read the old S:
+//
+//   u = k / sqrt(sum k^2 + eps),   w = exp(-rate * sigmoid(z + z_bias)),   a = sigmoid(a_pre + a_bias)
+//   S <- diag(w) S - (a * u) (u^T S) + k v^T,     o = S^T r
+//
+// r, k, v, z and a_pre are rows of the activations' type; everything from there to o is float.  The state lives in the request's
+// slot ([slots][H][dk][dv]), is read at the start of a request's portion and left there at its end.  With |k| = kn, k = kn u,
+// and both sums over key channels that a token needs come from the old S:
+//   p = u . S[:, c],  R = r . (w * S[:, c]);   S[:, c] = w * S[:, c] + u * (kn v_c - a p);   o_c = R - (r . (a u)) p + (r . k) v_c
+// so a token costs one round of shuffles for two sums.
+//
+//   general_delta_scan_kernel      steps of single tokens and short portions: inputs made and walked in one kernel
+//   general_delta_prepare_kernel   steps with portions: per token and head a row of floats [r | u | w | a | v | kn, r.(a u), r.k, 0]
+//   general_delta_walk_kernel      the walk over the tokens, whose rows arrive by asynchronous copies a chunk ahead
+#include "common.cuh"
+
+struct GDeltaArgs {
+    const void* r;              // [n, H * dk] rows of T
+    const void* k;              // [n, H * dk]
+    const void* v;              // [n, H * dv]
+    const void* a_pre;          // [n, H * dk]
+    const void* z;              // [n, H * dk]
+    long long ldr, ldk, ldv, lda, ldz;
+    const float* a_bias;        // [H * dk] or null
+    const float* z_bias;        // [H * dk] or null
+    float* state;               // [slots][H][dk][dv]
+    float* out;                 // [n, H * dv] float, row stride ldo
+    long long ldo;
+    const int* q_start;
+    const int* state_slots;
+    int H, dk, dv;
+    float rate, unit_eps;
+    int chunk;                  // tokens staged in shared memory at a time
+};
+
+__device__ __forceinline__ float gd_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// A warp makes one token's inputs of one head: calls put(i, r, u, w, a) for its channels i (lane, lane + 32, ...) and returns
+// the three sums to every lane.
+template <typename T, typename Put>
+__device__ __forceinline__ void gd_inputs(const GDeltaArgs& A, size_t row, int h, int lane, Put put, float& kn, float& ra, float& rk) {
+    const T* rp = (const T*)A.r + row * A.ldr + h * A.dk;
+    const T* kp = (const T*)A.k + row * A.ldk + h * A.dk;
+    const T* ap = (const T*)A.a_pre + row * A.lda + h * A.dk;
+    const T* zp = (const T*)A.z + row * A.ldz + h * A.dk;
+    const float* ab = A.a_bias ? A.a_bias + h * A.dk : nullptr;
+    const float* zb = A.z_bias ? A.z_bias + h * A.dk : nullptr;
+    float ss = 0.0f;
+    for (int i = lane; i < A.dk; i += 32) { const float x = to_f32<T>(kp[i]); ss = fmaf(x, x, ss); }
+    kn = sqrtf(warp_sum(ss) + A.unit_eps);
+    const float inv = 1.0f / kn;
+    float sa = 0.0f, sk = 0.0f;
+    for (int i = lane; i < A.dk; i += 32) {
+        const float x = to_f32<T>(kp[i]), r = to_f32<T>(rp[i]), u = x * inv;
+        const float a = gd_sigmoid(to_f32<T>(ap[i]) + (ab ? ab[i] : 0.0f));
+        const float w = expf(-A.rate * gd_sigmoid(to_f32<T>(zp[i]) + (zb ? zb[i] : 0.0f)));
+        sa = fmaf(r, a * u, sa);
+        sk = fmaf(r, x, sk);
+        put(i, r, u, w, a);
+    }
+    ra = warp_sum(sa);
+    rk = warp_sum(sk);
+}
+
+// Grid (request, head, tile of DVT value channels).  A thread keeps DKP rows of one column of S in registers; the P threads
+// that share a column are neighbouring lanes.  Key channels beyond dk are padded with r = u = a = 0, w = 1.
+template <typename T, int DKP>
+__global__ void general_delta_scan_kernel(GDeltaArgs A, int P, int DVT) {
+    extern __shared__ __align__(16) float sm[];
+    const int r = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * DVT;
+    const int tid = threadIdx.x, nthreads = blockDim.x, lane = tid & 31, warp = tid >> 5, nwarps = nthreads >> 5;
+    const int part = tid % P, cl = tid / P, col = col0 + cl;
+    const bool col_ok = cl < DVT && col < A.dv;
+    const int TC = A.chunk, pstride = DKP + 4, tstride = P * pstride;
+    float* rs = sm;
+    float* us = rs + TC * tstride;
+    float* ws = us + TC * tstride;
+    float* as = ws + TC * tstride;
+    float* vs = as + TC * tstride;                // [TC][DVT]
+    float* os = vs + TC * DVT;                    // [TC][DVT]
+    float* sc = os + TC * DVT;                    // [TC][4]: kn, r.(a u), r.k
+    pdl_start();
+    const int row0 = A.q_start[r], row1 = A.q_start[r + 1];
+    float* st = A.state + (((size_t)A.state_slots[r] * A.H + h) * A.dk) * A.dv;
+    float S[DKP];
+#pragma unroll
+    for (int i = 0; i < DKP; ++i) {
+        const int kr = part * DKP + i;
+        S[i] = (col_ok && kr < A.dk) ? st[(size_t)kr * A.dv + col] : 0.0f;
+    }
+    for (int idx = tid; idx < TC * P * DKP; idx += nthreads) {
+        const int tt = idx / (P * DKP), i = idx - tt * (P * DKP);
+        if (i >= A.dk) {
+            const int at = tt * tstride + (i / DKP) * pstride + i % DKP;
+            rs[at] = us[at] = as[at] = 0.0f;
+            ws[at] = 1.0f;
+        }
+    }
+    for (int c0 = row0; c0 < row1; c0 += TC) {
+        const int tc = min(TC, row1 - c0);
+        __syncthreads();                          // the chunk before has been read
+        for (int tt = warp; tt < tc; tt += nwarps) {
+            float kn, ra, rk;
+            gd_inputs<T>(A, (size_t)(c0 + tt), h, lane, [&](int i, float rv, float u, float w, float a) {
+                const int at = tt * tstride + (i / DKP) * pstride + i % DKP;
+                rs[at] = rv;
+                us[at] = u;
+                ws[at] = w;
+                as[at] = a;
+            }, kn, ra, rk);
+            if (lane == 0) { sc[tt * 4] = kn; sc[tt * 4 + 1] = ra; sc[tt * 4 + 2] = rk; }
+        }
+        for (int idx = tid; idx < tc * DVT; idx += nthreads) {
+            const int tt = idx / DVT, j = idx - tt * DVT, c = col0 + j;
+            vs[idx] = c < A.dv ? to_f32<T>(((const T*)A.v)[(size_t)(c0 + tt) * A.ldv + h * A.dv + c]) : 0.0f;
+        }
+        __syncthreads();
+        if (cl < DVT) {
+            for (int tt = 0; tt < tc; ++tt) {
+                const int at = tt * tstride + part * pstride;
+                const float4* r4 = reinterpret_cast<const float4*>(rs + at);
+                const float4* u4 = reinterpret_cast<const float4*>(us + at);
+                const float4* w4 = reinterpret_cast<const float4*>(ws + at);
+                const float4* a4 = reinterpret_cast<const float4*>(as + at);
+                float p0 = 0.0f, p1 = 0.0f, q0 = 0.0f, q1 = 0.0f;
+#pragma unroll
+                for (int i = 0; i < DKP / 4; ++i) {
+                    const float4 u = u4[i], w = w4[i], rv = r4[i];
+                    p0 = fmaf(S[4 * i], u.x, p0);
+                    p1 = fmaf(S[4 * i + 1], u.y, p1);
+                    p0 = fmaf(S[4 * i + 2], u.z, p0);
+                    p1 = fmaf(S[4 * i + 3], u.w, p1);
+                    S[4 * i] *= w.x; S[4 * i + 1] *= w.y; S[4 * i + 2] *= w.z; S[4 * i + 3] *= w.w;
+                    q0 = fmaf(S[4 * i], rv.x, q0);
+                    q1 = fmaf(S[4 * i + 1], rv.y, q1);
+                    q0 = fmaf(S[4 * i + 2], rv.z, q0);
+                    q1 = fmaf(S[4 * i + 3], rv.w, q1);
+                }
+                float p = p0 + p1, q = q0 + q1;
+                for (int o = 1; o < P; o <<= 1) {
+                    p += __shfl_xor_sync(0xffffffffu, p, o);
+                    q += __shfl_xor_sync(0xffffffffu, q, o);
+                }
+                const float v = vs[tt * DVT + cl], knv = sc[tt * 4] * v;
+#pragma unroll
+                for (int i = 0; i < DKP / 4; ++i) {
+                    const float4 u = u4[i], a = a4[i];
+                    S[4 * i] = fmaf(u.x, fmaf(-a.x, p, knv), S[4 * i]);
+                    S[4 * i + 1] = fmaf(u.y, fmaf(-a.y, p, knv), S[4 * i + 1]);
+                    S[4 * i + 2] = fmaf(u.z, fmaf(-a.z, p, knv), S[4 * i + 2]);
+                    S[4 * i + 3] = fmaf(u.w, fmaf(-a.w, p, knv), S[4 * i + 3]);
+                }
+                if (part == 0) os[tt * DVT + cl] = fmaf(sc[tt * 4 + 2], v, fmaf(-sc[tt * 4 + 1], p, q));
+            }
+        }
+        __syncthreads();
+        for (int idx = tid; idx < tc * DVT; idx += nthreads) {
+            const int tt = idx / DVT, j = idx - tt * DVT, c = col0 + j;
+            if (c < A.dv) A.out[(size_t)(c0 + tt) * A.ldo + h * A.dv + c] = os[idx];
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < DKP; ++i) {
+        const int kr = part * DKP + i;
+        if (col_ok && kr < A.dk) st[(size_t)kr * A.dv + col] = S[i];
+    }
+}
+
+// Floats of a (token, head) row of the prepared inputs, a multiple of 4 (ops.py has the same formula).
+__host__ __device__ static inline int gd_work_row(int dk, int dv) { return (4 * dk + dv + 4 + 3) / 4 * 4; }
+
+template <typename T>
+__global__ void __launch_bounds__(128) general_delta_prepare_kernel(GDeltaArgs A, float* __restrict__ work, int n) {
+    pdl_start();
+    const int lane = threadIdx.x & 31;
+    const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (item >= (long long)n * A.H) return;
+    const size_t row = (size_t)(item / A.H);
+    const int h = (int)(item % A.H), dk = A.dk;
+    float* w = work + (size_t)item * gd_work_row(dk, A.dv);
+    float kn, ra, rk;
+    gd_inputs<T>(A, row, h, lane, [&](int i, float rv, float u, float wv, float a) {
+        w[i] = rv;
+        w[dk + i] = u;
+        w[2 * dk + i] = wv;
+        w[3 * dk + i] = a;
+    }, kn, ra, rk);
+    const T* vp = (const T*)A.v + row * A.ldv + h * A.dv;
+    for (int i = lane; i < A.dv; i += 32) w[4 * dk + i] = to_f32<T>(vp[i]);
+    if (lane < 4) w[4 * dk + A.dv + lane] = lane == 0 ? kn : lane == 1 ? ra : lane == 2 ? rk : 0.0f;
+}
+
+__device__ __forceinline__ void gd_copy(float* smem, const float* gmem, int bytes) {
+    const uint32_t dst = (uint32_t)__cvta_generic_to_shared(smem);
+    if (bytes == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(gmem) : "memory");
+    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(gmem) : "memory");
+}
+
+// Grid (request, head, tile of DVT value channels), P lanes of a warp per column of S, DKP rows of the column in a thread.
+template <int DKP>
+__global__ void __launch_bounds__(128) general_delta_walk_kernel(GDeltaArgs A, const float* __restrict__ work, int P, int DVT) {
+    extern __shared__ __align__(16) float sm[];
+    pdl_start();
+    const int r = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * DVT;
+    const int tid = threadIdx.x, nthreads = blockDim.x;
+    const int part = tid % P, cl = tid / P, col = col0 + cl;
+    const bool col_ok = cl < DVT && col < A.dv;
+    const int pstride = DKP + 4, tstride = P * pstride, dk = A.dk, TC = A.chunk, wrow = gd_work_row(dk, A.dv);
+    // two buffers of a chunk's rows: [r, u, w, a: TC x tstride each][v: TC x DVT][scalars: TC x 4], then the outputs [TC x DVT]
+    const int buf_floats = TC * (4 * tstride + DVT + 4);
+    float* os = sm + 2 * buf_floats;
+    const int row0 = A.q_start[r], row1 = A.q_start[r + 1];
+    float* st = A.state + (((size_t)A.state_slots[r] * A.H + h) * dk) * A.dv;
+    float S[DKP];
+#pragma unroll
+    for (int i = 0; i < DKP; ++i) {
+        const int kr = part * DKP + i;
+        S[i] = (col_ok && kr < dk) ? st[(size_t)kr * A.dv + col] : 0.0f;
+    }
+    // key channels beyond dk, written once (the copies never touch them)
+    for (int idx = tid; idx < 2 * TC * P * DKP; idx += nthreads) {
+        const int b = idx / (TC * P * DKP), rest = idx - b * (TC * P * DKP);
+        const int tt = rest / (P * DKP), i = rest - tt * (P * DKP);
+        if (i >= dk) {
+            float* base = sm + b * buf_floats + tt * tstride + (i / DKP) * pstride + i % DKP;
+            base[0] = 0.0f;
+            base[TC * tstride] = 0.0f;
+            base[2 * TC * tstride] = 1.0f;
+            base[3 * TC * tstride] = 0.0f;
+        }
+    }
+    const bool wide = (dk & 3) == 0;
+    const int piece = wide ? 4 : 1, pieces = dk / piece;
+    auto fetch = [&](int c0, int b) {
+        const int tc = min(TC, row1 - c0);
+        float* base = sm + b * buf_floats;
+        float* vs = base + 4 * TC * tstride;
+        float* sc = vs + TC * DVT;
+        for (int idx = tid; idx < tc * pieces; idx += nthreads) {
+            const int tt = idx / pieces, i = (idx - tt * pieces) * piece;
+            const float* w = work + ((size_t)(c0 + tt) * A.H + h) * wrow + i;
+            float* at = base + tt * tstride + (i / DKP) * pstride + i % DKP;
+            gd_copy(at, w, 4 * piece);
+            gd_copy(at + TC * tstride, w + dk, 4 * piece);
+            gd_copy(at + 2 * TC * tstride, w + 2 * dk, 4 * piece);
+            gd_copy(at + 3 * TC * tstride, w + 3 * dk, 4 * piece);
+        }
+        for (int idx = tid; idx < tc * DVT; idx += nthreads) {
+            const int tt = idx / DVT, j = idx - tt * DVT, c = col0 + j;
+            if (c < A.dv) gd_copy(vs + idx, work + ((size_t)(c0 + tt) * A.H + h) * wrow + 4 * dk + c, 4);
+        }
+        for (int idx = tid; idx < 3 * tc; idx += nthreads) {
+            const int tt = idx / 3, j = idx - tt * 3;
+            gd_copy(sc + tt * 4 + j, work + ((size_t)(c0 + tt) * A.H + h) * wrow + 4 * dk + A.dv + j, 4);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (row0 < row1) fetch(row0, 0);
+    int b = 0;
+    for (int c0 = row0; c0 < row1; c0 += TC, b ^= 1) {
+        const int tc = min(TC, row1 - c0);
+        if (c0 + TC < row1) {
+            fetch(c0 + TC, b ^ 1);                 // its buffer was walked two chunks ago; the barriers since cover it
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();                           // everybody's copies of this chunk have landed; the outputs before are stored
+        const float* base = sm + b * buf_floats;
+        const float* vs = base + 4 * TC * tstride;
+        const float* sc = vs + TC * DVT;
+        if (cl < DVT) {
+            // the rows of the token after this one are read while this one's sums run; two register sets take turns
+            struct Rows { float4 r[DKP / 4], u[DKP / 4], w[DKP / 4], a[DKP / 4]; float kn, ra, rk, v; };
+            const float* mine = base + part * pstride;
+            auto read = [&](Rows& x, int tt) {
+                const float* at = mine + tt * tstride;
+#pragma unroll
+                for (int i = 0; i < DKP / 4; ++i) {
+                    x.r[i] = reinterpret_cast<const float4*>(at)[i];
+                    x.u[i] = reinterpret_cast<const float4*>(at + TC * tstride)[i];
+                    x.w[i] = reinterpret_cast<const float4*>(at + 2 * TC * tstride)[i];
+                    x.a[i] = reinterpret_cast<const float4*>(at + 3 * TC * tstride)[i];
+                }
+                x.kn = sc[4 * tt];
+                x.ra = sc[4 * tt + 1];
+                x.rk = sc[4 * tt + 2];
+                x.v = col_ok ? vs[tt * DVT + cl] : 0.0f;
+            };
+            auto token = [&](const Rows& x, Rows& next, int tt) {
+                if (tt + 1 < tc) read(next, tt + 1);
+                float p0 = 0.0f, p1 = 0.0f, p2 = 0.0f, p3 = 0.0f, q0 = 0.0f, q1 = 0.0f, q2 = 0.0f, q3 = 0.0f;
+#pragma unroll
+                for (int i = 0; i < DKP / 4; ++i) {
+                    p0 = fmaf(S[4 * i], x.u[i].x, p0);
+                    p1 = fmaf(S[4 * i + 1], x.u[i].y, p1);
+                    p2 = fmaf(S[4 * i + 2], x.u[i].z, p2);
+                    p3 = fmaf(S[4 * i + 3], x.u[i].w, p3);
+                    S[4 * i] *= x.w[i].x; S[4 * i + 1] *= x.w[i].y; S[4 * i + 2] *= x.w[i].z; S[4 * i + 3] *= x.w[i].w;
+                    q0 = fmaf(S[4 * i], x.r[i].x, q0);
+                    q1 = fmaf(S[4 * i + 1], x.r[i].y, q1);
+                    q2 = fmaf(S[4 * i + 2], x.r[i].z, q2);
+                    q3 = fmaf(S[4 * i + 3], x.r[i].w, q3);
+                }
+                float p = (p0 + p1) + (p2 + p3), q = (q0 + q1) + (q2 + q3);
+#pragma unroll
+                for (int o = 1; o < 32; o <<= 1) {
+                    if (o < P) {
+                        p += __shfl_xor_sync(0xffffffffu, p, o);
+                        q += __shfl_xor_sync(0xffffffffu, q, o);
+                    }
+                }
+                const float knv = x.kn * x.v;
+#pragma unroll
+                for (int i = 0; i < DKP / 4; ++i) {
+                    S[4 * i] = fmaf(x.u[i].x, fmaf(-x.a[i].x, p, knv), S[4 * i]);
+                    S[4 * i + 1] = fmaf(x.u[i].y, fmaf(-x.a[i].y, p, knv), S[4 * i + 1]);
+                    S[4 * i + 2] = fmaf(x.u[i].z, fmaf(-x.a[i].z, p, knv), S[4 * i + 2]);
+                    S[4 * i + 3] = fmaf(x.u[i].w, fmaf(-x.a[i].w, p, knv), S[4 * i + 3]);
+                }
+                if (part == 0) os[tt * DVT + cl] = fmaf(x.rk, x.v, fmaf(-x.ra, p, q));
+            };
+            Rows even, odd;
+            read(even, 0);
+            for (int tt = 0; tt < tc; tt += 2) {
+                token(even, odd, tt);
+                if (tt + 1 < tc) token(odd, even, tt + 1);
+            }
+        }
+        __syncthreads();
+        for (int idx = tid; idx < tc * DVT; idx += nthreads) {
+            const int tt = idx / DVT, j = idx - tt * DVT, c = col0 + j;
+            if (c < A.dv) A.out[(size_t)(c0 + tt) * A.ldo + h * A.dv + c] = os[idx];
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < DKP; ++i) {
+        const int kr = part * DKP + i;
+        if (col_ok && kr < dk) st[(size_t)kr * A.dv + col] = S[i];
+    }
+}
+
+constexpr int GD_WALK_SMEM = 80 * 1024;
+
+template <int DKP>
+static int launch_gd_walk(const GDeltaArgs& A, dim3 grid, int threads, size_t bytes, const float* work, int P, int dvt, cudaStream_t s) {
+    static unsigned long long configured = 0;
+    if (int e = vcb_allow_dynamic_smem(general_delta_walk_kernel<DKP>, GD_WALK_SMEM, &configured)) return e;
+    vcb_launch(general_delta_walk_kernel<DKP>, grid, threads, bytes, s, A, work, P, dvt);
+    return vcb_last_error();
+}
+
+template <typename T>
+static int launch_gd_scan(const GDeltaArgs& A, int n_reqs, cudaStream_t s) {
+    const int dkp = A.dk <= 32 ? 8 : A.dk <= 64 ? 16 : 32;
+    int P = 1;
+    while (P * dkp < A.dk) P <<= 1;
+    if (P > 32) return VCB_ERR_UNSUPPORTED;
+    const int dvt = P <= 8 ? 32 : 256 / P;
+    const int threads = ((dvt * P + 31) / 32) * 32;
+    int chunk = 8;
+    auto bytes = [&](int tc) { return ((size_t)tc * (4 * P * (dkp + 4) + 2 * dvt + 4)) * sizeof(float); };
+    while (chunk > 1 && bytes(chunk) > 48 * 1024) chunk >>= 1;
+    GDeltaArgs B = A;
+    B.chunk = chunk;
+    dim3 grid(n_reqs, A.H, (A.dv + dvt - 1) / dvt);
+    if (dkp == 8) vcb_launch(general_delta_scan_kernel<T, 8>, grid, threads, bytes(chunk), s, B, P, dvt);
+    else if (dkp == 16) vcb_launch(general_delta_scan_kernel<T, 16>, grid, threads, bytes(chunk), s, B, P, dvt);
+    else vcb_launch(general_delta_scan_kernel<T, 32>, grid, threads, bytes(chunk), s, B, P, dvt);
+    return vcb_last_error();
+}
+
+template <typename T>
+static int launch_gd_portions(const GDeltaArgs& A, int n_reqs, int n_tokens, float* work, cudaStream_t s) {
+    const int dkp = A.dk > 256 ? 16 : 8;
+    int P = 1;
+    while (P * dkp < A.dk) P <<= 1;
+    const int dvt = 128 / P >= 32 ? 32 : 128 / P;
+    int chunk = 16;
+    auto bytes = [&](int tc) { return (size_t)tc * (2 * (4 * P * (dkp + 4) + dvt + 4) + dvt) * sizeof(float); };
+    while (chunk > 4 && bytes(chunk) > GD_WALK_SMEM) chunk >>= 1;
+    if (P > 32 || bytes(chunk) > GD_WALK_SMEM) return launch_gd_scan<T>(A, n_reqs, s);     // very long keys: the kernel above
+    const long long items = (long long)n_tokens * A.H;
+    vcb_launch(general_delta_prepare_kernel<T>, dim3((unsigned)((items + 3) / 4)), 128, 0, s, A, work, n_tokens);
+    if (int e = vcb_last_error()) return e;
+    GDeltaArgs B = A;
+    B.chunk = chunk;
+    dim3 grid(n_reqs, A.H, (A.dv + dvt - 1) / dvt);
+    const int threads = dvt * P;
+    if (dkp == 8) return launch_gd_walk<8>(B, grid, threads, bytes(chunk), work, P, dvt, s);
+    return launch_gd_walk<16>(B, grid, threads, bytes(chunk), work, P, dvt, s);
+}
+
+VCB_EXPORT int vcb_general_delta(const void* r, long long ldr, const void* k, long long ldk, const void* v, long long ldv,
+                                 const void* a_pre, long long lda, const void* z, long long ldz, const float* a_bias, const float* z_bias,
+                                 float* state, float* out, long long ldo, const int* q_start, const int* state_slots, int n_reqs, int H,
+                                 int dk, int dv, float rate, float unit_eps, float* work, int n_tokens, int dtype, void* stream) {
+    if (n_reqs <= 0) return 0;
+    if (!r || !k || !v || !a_pre || !z || !state || !out || H <= 0 || dk <= 0 || dv <= 0 || H > 65535 || (dv + 7) / 8 > 65535) return VCB_ERR_BAD_ARG;
+    GDeltaArgs A{r, k, v, a_pre, z, ldr, ldk, ldv, lda, ldz, a_bias, z_bias, state, out, ldo, q_start, state_slots, H, dk, dv, rate, unit_eps, 0};
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype != VCB_F32 && dtype != VCB_BF16) return VCB_ERR_BAD_ARG;
+    if (work && n_tokens > 0)
+        return dtype == VCB_F32 ? launch_gd_portions<float>(A, n_reqs, n_tokens, work, s) : launch_gd_portions<__nv_bfloat16>(A, n_reqs, n_tokens, work, s);
+    return dtype == VCB_F32 ? launch_gd_scan<float>(A, n_reqs, s) : launch_gd_scan<__nv_bfloat16>(A, n_reqs, s);
+}
+
+// ------------------------------------------------------------------------------- out = tanh(x), rows of T
+template <typename T>
+__global__ void tanh_rows_kernel(const T* __restrict__ x, long long ldx, T* __restrict__ out, long long ldo, int n, int width) {
+    pdl_start();
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < (long long)n * width; i += (long long)gridDim.x * blockDim.x) {
+        const long long t = i / width;
+        const int c = (int)(i - t * width);
+        out[t * ldo + c] = from_f32<T>(tanhf(to_f32<T>(x[t * ldx + c])));
+    }
+}
+
+VCB_EXPORT int vcb_tanh_rows(const void* x, long long ldx, void* out, long long ldo, int n, int width, int dtype, void* stream) {
+    if (n <= 0 || width <= 0) return 0;
+    if (!x || !out) return VCB_ERR_BAD_ARG;
+    const long long total = (long long)n * width;
+    const int blocks = (int)((total + 255) / 256 < vcb_sm_count() * 8 ? (total + 255) / 256 : vcb_sm_count() * 8);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == VCB_F32) vcb_launch(tanh_rows_kernel<float>, blocks, 256, 0, s, (const float*)x, ldx, (float*)out, ldo, n, width);
+    else if (dtype == VCB_BF16) vcb_launch(tanh_rows_kernel<__nv_bfloat16>, blocks, 256, 0, s, (const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)out, ldo, n, width);
+    else return VCB_ERR_BAD_ARG;
+    return vcb_last_error();
+}

@@ -31,6 +31,7 @@ _SIGNATURES = {
     "vcb_embedding": [_P, _P, _P, _I, _I, _I, _P],
     "vcb_add_rmsnorm": [_P, _P, _P, _P, _P, _I, _I, _F, _I, _P],
     "vcb_silu_mul": [_P, _P, _I, _I, _I, _P],
+    "vcb_relu_mul": [_P, _P, _I, _I, _I, _P],
     "vcb_add_bias": [_P, _P, _I, _I, _I, _P],
     "vcb_rope_cache_write": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
     "vcb_attention_simt": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P],
@@ -40,6 +41,8 @@ _SIGNATURES = {
     "vcb_gemm_bf16_tcgen05": [_P, _I, _I, _P, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P],
     "vcb_gemm_bf16_tcgen05_fused": [_P, _I, _I, _P, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P,
                                     _P, _I, _I, _I, _F, _P, _I, _P, _P, _I, _I, _P],
+    "vcb_gemm_bf16_tcgen05_fused_act": [_P, _I, _I, _P, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P,
+                                        _P, _I, _I, _I, _F, _P, _I, _P, _P, _I, _I, _I, _P],
     "vcb_tile_weights": [_P, _I, _I, _I, _I, _P, _P],
     "vcb_repetition_penalty": [_P, _I, _P, _P, _P, _I, _I, _P],
     "vcb_sample": [_P, _I, _I, _P, _P, _P, _I, _P],
@@ -83,6 +86,14 @@ _SIGNATURES = {
     "vcb_stream_norm": [_P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _F, _F, _I, _P],
     "vcb_stream_join": [_P, _L, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _P],
     "vcb_causal_conv": [_P, _L, _P, _P, _P, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "vcb_causal_conv_as": [_P, _L, _P, _P, _P, _P, _L, _P, _L, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "vcb_conv_rope_cache_write": [_P, _L, _P, _P, _I, _P, _L, _P, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
+    "vcb_pool_blocks": [_P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
+    "vcb_attention_pooled": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _I, _P],
+    "vcb_selective_scan": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P],
+    "vcb_general_delta": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _F, _F, _P, _I, _I, _P],
+    "vcb_tanh_rows": [_P, _L, _P, _L, _I, _I, _I, _P],
+    "vcb_pair_norm": [_P, _P, _P, _P, _F, _F, _F, _P, _P, _P, _P, _I, _I, _F, _F, _I, _P],
     "vcb_gate_blocks": [_P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _F, _I, _P],
     "vcb_linear_recurrence": [_P, _P, _L, _P, _L, _P, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _P],
     "vcb_gated_delta_scan": [_P, _P, _P, _L, _L, _L, _P, _L, _P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _P, _I, _P],
@@ -224,6 +235,14 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
     _need(gate_up.shape == (n, 2 * inter) and gate_up.dtype == out.dtype, "silu_mul: gate_up must be [n, 2*inter]")
     _check(lib().vcb_silu_mul(_dev(gate_up, "gate_up"), _dev(out, "out"), n, inter,
                               dtype_code(out.dtype), _stream()), "silu_mul")
+
+
+def relu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
+    """out[t, i] = max(gate_up[t, i], 0) * gate_up[t, inter + i]."""
+    n, inter = out.shape
+    _need(gate_up.shape == (n, 2 * inter) and gate_up.dtype == out.dtype, "relu_mul: gate_up must be [n, 2*inter]")
+    _check(lib().vcb_relu_mul(_dev(gate_up, "gate_up"), _dev(out, "out"), n, inter,
+                              dtype_code(out.dtype), _stream()), "relu_mul")
 
 
 def cast_rows(x: torch.Tensor, delta: Optional[torch.Tensor], mult: float, out: torch.Tensor) -> None:
@@ -545,12 +564,12 @@ def sumsq_parts(features: int) -> int:
 
 def gemm_bf16_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan=None, max_ctas: Optional[int] = None,
                       use_tiled: bool = True, x_scale: Optional[RowScale] = None,
-                      fuse: Optional[ResidualNorm] = None, gated: bool = False) -> None:
+                      fuse: Optional[ResidualNorm] = None, gated: bool = False, gate_act: str = "silu") -> None:
     """out = x @ w^T on tcgen05 tensor cores fed by TMA (see gemm_tcgen05.cu); out bfloat16 or float32.
     When the weights are the 128-row operand and tile_weights(w) has been made, the image is used
     (``use_tiled`` False forces the tensor-map path).  ``x_scale`` and ``fuse`` (up to 128 tokens):
     see RowScale and ResidualNorm.  ``gated``: w is a gate-and-up matrix [2 * inter, k] with a gated
-    image (tile_weights(w, inter)) and out [tokens, inter] = silu(x gate^T) * (x up^T)."""
+    image (tile_weights(w, inter)) and out [tokens, inter] = act(x gate^T) * (x up^T), act "silu" or "relu"."""
     m, k = x.shape
     n = w.shape[0]
     _need(w.shape[1] == k and out.shape == (m, n // 2 if gated else n), "gemm_bf16_tcgen05: shapes do not agree")
@@ -592,14 +611,16 @@ def gemm_bf16_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan=
         max_ctas = _cta_choice.get((n, k, bn, bool(gated), fuse is not None), 2 * sms if bn in (32, 64) else sms)
     partial = scratch("gemm_partial", sms * 2 * 256 * 128, out.device)
     tickets = zeroed_ints("gemm_tickets", GEMM_MAX_TICKETS, out.device)
-    _check(lib().vcb_gemm_bf16_tcgen05_fused(p.data_ptr(), p.shape[0], p.stride(0),
+    _check(lib().vcb_gemm_bf16_tcgen05_fused_act(p.data_ptr(), p.shape[0], p.stride(0),
                                              None if tiled is None else tiled.data_ptr(),
                                              q.data_ptr(), q.shape[0], q.stride(0), k,
                                              out.data_ptr(), out.stride(0), 1 if out.dtype == torch.float32 else 0,
                                              1 if swapped else 0, bn, min(max_ctas, 2 * sms), partial.data_ptr(),
                                              tickets.data_ptr(), GEMM_MAX_TICKETS, status_tensor(out.device).data_ptr(),
-                                             *sc, *fu, n // 2 if gated else 0, _stream()), "gemm_bf16_tcgen05")
+                                             *sc, *fu, n // 2 if gated else 0, GATE_ACTS[gate_act], _stream()), "gemm_bf16_tcgen05")
 
+
+GATE_ACTS = {"silu": 0, "relu": 1}      # activations of the gated product's epilogue
 
 TCGEN05_MAX_TOKENS = 128      # up to here the engine's own tcgen05 product may run; above, the library's
 _tcgen05_linear = True
@@ -859,11 +880,12 @@ def linear_gated_fuses(tokens: int, w: torch.Tensor) -> bool:
         and _linear_choice.get((w.shape[0], w.shape[1], token_bucket(tokens), torch.bfloat16), True)
 
 
-def linear_gated(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_scale: Optional[RowScale] = None) -> None:
-    """out [tokens, inter] = silu(x gate^T) * (x up^T) for w = [gate; up] ([2 * inter, k]) in one kernel;
-    only where ``linear_gated_fuses`` said yes."""
+def linear_gated(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_scale: Optional[RowScale] = None,
+                 gate_act: str = "silu") -> None:
+    """out [tokens, inter] = act(x gate^T) * (x up^T) for w = [gate; up] ([2 * inter, k]) in one kernel (act "silu" or
+    "relu"); only where ``linear_gated_fuses`` said yes."""
     _need(linear_gated_fuses(x.shape[0], w), "linear_gated: ask linear_gated_fuses first")
-    gemm_bf16_tcgen05(x, w, out, x_scale=x_scale, gated=True)
+    gemm_bf16_tcgen05(x, w, out, x_scale=x_scale, gated=True, gate_act=gate_act)
 
 
 # ------------------------------------------------- residual stream: shift, gates, norms on results
@@ -1266,7 +1288,7 @@ def stream_join(x: torch.Tensor, y: torch.Tensor, mix: torch.Tensor, out_coef: t
 
 
 # ------------------------------------------------- recurrent mixers behind a short convolution
-CONV_MAX_TAPS = 8
+CONV_MAX_TAPS = 64
 
 
 def causal_conv(x: torch.Tensor, taps: torch.Tensor, state: torch.Tensor, out: torch.Tensor, q_start, state_slots, n_reqs: int,
@@ -1275,11 +1297,13 @@ def causal_conv(x: torch.Tensor, taps: torch.Tensor, state: torch.Tensor, out: t
     """out[t, c] = act(sum_j taps[c, j] * in[t - (J - 1) + j, c] + bias[c]) over each request's tokens, in = x + pre_bias;
     the J - 1 inputs before a request's first token of the step come from its slot of ``state`` (float32
     [slots, >= J - 1 rows, C] as a strided view: rows 0 .. J - 2, oldest first; zero at admission), which then receives the
-    step's last J - 1 inputs.  x rows of the activations' type [n, C]; taps float32 [C, J]; out float32 [n, C] rows."""
+    step's last J - 1 inputs.  x rows of the activations' type [n, C]; taps float32 [C, J]; out rows [n, C], float32 or of x's
+    type."""
     n, C = x.shape
     J = taps.shape[1]
     _rows(x, "x", x.dtype)
-    _rows(out, "out", torch.float32)
+    _rows(out, "out", out.dtype)
+    _need(out.dtype in (torch.float32, x.dtype), "causal_conv: out float32 or like x")
     _need(out.shape == (n, C) and taps.shape[0] == C and 1 <= J <= CONV_MAX_TAPS, f"causal_conv: taps [C, up to {CONV_MAX_TAPS}]")
     _need(act in ("none", "silu"), "causal_conv: act is 'none' or 'silu'")
     _need(state.dtype == torch.float32 and state.dim() == 3 and state.shape[2] == C and state.shape[1] >= J - 1
@@ -1287,9 +1311,9 @@ def causal_conv(x: torch.Tensor, taps: torch.Tensor, state: torch.Tensor, out: t
           "causal_conv: state float32 [slots, J - 1, C] with contiguous rows")
     for t, name in ((pre_bias, "pre_bias"), (bias, "bias")):
         _need(t is None or t.numel() == C, f"causal_conv: {name} [C]")
-    _check(lib().vcb_causal_conv(x.data_ptr(), x.stride(0), None if pre_bias is None else _dev(pre_bias, "pre_bias", torch.float32),
+    _check(lib().vcb_causal_conv_as(x.data_ptr(), x.stride(0), None if pre_bias is None else _dev(pre_bias, "pre_bias", torch.float32),
                                  _dev(taps, "taps", torch.float32), None if bias is None else _dev(bias, "bias", torch.float32),
-                                 state.data_ptr(), state.stride(0), out.data_ptr(), out.stride(0),
+                                 state.data_ptr(), state.stride(0), out.data_ptr(), out.stride(0), 1 if out.dtype == torch.float32 else 0,
                                  _dev(q_start, "q_start", torch.int32), _dev(state_slots, "state_slots", torch.int32), n_reqs,
                                  max_q_len, C, J, 1 if act == "silu" else 0, dtype_code(x.dtype), _stream()), "causal_conv")
 
@@ -1378,6 +1402,159 @@ def gated_delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta_pre
                                       _dev(state_slots, "state_slots", torch.int32), n_reqs, H, G, dk, dv, float(q_scale),
                                       float(unit_eps), dtype_code(beta_pre.dtype), work.data_ptr() if portions else None,
                                       n if portions else 0, _stream()), "gated_delta_scan")
+
+
+# ------------------------------------------------- attention over a window of tokens and means of blocks before it
+def conv_rope_cache_write(proj: torch.Tensor, bias: Optional[torch.Tensor], taps: torch.Tensor, state: torch.Tensor,
+                          inv_freq: Optional[torch.Tensor], q_factor: Optional[torch.Tensor], q_out: torch.Tensor, cache: torch.Tensor,
+                          q_start, positions, state_slots, block_table, n_reqs: int, max_q_len: int, *, num_heads: int, num_kv_heads: int,
+                          head_dim: int, v_head_dim: int, row: int, page_size: int) -> None:
+    """proj rows [n, C] hold q, k and v one after the other, C = heads * head_dim + kv heads * (head_dim + v_head_dim).
+    u = proj + bias passes a causal convolution over time per channel (``taps`` float32 [C, J], last column the current token's;
+    the J - 1 inputs before a portion come from the request's slot of ``state``, float32 [slots, >= J - 1, C], zero at admission,
+    and the last J - 1 are left there), then the pairs (2i, 2i + 1) of q and k with i < len(inv_freq) turn by
+    positions * inv_freq[i] (None: no rotation) and a head's queries are multiplied by ``q_factor`` (float32 [heads] or None).
+    Queries go to q_out [n, heads * head_dim], keys and values to the token's slot of the cache (rows of ``row`` elements)."""
+    n, C = proj.shape
+    _rows(proj, "proj", q_out.dtype)
+    J = taps.shape[1]
+    rot = 0 if inv_freq is None else 2 * inv_freq.numel()
+    _need(C == num_heads * head_dim + num_kv_heads * (head_dim + v_head_dim) and taps.shape[0] == C and 1 <= J <= CONV_MAX_TAPS,
+          f"conv_rope_cache_write: proj [n, C], taps [C, up to {CONV_MAX_TAPS}]")
+    _need(bias is None or bias.numel() == C, "conv_rope_cache_write: bias [C]")
+    _need(state.dtype == torch.float32 and state.dim() == 3 and state.shape[2] == C and state.shape[1] >= max(1, J - 1)
+          and state.is_contiguous(), "conv_rope_cache_write: state float32 [slots, J - 1, C]")
+    _need(rot <= head_dim and (q_factor is None or q_factor.numel() == num_heads), "conv_rope_cache_write: rotation, one factor per head")
+    _need(q_out.shape == (n, num_heads * head_dim) and cache.dtype == q_out.dtype, "conv_rope_cache_write: q_out, cache")
+    _check(lib().vcb_conv_rope_cache_write(
+        proj.data_ptr(), proj.stride(0), None if bias is None else _dev(bias, "bias", torch.float32), _dev(taps, "taps", torch.float32), J,
+        state.data_ptr(), state.stride(0), None if inv_freq is None else _dev(inv_freq, "inv_freq", torch.float32), rot,
+        None if q_factor is None else _dev(q_factor, "q_factor", torch.float32), _dev(q_out, "q_out"), _dev(cache, "cache"),
+        _dev(q_start, "q_start", torch.int32), _dev(positions, "positions", torch.int32), _dev(state_slots, "state_slots", torch.int32),
+        _dev(block_table, "block_table", torch.int32), block_table.shape[1], n_reqs, max_q_len, num_heads, num_kv_heads, head_dim,
+        v_head_dim, row, page_size, cache.shape[0], status_tensor(proj.device).data_ptr(), dtype_code(q_out.dtype), _stream()),
+        "conv_rope_cache_write")
+
+
+def pool_blocks(cache: torch.Tensor, pooled: torch.Tensor, q_start, ctx_lens, block_table, pool_table, n_reqs: int, max_q_len: int, *,
+                num_kv_heads: int, head_dim: int, v_head_dim: int, row: int, page_size: int, pool: int) -> None:
+    """For every block of ``pool`` tokens whose last token this step brought: the mean of its keys and of its values as the
+    cache holds them into row b of the request's pages in ``pooled`` (same layout, ``pool_table`` its block table)."""
+    _need(cache.dtype == pooled.dtype and cache.shape[1:] == pooled.shape[1:], "pool_blocks: one page layout for tokens and blocks")
+    _check(lib().vcb_pool_blocks(_dev(cache, "cache"), _dev(pooled, "pooled"), _dev(q_start, "q_start", torch.int32),
+                                 _dev(ctx_lens, "ctx_lens", torch.int32), _dev(block_table, "block_table", torch.int32), block_table.shape[1],
+                                 _dev(pool_table, "pool_table", torch.int32), pool_table.shape[1], n_reqs, max_q_len, num_kv_heads,
+                                 head_dim, v_head_dim, row, page_size, cache.shape[0], pooled.shape[0], pool,
+                                 status_tensor(cache.device).data_ptr(), dtype_code(cache.dtype), _stream()), "pool_blocks")
+
+
+def attention_pooled(q: torch.Tensor, cache: torch.Tensor, pooled: Optional[torch.Tensor], out: torch.Tensor, positions, req_of_token,
+                     block_table, pool_table: Optional[torch.Tensor], *, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int,
+                     row: int, page_size: int, window: int, pool: int, scale: float) -> None:
+    """Plain form, both types: softmax over the tokens j with 0 <= i - j < window (0: all) and, with ``pool`` P > 0 and a window,
+    the means of the blocks b with (b + 1) P - 1 <= i - window (``pooled`` pages, ``pool_table``)."""
+    _need(q.dtype == cache.dtype == out.dtype, "attention_pooled: one type")
+    _need(head_dim <= 1024 and v_head_dim <= 512, "attention_pooled: head sizes up to 1024 (keys) and 512 (values)")
+    with_pool = pool > 0 and window > 0
+    _need(not with_pool or (pooled is not None and pool_table is not None and pooled.dtype == q.dtype), "attention_pooled: pages of blocks")
+    _check(lib().vcb_attention_pooled(_dev(q, "q"), _dev(cache, "cache"), _dev(pooled, "pooled") if with_pool else None, _dev(out, "out"),
+                                      _dev(positions, "positions", torch.int32), _dev(req_of_token, "req_of_token", torch.int32),
+                                      _dev(block_table, "block_table", torch.int32), block_table.shape[1],
+                                      _dev(pool_table, "pool_table", torch.int32) if with_pool else None,
+                                      pool_table.shape[1] if with_pool else 0, q.shape[0], num_heads, num_kv_heads, head_dim, v_head_dim,
+                                      row, page_size, window, pool if with_pool else 0, float(scale), cache.shape[0],
+                                      pooled.shape[0] if with_pool else 0, status_tensor(q.device).data_ptr(), dtype_code(q.dtype),
+                                      _stream()), "attention_pooled")
+
+
+# ------------------------------------------------- selective state space, generalised delta rule, joined results
+SELECTIVE_MAX_STATE = 512
+
+
+def selective_scan(x: torch.Tensor, dt_pre: torch.Tensor, b: torch.Tensor, c: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor,
+                   a_log2: torch.Tensor, d: torch.Tensor, state: torch.Tensor, out: torch.Tensor, q_start, state_slots, n_reqs: int,
+                   max_q_len: int) -> None:
+    """Per request and channel c over the step's tokens, S (float32 [N]) read from and left in the request's slot of ``state``
+    [slots, I, N]:  dt = softplus(dt_pre + dt_bias);  S <- 2^(dt * a_log2[c]) S + dt x B;  y = S . C + d x;  out = y * silu(z).
+    x, dt_pre, z, out rows [n, I], b, c rows [n, N] of the activations' type (strided views allowed); a_log2 = A * log2(e)."""
+    n, I = x.shape
+    N = b.shape[1]
+    for t, name in ((x, "x"), (dt_pre, "dt_pre"), (b, "b"), (c, "c"), (z, "z"), (out, "out")):
+        _rows(t, name, x.dtype)
+    _need(dt_pre.shape == z.shape == out.shape == (n, I) and b.shape == c.shape == (n, N), "selective_scan: shapes")
+    _need(a_log2.shape == (I, N) and dt_bias.numel() == I and d.numel() == I and 1 <= N <= SELECTIVE_MAX_STATE,
+          f"selective_scan: a_log2 [I, up to {SELECTIVE_MAX_STATE}], dt_bias and d [I]")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (I, N), "selective_scan: state float32 [slots, I, N]")
+    _check(lib().vcb_selective_scan(x.data_ptr(), x.stride(0), dt_pre.data_ptr(), dt_pre.stride(0), b.data_ptr(), b.stride(0), c.data_ptr(),
+                                    c.stride(0), z.data_ptr(), z.stride(0), _dev(dt_bias, "dt_bias", torch.float32),
+                                    _dev(a_log2, "a_log2", torch.float32), _dev(d, "d", torch.float32), state.data_ptr(), out.data_ptr(),
+                                    out.stride(0), _dev(q_start, "q_start", torch.int32), _dev(state_slots, "state_slots", torch.int32),
+                                    n_reqs, max_q_len, I, N, dtype_code(x.dtype), _stream()), "selective_scan")
+
+
+def general_delta_work(n: int, num_heads: int, head_dim: int, v_head_dim: int) -> int:
+    """Floats of the prepared inputs of ``n`` tokens (csrc/general_delta.cu, gd_work_row)."""
+    return n * num_heads * ((4 * head_dim + v_head_dim + 4 + 3) // 4 * 4)
+
+
+def general_delta(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a_pre: torch.Tensor, z: torch.Tensor, a_bias: Optional[torch.Tensor],
+                  z_bias: Optional[torch.Tensor], state: torch.Tensor, out: torch.Tensor, q_start, state_slots, n_reqs: int,
+                  max_q_len: int, *, num_heads: int, rate: float, unit_eps: float, work: Optional[torch.Tensor] = None) -> None:
+    """The generalised delta rule per request and head over the step's tokens, S (float32 [dk, dv]) read from and left in the
+    request's slot of ``state`` [slots, heads, dk, dv]:  u = k / sqrt(sum k^2 + unit_eps), w = exp(-rate * sigmoid(z + z_bias)),
+    a = sigmoid(a_pre + a_bias);  S <- diag(w) S - (a * u) (u^T S) + k v^T (both terms of the old S);  out = S^T r.
+    r, k, a_pre, z rows [n, heads * dk] and v [n, heads * dv] of the activations' type; out float32 [n, heads * dv].  Steps with a
+    portion of DELTA_PORTIONS_FROM tokens or more take ``work`` (float32, general_delta_work(...) elements)."""
+    n, H = r.shape[0], num_heads
+    _need(r.shape[1] % H == 0 and v.shape[1] % H == 0, "general_delta: head count")
+    dk, dv = r.shape[1] // H, v.shape[1] // H
+    for t, name in ((r, "r"), (k, "k"), (v, "v"), (a_pre, "a_pre"), (z, "z")):
+        _rows(t, name, r.dtype)
+    _rows(out, "out", torch.float32)
+    _need(k.shape == a_pre.shape == z.shape == r.shape and v.shape == out.shape == (n, H * dv), "general_delta: shapes")
+    _need(dk <= 1024 and all(t is None or t.numel() == H * dk for t in (a_bias, z_bias)), "general_delta: keys of up to 1024 channels, biases [heads * dk]")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dk, dv),
+          "general_delta: state float32 [slots, heads, dk, dv]")
+    portions = max_q_len >= DELTA_PORTIONS_FROM
+    if portions:
+        _need(work is not None and work.dtype == torch.float32 and work.is_contiguous() and work.numel() >= general_delta_work(n, H, dk, dv),
+              "general_delta: work too small")
+    _check(lib().vcb_general_delta(r.data_ptr(), r.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), a_pre.data_ptr(),
+                                   a_pre.stride(0), z.data_ptr(), z.stride(0), None if a_bias is None else _dev(a_bias, "a_bias", torch.float32),
+                                   None if z_bias is None else _dev(z_bias, "z_bias", torch.float32), state.data_ptr(), out.data_ptr(),
+                                   out.stride(0), _dev(q_start, "q_start", torch.int32), _dev(state_slots, "state_slots", torch.int32), n_reqs,
+                                   H, dk, dv, float(rate), float(unit_eps), work.data_ptr() if portions else None, n if portions else 0,
+                                   dtype_code(r.dtype), _stream()), "general_delta")
+    if portions:
+        add_launches(1)            # prepared, then walked
+
+
+def tanh_rows(x: torch.Tensor, out: torch.Tensor) -> None:
+    """out = tanh(x), rows of one type (strided views allowed), evaluated in float."""
+    _rows(x, "x", out.dtype)
+    _rows(out, "out", out.dtype)
+    _need(x.shape == out.shape, "tanh_rows: one shape")
+    _check(lib().vcb_tanh_rows(x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), x.shape[0], x.shape[1], dtype_code(x.dtype), _stream()),
+           "tanh_rows")
+
+
+def pair_norm(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch.Tensor, sa: float, sb: float, eps_ab: float,
+              out: Optional[torch.Tensor] = None, *, x: Optional[torch.Tensor] = None, gain: Optional[torch.Tensor] = None, eps: float = 0.0,
+              next_gain: Optional[torch.Tensor] = None, next_eps: float = 0.0) -> None:
+    """y = sa * rms(a) * wa + sb * rms(b) * wb with rms(u) = u / sqrt(mean(u^2) + eps_ab), in float.  Without ``x``: out = y.
+    With ``x`` (the float32 residual stream): x += rms(y; eps) * gain in place and, with ``out``, out = rms(x; next_eps) *
+    next_gain, the input of the sublayer that follows."""
+    n, hidden = a.shape
+    _need(b.shape == a.shape and a.dtype == b.dtype and wa.numel() == wb.numel() == hidden, "pair_norm: shapes")
+    _need(out is None or (out.shape == a.shape and out.dtype == a.dtype), "pair_norm: out like a")
+    _need(x is not None or out is not None, "pair_norm: nothing to write")
+    if x is not None:
+        _need(x.shape == a.shape and gain is not None and gain.numel() == hidden and (out is None or next_gain.numel() == hidden), "pair_norm: gains")
+    opt = lambda t, name: None if t is None else _dev(t, name, torch.float32)
+    _check(lib().vcb_pair_norm(_dev(a, "a"), _dev(b, "b"), _dev(wa, "wa", torch.float32), _dev(wb, "wb", torch.float32), float(sa), float(sb),
+                               float(eps_ab), opt(gain, "gain"), opt(x, "x"), opt(next_gain, "next_gain"),
+                               None if out is None else _dev(out, "out"), n, hidden, float(eps), float(next_eps), dtype_code(a.dtype), _stream()),
+           "pair_norm")
 
 
 # ------------------------------------------------------------------ latent attention

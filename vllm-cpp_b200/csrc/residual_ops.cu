@@ -447,3 +447,195 @@ VCB_EXPORT int vcb_norm_residual_norm(const void* y, const float* gain, float* x
         return VCB_ERR_BAD_ARG;
     return vcb_last_error();
 }
+
+// ------------------------------------- two results normed and joined, then as above
+// One CTA per row:  y = sa * (a / sqrt(mean(a^2) + eps_ab)) * wa + sb * (b / sqrt(mean(b^2) + eps_ab)) * wb.
+// x null: out = y.  Else y goes on in float as in norm_residual_norm_kernel:  x += (y / sqrt(mean(y^2) + eps)) * gain;
+// out (may be null) = (x / sqrt(mean(x^2) + eps_next)) * next_gain.
+struct PairNormArgs {
+    const void* a;
+    const void* b;
+    const float* wa;
+    const float* wb;
+    float sa, sb, eps_ab;
+    const float* gain;
+    float* x;
+    const float* next_gain;
+    void* out;
+    int hidden;
+    float eps, eps_next;
+};
+
+// Two sums over the CTA at once.
+__device__ __forceinline__ float2 block_sum2(float u, float v, float* scratch) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    u = warp_sum(u);
+    v = warp_sum(v);
+    __syncthreads();
+    if (lane == 0) { scratch[warp] = u; scratch[33 + warp] = v; }
+    __syncthreads();
+    if (warp == 0) {
+        const float s = warp_sum(lane < nwarps ? scratch[lane] : 0.0f), t = warp_sum(lane < nwarps ? scratch[33 + lane] : 0.0f);
+        if (lane == 0) { scratch[32] = s; scratch[65] = t; }
+    }
+    __syncthreads();
+    return make_float2(scratch[32], scratch[65]);
+}
+
+template <typename T>
+__global__ void pair_norm_kernel(PairNormArgs p) {
+    __shared__ float scratch[66];
+    pdl_start();
+    const int n = p.hidden;
+    const size_t row = (size_t)blockIdx.x * n;
+    const T* a = (const T*)p.a + row;
+    const T* b = (const T*)p.b + row;
+    T* out = p.out ? (T*)p.out + row : nullptr;
+    float ssa = 0.0f, ssb = 0.0f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const float u = to_f32<T>(a[i]), v = to_f32<T>(b[i]);
+        ssa += u * u;
+        ssb += v * v;
+    }
+    const float2 ss = block_sum2(ssa, ssb, scratch);
+    const float ra = 1.0f / sqrtf(ss.x / (float)n + p.eps_ab), rb = 1.0f / sqrtf(ss.y / (float)n + p.eps_ab);
+    auto joined = [&](int i) { return p.sa * ((to_f32<T>(a[i]) * ra) * p.wa[i]) + p.sb * ((to_f32<T>(b[i]) * rb) * p.wb[i]); };
+    if (!p.x) {
+        for (int i = threadIdx.x; i < n; i += blockDim.x) out[i] = from_f32<T>(joined(i));
+        return;
+    }
+    float* x = p.x + row;
+    float ssy = 0.0f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) { const float y = joined(i); ssy += y * y; }
+    ssy = block_sum(ssy, scratch);
+    const float ry = 1.0f / sqrtf(ssy / (float)n + p.eps);
+    float sx = 0.0f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const float v = x[i] + (joined(i) * ry) * p.gain[i];
+        x[i] = v;
+        sx += v * v;
+    }
+    if (!out) return;
+    sx = block_sum(sx, scratch);
+    const float rn = 1.0f / sqrtf(sx / (float)n + p.eps_next);
+    for (int i = threadIdx.x; i < n; i += blockDim.x) out[i] = from_f32<T>(x[i] * rn * p.next_gain[i]);      // its own writes
+}
+
+// The same for bfloat16 rows of a multiple of 8 elements that fit the CTA's registers (16-byte accesses).
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* q = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(q[e]); v[2 * e] = f.x; v[2 * e + 1] = f.y; }
+}
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    const float4 u = *reinterpret_cast<const float4*>(p), w = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w; v[4] = w.x; v[5] = w.y; v[6] = w.z; v[7] = w.w;
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
+    uint4 raw;
+    __nv_bfloat162* q = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) q[e] = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
+    *reinterpret_cast<uint4*>(p) = raw;
+}
+
+template <int NCH>
+__global__ void pair_norm_bf16x8_kernel(PairNormArgs p) {
+    __shared__ float scratch[66];
+    pdl_start();
+    const int n = p.hidden, nvec = n >> 3;
+    const size_t row = (size_t)blockIdx.x * n;
+    const __nv_bfloat16* a = (const __nv_bfloat16*)p.a + row;
+    const __nv_bfloat16* b = (const __nv_bfloat16*)p.b + row;
+    __nv_bfloat16* out = p.out ? (__nv_bfloat16*)p.out + row : nullptr;
+    float u[NCH][8], v[NCH][8];
+    float ssa = 0.0f, ssb = 0.0f;
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+        const int i = threadIdx.x + c * blockDim.x;
+        if (i < nvec) {
+            load8(a + (size_t)i * 8, u[c]);
+            load8(b + (size_t)i * 8, v[c]);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) { ssa += u[c][e] * u[c][e]; ssb += v[c][e] * v[c][e]; }
+        }
+    }
+    const float2 ss = block_sum2(ssa, ssb, scratch);
+    const float ra = 1.0f / sqrtf(ss.x / (float)n + p.eps_ab), rb = 1.0f / sqrtf(ss.y / (float)n + p.eps_ab);
+    float ssy = 0.0f;
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+        const int i = threadIdx.x + c * blockDim.x;
+        if (i < nvec) {
+            float wa[8], wb[8];
+            load8(p.wa + i * 8, wa);
+            load8(p.wb + i * 8, wb);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                u[c][e] = p.sa * ((u[c][e] * ra) * wa[e]) + p.sb * ((v[c][e] * rb) * wb[e]);
+                ssy += u[c][e] * u[c][e];
+            }
+            if (!p.x) store8(out + (size_t)i * 8, u[c]);
+        }
+    }
+    if (!p.x) return;
+    ssy = block_sum(ssy, scratch);
+    const float ry = 1.0f / sqrtf(ssy / (float)n + p.eps);
+    float* x = p.x + row;
+    float sx = 0.0f;
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+        const int i = threadIdx.x + c * blockDim.x;
+        if (i < nvec) {
+            float g[8], xs[8];
+            load8(p.gain + i * 8, g);
+            load8(x + (size_t)i * 8, xs);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                u[c][e] = xs[e] + (u[c][e] * ry) * g[e];
+                sx += u[c][e] * u[c][e];
+            }
+            *reinterpret_cast<float4*>(x + (size_t)i * 8) = make_float4(u[c][0], u[c][1], u[c][2], u[c][3]);
+            *reinterpret_cast<float4*>(x + (size_t)i * 8 + 4) = make_float4(u[c][4], u[c][5], u[c][6], u[c][7]);
+        }
+    }
+    if (!out) return;
+    sx = block_sum(sx, scratch);
+    const float rn = 1.0f / sqrtf(sx / (float)n + p.eps_next);
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+        const int i = threadIdx.x + c * blockDim.x;
+        if (i < nvec) {
+            float g[8];
+            load8(p.next_gain + i * 8, g);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) u[c][e] = u[c][e] * rn * g[e];
+            store8(out + (size_t)i * 8, u[c]);
+        }
+    }
+}
+
+VCB_EXPORT int vcb_pair_norm(const void* a, const void* b, const float* wa, const float* wb, float sa, float sb, float eps_ab,
+                             const float* gain, float* x, const float* next_gain, void* out, int n_tokens, int hidden, float eps,
+                             float eps_next, int dtype, void* stream) {
+    if (n_tokens <= 0) return 0;
+    if (hidden <= 0 || !a || !b || !wa || !wb || (x && !gain) || (!x && !out) || (x && out && !next_gain)) return VCB_ERR_BAD_ARG;
+    PairNormArgs p{a, b, wa, wb, sa, sb, eps_ab, gain, x, next_gain, out, hidden, eps, eps_next};
+    const int threads = hidden >= 4096 ? 512 : hidden >= 1024 ? 256 : 128;
+    cudaStream_t s = (cudaStream_t)stream;
+    const uintptr_t addrs = (uintptr_t)a | (uintptr_t)b | (uintptr_t)wa | (uintptr_t)wb | (uintptr_t)gain | (uintptr_t)x | (uintptr_t)next_gain | (uintptr_t)out;
+    if (dtype == VCB_BF16 && hidden % 8 == 0 && hidden / 8 <= 4 * 256 && !(addrs & 15)) {
+        const int nvec = hidden / 8;
+        const int vt = nvec >= 256 ? 256 : (nvec + 31) / 32 * 32;
+        const int nch = (nvec + vt - 1) / vt;
+        if (nch == 1) vcb_launch(pair_norm_bf16x8_kernel<1>, n_tokens, vt, 0, s, p);
+        else if (nch == 2) vcb_launch(pair_norm_bf16x8_kernel<2>, n_tokens, vt, 0, s, p);
+        else vcb_launch(pair_norm_bf16x8_kernel<4>, n_tokens, vt, 0, s, p);
+        return vcb_last_error();
+    }
+    if (dtype == VCB_F32) vcb_launch(pair_norm_kernel<float>, n_tokens, threads, 0, s, p);
+    else if (dtype == VCB_BF16) vcb_launch(pair_norm_kernel<__nv_bfloat16>, n_tokens, threads, 0, s, p);
+    else return VCB_ERR_BAD_ARG;
+    return vcb_last_error();
+}

@@ -1,0 +1,245 @@
+// A selective state space: per channel c a state of N numbers that decays and is driven by the token, with step sizes,
+// drive and read-out made from the token itself,
+//
+//   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,     y_c = sum_n S[c, n] C_n + D_c x_c,     out_c = y_c * silu(z_c)
+//
+// dt = softplus(dt_pre + dt_bias).  x, dt_pre, B, C and z are rows of the activations' type; step sizes, exponentials, state,
+// sums and the gate are float.  The state lives in the request's slot ([slots][I][N]), is read at the start of a request's
+// portion and left there at its end.
+//
+//   selective_step_kernel    single tokens: a thread per channel and NPT states
+//   selective_scan_kernel    portions: the same threads walk the request's tokens, whose step sizes, drives, B and C are made
+//                            once per chunk in shared memory while the values of the chunk after are on their way
+//
+// Exponentials are ex2.approx (2^-22 relative) of dt * A log2(e).  The reference has no recurrent mixer.
+#include "common.cuh"
+
+struct SelectiveArgs {
+    const void* x;              // [n, I] rows of T
+    const void* dt_pre;         // [n, I]
+    const void* b;              // [n, N]
+    const void* c;              // [n, N]
+    const void* z;              // [n, I]
+    long long ldx, lddt, ldb, ldc, ldz;
+    const float* dt_bias;       // [I]
+    const float* a2;            // [I, N]: A * log2(e), A < 0
+    const float* d;             // [I]
+    float* state;               // [slots][I][N]
+    void* out;                  // [n, I] of T
+    long long ldo;
+    const int* q_start;
+    const int* state_slots;
+    int I, N;
+};
+
+__device__ __forceinline__ float ss_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float ss_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float ss_silu(float z) { return z / (1.0f + expf(-z)); }
+
+// NPT consecutive floats of a row of N (those beyond N: zero); quads where the row allows.
+template <int NPT>
+__device__ __forceinline__ void ss_load(const float* p, int n0, int N, bool quads, float (&v)[NPT]) {
+    if (quads && n0 + NPT <= N) {
+#pragma unroll
+        for (int i = 0; i < NPT; i += 4) {
+            const float4 q = *reinterpret_cast<const float4*>(p + n0 + i);
+            v[i] = q.x; v[i + 1] = q.y; v[i + 2] = q.z; v[i + 3] = q.w;
+        }
+        return;
+    }
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) v[i] = n0 + i < N ? p[n0 + i] : 0.0f;
+}
+template <int NPT>
+__device__ __forceinline__ void ss_store(float* p, int n0, int N, bool quads, const float (&v)[NPT]) {
+    if (quads && n0 + NPT <= N) {
+#pragma unroll
+        for (int i = 0; i < NPT; i += 4) *reinterpret_cast<float4*>(p + n0 + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+        return;
+    }
+#pragma unroll
+    for (int i = 0; i < NPT; ++i)
+        if (n0 + i < N) p[n0 + i] = v[i];
+}
+
+// Grid (tiles of channels, requests); L lanes of a warp share a channel.
+template <typename T, int NPT>
+__global__ void __launch_bounds__(128) selective_step_kernel(SelectiveArgs a, int L) {
+    const int per = 128 / L, ch = blockIdx.x * per + threadIdx.x / L, part = threadIdx.x % L;
+    const bool there = ch < a.I;
+    const int c = there ? ch : a.I - 1, n0 = part * NPT;
+    const bool quads = (a.N & 3) == 0;
+    float A[NPT];
+    ss_load<NPT>(a.a2 + (size_t)c * a.N, n0, a.N, quads, A);
+    const float bias = a.dt_bias[c], dc = a.d[c];
+    const int r = blockIdx.y;
+    const size_t row = (size_t)a.q_start[r];                 // the step's index arrays are older than the kernel before
+    float* st = a.state + ((size_t)a.state_slots[r] * a.I + c) * a.N;
+    pdl_start();
+    float S[NPT];
+    ss_load<NPT>(st, n0, a.N, quads, S);
+    const float x = to_f32<T>(((const T*)a.x)[row * a.ldx + c]);
+    const float dt = ss_softplus(to_f32<T>(((const T*)a.dt_pre)[row * a.lddt + c]) + bias);
+    const float z = to_f32<T>(((const T*)a.z)[row * a.ldz + c]);
+    const T* bp = (const T*)a.b + row * a.ldb;
+    const T* cp = (const T*)a.c + row * a.ldc;
+    const float dx = dt * x;
+    float y = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) {
+        const bool in = n0 + i < a.N;
+        const float bn = in ? to_f32<T>(bp[n0 + i]) : 0.0f, cn = in ? to_f32<T>(cp[n0 + i]) : 0.0f;
+        S[i] = fmaf(ss_exp2(dt * A[i]), S[i], dx * bn);
+        y = fmaf(S[i], cn, y);
+    }
+    for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    if (!there) return;
+    ss_store<NPT>(st, n0, a.N, quads, S);
+    if (part == 0) ((T*)a.out)[row * a.ldo + c] = from_f32<T>(fmaf(dc, x, y) * ss_silu(z));
+}
+
+// Grid (tiles of CB channels, requests), CB * L threads.  TC tokens of a chunk; CB, L and TC are such that a thread stages
+// PER values of each kind: TC * CB = PER * threads for the channels' values.
+template <typename T, int NPT, int L, int CB, int TC>
+__global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a) {
+    constexpr int THREADS = CB * L, PER = (TC * CB + THREADS - 1) / THREADS, NP = L * NPT, PERN = (TC * NP + THREADS - 1) / THREADS;
+    __shared__ __align__(16) float dts[TC][CB], dxs[TC][CB], ys[TC][CB + 1];
+    __shared__ __align__(16) float bs[TC][NP], cs[TC][NP];
+    const int tid = threadIdx.x, part = tid % L, cl = tid / L, c0 = blockIdx.x * CB;
+    const int c = min(c0 + cl, a.I - 1), n0 = part * NPT;
+    const bool there = c0 + cl < a.I, quads = (a.N & 3) == 0;
+    float A[NPT], S[NPT];
+    ss_load<NPT>(a.a2 + (size_t)c * a.N, n0, a.N, quads, A);
+    const int sc = tid % CB, st0 = tid / CB;                 // staging: channel sc, tokens st0, st0 + L, ...
+    const int scc = min(c0 + sc, a.I - 1);
+    const float bias = a.dt_bias[scc], dc = a.d[scc];
+    pdl_start();
+    const int r = blockIdx.y;
+    const int row0 = a.q_start[r], len = a.q_start[r + 1] - row0;
+    if (len <= 0) return;
+    float* st = a.state + ((size_t)a.state_slots[r] * a.I + c) * a.N;
+    ss_load<NPT>(st, n0, a.N, quads, S);
+    const T* xp = (const T*)a.x + (size_t)row0 * a.ldx + scc;
+    const T* dp = (const T*)a.dt_pre + (size_t)row0 * a.lddt + scc;
+    const T* zp = (const T*)a.z + (size_t)row0 * a.ldz + scc;
+    const T* bp = (const T*)a.b + (size_t)row0 * a.ldb;
+    const T* cp = (const T*)a.c + (size_t)row0 * a.ldc;
+    T* op = (T*)a.out + (size_t)row0 * a.ldo + scc;
+    float px[PER], pd[PER], pz[PER], pb[PERN], pc[PERN];     // the values of a chunk on their way
+    auto fetch = [&](int t0) {
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            const int t = st0 + k * L, tt = min(t0 + t, len - 1);
+            px[k] = to_f32<T>(xp[(size_t)tt * a.ldx]);
+            pd[k] = to_f32<T>(dp[(size_t)tt * a.lddt]);
+            pz[k] = to_f32<T>(zp[(size_t)tt * a.ldz]);
+        }
+#pragma unroll
+        for (int k = 0; k < PERN; ++k) {
+            const int idx = tid + k * THREADS, t = idx / NP, n = idx - t * NP, tt = min(t0 + t, len - 1);
+            const bool in = n < a.N && t < TC;
+            pb[k] = in ? to_f32<T>(bp[(size_t)tt * a.ldb + n]) : 0.0f;
+            pc[k] = in ? to_f32<T>(cp[(size_t)tt * a.ldc + n]) : 0.0f;
+        }
+    };
+    fetch(0);
+    for (int t0 = 0; t0 < len; t0 += TC) {
+        const int tc = min(TC, len - t0);
+        float zk[PER], xk[PER];
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            const int t = st0 + k * L;
+            if (t < TC) {
+                const float dt = ss_softplus(pd[k] + bias);
+                dts[t][sc] = dt;
+                dxs[t][sc] = dt * px[k];
+            }
+            zk[k] = pz[k];
+            xk[k] = px[k];
+        }
+#pragma unroll
+        for (int k = 0; k < PERN; ++k) {
+            const int idx = tid + k * THREADS, t = idx / NP, n = idx - t * NP;
+            if (t < TC) { bs[t][n] = pb[k]; cs[t][n] = pc[k]; }
+        }
+        __syncthreads();
+        if (t0 + TC < len) fetch(t0 + TC);
+#pragma unroll 4
+        for (int t = 0; t < tc; ++t) {
+            const float dt = dts[t][cl], dx = dxs[t][cl];
+            float y = 0.0f;
+#pragma unroll
+            for (int i = 0; i < NPT; i += 4) {
+                const float4 b4 = *reinterpret_cast<const float4*>(&bs[t][n0 + i]), c4 = *reinterpret_cast<const float4*>(&cs[t][n0 + i]);
+                S[i] = fmaf(ss_exp2(dt * A[i]), S[i], dx * b4.x);
+                S[i + 1] = fmaf(ss_exp2(dt * A[i + 1]), S[i + 1], dx * b4.y);
+                S[i + 2] = fmaf(ss_exp2(dt * A[i + 2]), S[i + 2], dx * b4.z);
+                S[i + 3] = fmaf(ss_exp2(dt * A[i + 3]), S[i + 3], dx * b4.w);
+                y = fmaf(S[i], c4.x, y);
+                y = fmaf(S[i + 1], c4.y, y);
+                y = fmaf(S[i + 2], c4.z, y);
+                y = fmaf(S[i + 3], c4.w, y);
+            }
+#pragma unroll
+            for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+            if (part == 0) ys[t][cl] = y;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            const int t = st0 + k * L;
+            if (t < tc && c0 + sc < a.I) op[(size_t)(t0 + t) * a.ldo] = from_f32<T>(fmaf(dc, xk[k], ys[t][sc]) * ss_silu(zk[k]));
+        }
+        // ys is written again only after the next chunk's first barrier
+    }
+    if (there) ss_store<NPT>(st, n0, a.N, quads, S);
+}
+
+template <typename T, int NPT, int L, int CB>
+static void launch_scan(const SelectiveArgs& a, int n_reqs, cudaStream_t s) {
+    vcb_launch(selective_scan_kernel<T, NPT, L, CB, (NPT > 4 ? 4 : 16)>, dim3((a.I + CB - 1) / CB, n_reqs), CB * L, 0, s, a);
+}
+
+template <typename T>
+static int launch_selective(const SelectiveArgs& a, int n_reqs, int max_q_len, cudaStream_t s) {
+    const int npt = a.N <= 128 ? 4 : 16;
+    int L = 1;
+    while (L * npt < a.N) L <<= 1;
+    if (L > 32) return VCB_ERR_UNSUPPORTED;
+    if (max_q_len == 1) {
+        dim3 grid((a.I + 128 / L - 1) / (128 / L), n_reqs);
+        if (npt == 4) vcb_launch(selective_step_kernel<T, 4>, grid, 128, 0, s, a, L);
+        else vcb_launch(selective_step_kernel<T, 16>, grid, 128, 0, s, a, L);
+        return vcb_last_error();
+    }
+    if (npt == 16) {
+        if (L == 16) launch_scan<T, 16, 16, 8>(a, n_reqs, s);
+        else launch_scan<T, 16, 32, 8>(a, n_reqs, s);
+        return vcb_last_error();
+    }
+    switch (L) {
+        case 1: launch_scan<T, 4, 1, 32>(a, n_reqs, s); break;
+        case 2: launch_scan<T, 4, 2, 32>(a, n_reqs, s); break;
+        case 4: launch_scan<T, 4, 4, 32>(a, n_reqs, s); break;
+        case 8: launch_scan<T, 4, 8, 16>(a, n_reqs, s); break;
+        case 16: launch_scan<T, 4, 16, 8>(a, n_reqs, s); break;
+        default: launch_scan<T, 4, 32, 8>(a, n_reqs, s); break;
+    }
+    return vcb_last_error();
+}
+
+VCB_EXPORT int vcb_selective_scan(const void* x, long long ldx, const void* dt_pre, long long lddt, const void* b, long long ldb,
+                                  const void* c, long long ldc, const void* z, long long ldz, const float* dt_bias, const float* a2,
+                                  const float* d, float* state, void* out, long long ldo, const int* q_start, const int* state_slots,
+                                  int n_reqs, int max_q_len, int I, int N, int dtype, void* stream) {
+    if (n_reqs <= 0 || max_q_len <= 0) return 0;
+    if (!x || !dt_pre || !b || !c || !z || !dt_bias || !a2 || !d || !state || !out || I <= 0 || N <= 0 || n_reqs > 65535) return VCB_ERR_BAD_ARG;
+    SelectiveArgs a{x, dt_pre, b, c, z, ldx, lddt, ldb, ldc, ldz, dt_bias, a2, d, state, out, ldo, q_start, state_slots, I, N};
+    if (dtype == VCB_F32) return launch_selective<float>(a, n_reqs, max_q_len, (cudaStream_t)stream);
+    if (dtype == VCB_BF16) return launch_selective<__nv_bfloat16>(a, n_reqs, max_q_len, (cudaStream_t)stream);
+    return VCB_ERR_BAD_ARG;
+}

@@ -108,10 +108,13 @@ def plan_for_model(cfg: EngineConfig, model, total: int, in_place: int, max_mode
     workspace = model.workspace_bytes(cfg.max_num_batched_tokens, cfg.max_num_seqs, cfg.max_num_seqs)
     state = sum(int(torch.empty((), dtype=s.dtype).element_size()) * int(torch.Size(s.shape).numel())
                 for s in simple if isinstance(s, StateSpec))
+    summary_pages = CacheManager.fixed_bytes(specs, cfg.block_size, cfg.max_num_seqs, model.dtype)
     heads = [(getattr(p, "nh", 0), getattr(p, "d", 0)) for blk in model.blocks for p in blk.parts.values()]
     slices = step_slices(cfg, model.hidden, model.vocab, el, workspace, len({s for s in simple if hasattr(s, "num_kv_heads")}),
                          max((h for h, _ in heads), default=0), max((d for _, d in heads), default=0), sm_count, state,
                          launches_per_step=8 * len(model.spec.run_order) + 4)
+    if summary_pages:
+        slices.append(("pages of block summaries kept ready", _round(summary_pages)))
     weights = sum(t.numel() * t.element_size() for t in model.tensors())
     images = sum(t.numel() * t.element_size() for t in model.tile_images())
     return plan(cfg, total, in_place, slices, CacheManager.bytes_per_page(specs, cfg.block_size, model.dtype), max_model_len,

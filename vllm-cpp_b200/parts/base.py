@@ -54,11 +54,17 @@ class PagedKVSpec:
     """Keys and values in pages.  ``window`` 0: all keys are kept; > 0: only the
     last ``window`` keys are read, pages left of the window are given back.
     ``planes`` 2: a page holds the keys and then the values of its slots; 1: one row per slot
-    that the mixer reads as key and as value (a cached latent row, ``head_dim`` its width)."""
+    that the mixer reads as key and as value (a cached latent row, ``head_dim`` its width).
+    ``stride`` > 1: a row for every ``stride`` tokens instead of one per token, written once the last of them is there (a
+    summary of a block of tokens): a request of n tokens holds n // stride rows.  ``keep_block`` > 1 (with a window): the
+    tokens of the block of ``keep_block`` tokens that is not complete yet are kept although the window may have passed
+    them, because the block's summary is made of them."""
     num_kv_heads: int
     head_dim: int
     window: int = 0
     planes: int = 2
+    stride: int = 1
+    keep_block: int = 1
 
 
 @dataclass(frozen=True)

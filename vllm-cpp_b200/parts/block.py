@@ -149,7 +149,8 @@ class SandwichNormBlock(Block):
     before the next sublayer are one kernel (ops.norm_residual_norm): the one after the mixer prepares the
     feed-forward's input, the one after the feed-forward the next layer's, when that layer is of this arrangement
     too (NormedInput).  The residual stream is float32 throughout.  A layer whose feed-forward is "none" has only
-    the first line."""
+    the first line.  A mixer that offers its result as two that are normed and joined (``pair_result``, parts/parallel.py)
+    has the join in the same kernel (ops.pair_norm)."""
 
     SLOTS = {"mixer": "mixer", "feed_forward": "feed_forward",
              "mixer_norm": "norm", "mixer_post_norm": "norm", "mixer_scale": "scale",
@@ -170,8 +171,12 @@ class SandwichNormBlock(Block):
     def accepts_normed(self, n_tokens):
         return self.mixer_norm.folded(None)
 
+    def _pair(self):
+        offer = getattr(self.mixer, "pair_result", None)
+        return offer() if offer else None
+
     def workspace_bytes(self, n_tokens, n_reqs, hidden, dtype):
-        return 2 * workspace_piece((n_tokens, hidden), dtype) + super().workspace_bytes(n_tokens, n_reqs, hidden, dtype)
+        return (3 if self._pair() else 2) * workspace_piece((n_tokens, hidden), dtype) + super().workspace_bytes(n_tokens, n_reqs, hidden, dtype)
 
     def forward(self, residual, delta, pending, step, cache, writes_cache, ws, next_block=None, carry=None):
         if isinstance(pending, ops.RowScale):
@@ -185,19 +190,32 @@ class SandwichNormBlock(Block):
         else:
             h = ws.take((n, hidden), delta.dtype)
             self.mixer_norm.forward(residual, delta if pending else None, h)
-        self.mixer.forward(h, y, step, cache, writes_cache, ws)
-        after = next_block.accepts_normed(n) if next_block is not None else None
-        if self.has_ff:
-            ops.norm_residual_norm(y, post_mixer[0], residual, post_mixer[1], next_gain=pre_ff[0], next_out=h, next_eps=pre_ff[1])
-            self.feed_forward.forward(h, y, step, ws)
-            last = post_ff
+        pair = self._pair()
+        if pair is None:
+            self.mixer.forward(h, y, step, cache, writes_cache, ws)
         else:
-            last = post_mixer
+            y2 = ws.take((n, hidden), delta.dtype)
+            self.mixer.forward_pair(h, y, y2, step, cache, writes_cache, ws)
+        after = next_block.accepts_normed(n) if next_block is not None else None
+
+        def join_mixer(next_gain=None, next_out=None, next_eps=0.0):
+            if pair is None:
+                ops.norm_residual_norm(y, post_mixer[0], residual, post_mixer[1], next_gain=next_gain, next_out=next_out, next_eps=next_eps)
+            else:
+                ops.pair_norm(y, y2, *pair, next_out, x=residual, gain=post_mixer[0], eps=post_mixer[1], next_gain=next_gain, next_eps=next_eps)
+
+        join_last = join_mixer
+        if self.has_ff:
+            join_mixer(pre_ff[0], h, pre_ff[1])
+            self.feed_forward.forward(h, y, step, ws)
+
+            def join_last(next_gain=None, next_out=None, next_eps=0.0):
+                ops.norm_residual_norm(y, post_ff[0], residual, post_ff[1], next_gain=next_gain, next_out=next_out, next_eps=next_eps)
         if after is None:
-            ops.norm_residual_norm(y, last[0], residual, last[1])
+            join_last()
             ws.release(mark)
             return False
-        ops.norm_residual_norm(y, last[0], residual, last[1], next_gain=after[0], next_out=delta, next_eps=after[1])
+        join_last(after[0], delta, after[1])
         ws.release(mark)
         return NormedInput()
 

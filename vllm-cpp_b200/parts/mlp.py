@@ -4,7 +4,7 @@
 gate and up are one product against the row-wise concatenation [W_gate; W_up],
 made at load; the reference runs them as two.
 
-``activation`` "clamped_swish" is another rule for the pair: g = min(gate, limit),
+``activation`` "relu" is max(gate, 0) instead of silu.  "clamped_swish" is another rule for the pair: g = min(gate, limit),
 u = clamp(up, -limit, limit), act = g * sigmoid(alpha * g) * (u + 1); ``biases`` gives
 all three projections a bias (tensors named as the matrices plus ``bias_suffix``),
 added in float before the clamps and after the down product.
@@ -29,7 +29,7 @@ class NoFeedForward(FeedForward):
 
 @register_feed_forward("gated_mlp")
 class GatedMLP(FeedForward):
-    ACTIVATIONS = ("silu", "clamped_swish")
+    ACTIVATIONS = ("silu", "relu", "clamped_swish")
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str, dtype, device,
                  tensor_names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), limit: float = 0.0,
@@ -38,7 +38,7 @@ class GatedMLP(FeedForward):
             raise ValueError(f"gated_mlp: activation {activation!r} is not built (known: {self.ACTIVATIONS})")
         if activation == "clamped_swish" and not limit > 0:
             raise ValueError("gated_mlp: the clamped activation needs a positive limit")
-        if biases and activation == "silu":
+        if biases and activation != "clamped_swish":
             raise ValueError("gated_mlp: biases are built for the clamped activation only")
         self.hidden, self.inter = hidden_size, intermediate_size
         self.names = tuple(tensor_names)          # local names of the gate, up and down matrices
@@ -70,10 +70,10 @@ class GatedMLP(FeedForward):
             self.b_down = tensors[down + sfx].contiguous()
 
     def product_weights(self):
-        return [(self.w_gate_up, self.inter if self.activation == "silu" else 0), (self.w_down, 0)]
+        return [(self.w_gate_up, self.inter if self.activation != "clamped_swish" else 0), (self.w_down, 0)]
 
     def fuses_norm(self, n_tokens):
-        if self.activation != "silu":
+        if self.activation == "clamped_swish":
             return False
         return ops.linear_fuses_norm(n_tokens, self.w_gate_up) and ops.linear_fuses_norm(n_tokens, self.w_down)
 
@@ -95,10 +95,10 @@ class GatedMLP(FeedForward):
             ws.release(mark)
             return
         if ops.linear_gated_fuses(n, self.w_gate_up):
-            ops.linear_gated(x, self.w_gate_up, act, x_scale=x_scale)       # product and activation in one kernel
+            ops.linear_gated(x, self.w_gate_up, act, x_scale=x_scale, gate_act=self.activation)       # product and activation in one kernel
         else:
             gate_up = ws.take((n, 2 * self.inter), self.dtype)
             ops.linear(x, self.w_gate_up, gate_up, x_scale=x_scale)
-            ops.silu_mul(gate_up, act)
+            (ops.relu_mul if self.activation == "relu" else ops.silu_mul)(gate_up, act)
         ops.linear(act, self.w_down, out, fuse=fuse)
         ws.release(mark)
