@@ -100,6 +100,35 @@ def random_weights(cfg, seed, sharp=1.0, rank=12):
 
 
 # ------------------------------------------------------------- mechanisms
+_rounding = None        # inside ``rounded_like_bf16``: the generator of the perturbations
+
+
+class rounded_like_bf16:
+    """Inside this context every product's input and result carries a random relative error of up to half a bfloat16 unit: what
+    any computation with bfloat16 activations may differ by.  Where a design divides by a root mean square that is nearly zero
+    (a head whose first token has r . k near zero takes its sign from it), that is much more than elsewhere."""
+
+    def __init__(self, seed):
+        self.rng = np.random.default_rng(seed)
+
+    def __enter__(self):
+        global _rounding
+        _rounding = self.rng
+
+    def __exit__(self, *exc):
+        global _rounding
+        _rounding = None
+
+
+def perturbed(x):
+    return x if _rounding is None else x * (1.0 + _rounding.uniform(-1, 1, size=x.shape) * 2.0 ** -9)
+
+
+def product(h, w):
+    """W h for rows h."""
+    return perturbed(perturbed(h) @ w.T)
+
+
 def softplus(z):
     return np.where(z > 30, z, np.log1p(np.exp(np.minimum(z, 30))))
 
@@ -161,14 +190,14 @@ def windowed_attention(h, w, p, m, eps):
     """The left mixer of one request, whole."""
     n = h.shape[0]
     H, G, d, dv = m["heads"], kv_heads(m), m["dim"], m["vdim"]
-    q, k, v = (short_conv(h @ w[p + t].T + w[p + t + ".b"], w[p + t + ".conv"]) for t in ("q", "k", "v"))
+    q, k, v = (perturbed(short_conv(product(h, w[p + t]) + w[p + t + ".b"], w[p + t + ".conv"])) for t in ("q", "k", "v"))
     q, k, v = q.reshape(n, H, d), k.reshape(n, G, d), v.reshape(n, G, dv)
     if m.get("rot"):
         pos = np.arange(n, dtype=np.float64)
         q, k = (rotate_pairs(x, pos, m["rot"]["base"], m["rot"]["dims"]) for x in (q, k))
     mask = m.get("mask") or {}
     o = pooled_attention_core(q, k, v, m["scale"], w[p + "temp"], mask.get("size"), mask.get("pool"))
-    return o.reshape(n, H * dv) @ w[p + "o"].T
+    return product(o.reshape(n, H * dv), w[p + "o"])
 
 
 def selective_scan_core(x, dt, A, B, C, D, S=None):
@@ -184,13 +213,13 @@ def selective_scan_core(x, dt, A, B, C, D, S=None):
 def selective_state(h, w, p, m, eps):
     """The right mixer of one request, whole."""
     I, R, N = m["inner"], m["dt_rank"], m["state"]
-    xz = h @ w[p + "in"].T
+    xz = product(h, w[p + "in"])
     x, z = xz[:, :I], xz[:, I:]
     x = silu(short_conv(x, w[p + "conv"], w[p + "conv.b"]))
-    low = x @ w[p + "x"].T
-    dt = softplus(low[:, :R] @ w[p + "dt"].T + w[p + "dt.b"])
+    low = product(x, w[p + "x"])
+    dt = softplus(product(low[:, :R], w[p + "dt"]) + w[p + "dt.b"])
     y, _ = selective_scan_core(x, dt, -np.exp(w[p + "A_log"]), low[:, R:R + N], low[:, R + N:], w[p + "D"])
-    return (y * silu(z)) @ w[p + "o"].T
+    return product(y * silu(z), w[p + "o"])
 
 
 def parallel(h, w, p, m, eps):
@@ -215,16 +244,16 @@ def general_delta_core(r, k, v, decay, removal, S=None):
 
 def general_delta(h, w, p, m, eps):
     n, H, d = h.shape[0], m["heads"], m["dim"]
-    r, k, v = ((h @ w[p + t].T).reshape(n, H, d) for t in ("r", "k", "v"))
-    decay = np.exp(-DECAY_RATE * sigmoid(np.tanh(h @ w[p + "w1"].T) @ w[p + "w2"].T + w[p + "w0"]))
-    removal = sigmoid(h @ w[p + "a"].T + w[p + "a.b"])
+    r, k, v = (product(h, w[p + t]).reshape(n, H, d) for t in ("r", "k", "v"))
+    decay = np.exp(-DECAY_RATE * sigmoid(product(np.tanh(product(h, w[p + "w1"])), w[p + "w2"]) + w[p + "w0"]))
+    removal = sigmoid(product(h, w[p + "a"]) + w[p + "a.b"])
     o, _ = general_delta_core(r, k, v, decay.reshape(n, H, d), removal.reshape(n, H, d))
-    o = rms(o, eps).reshape(n, H * d) * w[p + "norm"] * sigmoid(h @ w[p + "g"].T)
-    return o @ w[p + "o"].T
+    o = rms(o, eps).reshape(n, H * d) * w[p + "norm"] * sigmoid(product(h, w[p + "g"]))
+    return product(o, w[p + "o"])
 
 
 def feed_forward(h, w, p):
-    return (np.maximum(h @ w[p + "gate"].T, 0.0) * (h @ w[p + "up"].T)) @ w[p + "down"].T
+    return product(np.maximum(product(h, w[p + "gate"]), 0.0) * product(h, w[p + "up"]), w[p + "down"])
 
 
 MIXERS = {"general_delta": general_delta, "parallel": parallel}
@@ -242,8 +271,18 @@ def forward(cfg, w, ids, return_layers=False):
         if layer.get("mlp") is not None:
             x = x + normed(feed_forward(normed(x, w[p + "norm2"], eps), w, p + "mlp."), w[p + "norm2b"], eps)
         after.append(x.copy())
-    logits = normed(x, w["final.norm"], eps) @ w["head"].T
+    logits = product(normed(x, w["final.norm"], eps), w["head"])
     return (logits, np.stack(after)) if return_layers else logits
+
+
+def rounding_error(cfg, w, ids, runs=4):
+    """Per row of the logits, the largest error over all tokens that perturbations of bfloat16's size caused in ``runs`` tries."""
+    want = forward(cfg, w, ids)
+    worst = np.zeros(len(want))
+    for seed in range(runs):
+        with rounded_like_bf16(seed):
+            worst = np.maximum(worst, np.abs(forward(cfg, w, ids) - want).max(axis=1))
+    return worst
 
 
 def greedy(logits):
