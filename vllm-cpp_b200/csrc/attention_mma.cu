@@ -70,6 +70,12 @@ struct MmaAttnArgs {
     // Nonzero: the softmax weights enter the P V product as two bfloat16 terms, p = hi + lo with hi the rounding of p and lo
     // that of the rest (16 bits of mantissa instead of 8), for designs that want their attention weights in 32-bit.
     int precise_weights;
+    // Rows for blocks of `pool` tokens beside the window's tokens (the POOLED forms of both kernels; window > 0): pages of the
+    // same layout in which row b of a request is the mean key and value of its tokens b pool .. b pool + pool - 1.  A query at
+    // position i sees the rows b with (b + 1) pool - 1 <= i - window.
+    const __nv_bfloat16* pooled;
+    const int* pool_table;         // [n_reqs, pt_stride]
+    int pt_stride, pool_pages, pool;
 };
 
 // 1 / (l + e^(sink - m)) * sigmoid(gate): what an output row is multiplied by.  m2: the reference of l in units of log2.
@@ -286,7 +292,7 @@ __device__ __forceinline__ void load_q_frags(uint32_t (&qf)[D / 16][4], uint32_t
 }
 
 // ------------------------------------------------------------------ decode
-template <int D, int STAGES>
+template <int D, int STAGES, bool POOLED>
 __global__ void __launch_bounds__(BLOCK_THREADS, 2)
 attention_decode_kernel(MmaAttnArgs a) {
     extern __shared__ __align__(1024) unsigned char smem[];
@@ -314,7 +320,10 @@ attention_decode_kernel(MmaAttnArgs a) {
     // more CTAs than one with a short context and the CTAs of a step with mixed contexts end together;
     // the CTAs beyond a request's splits leave at once.
     // (A number that would need more splits than the grid has falls back to equal parts.)
-    const int tile0 = lo / BN, tile1 = (hi + BN - 1) / BN;
+    // POOLED: the tiles of block rows come before the tiles of tokens, as tiles tile0 .. tok0 - 1 of the same run.  (A block that
+    // this step completes ends at pos, inside the window: every visible row was written by an earlier step.)
+    const int blocks = POOLED ? lo / a.pool : 0;
+    const int tok0 = lo / BN, tile0 = tok0 - (blocks + BN - 1) / BN, tile1 = (hi + BN - 1) / BN;
     const int grid_splits = gridDim.x;
     int per = (tile1 - tile0 + grid_splits - 1) / grid_splits, nsplit = grid_splits;
     if (a.split_tiles) {
@@ -362,22 +371,29 @@ attention_decode_kernel(MmaAttnArgs a) {
         if (producer) {
             PageWindow pw;
             const PageDiv pd(a.page);
-            pw.init(bt, pd.div(my0 * BN), hi, a.page, lane, a.num_pages);
+            bool bad = false;
+            if (POOLED && my0 < tok0) pw.init(a.pool_table + (size_t)r * a.pt_stride, pd.div((my0 - tile0) * BN), blocks, a.page, lane, a.pool_pages);
+            else pw.init(bt, pd.div(my0 * BN), hi, a.page, lane, a.num_pages);
             const int cache_heads = a.nkv / a.kv_share;
             const size_t page_stride = (size_t)a.planes * cache_heads * a.page * D, head_base = (size_t)(g / a.kv_share) * a.page * D,
                          v_off = (size_t)(a.planes - 1) * cache_heads * a.page * D;
             for (int tile = my0; tile < my1; ++tile, ++it) {
                 const int st = it % STAGES;
-                if (!waited && (tile + 1) * BN > pos) { pdl_wait(); waited = true; }   // the tile with this step's row
+                const bool of_blocks = POOLED && tile < tok0;
+                if (POOLED && tile == tok0 && my0 < tok0) {          // from the block rows to the tokens
+                    bad = pw.bad;
+                    pw.init(bt, pd.div(tile * BN), hi, a.page, lane, a.num_pages);
+                }
+                if (!waited && !of_blocks && (tile + 1) * BN > pos) { pdl_wait(); waited = true; }   // the tile with this step's row
                 if (!cx_mbar_wait(empty0 + 8 * st, ((it / STAGES) & 1) ^ 1)) gave_up = true;
                 // one plane of rows that are key and value at once: the tile is fetched once and read as both
                 if (lane == 0) cx_mbar_expect_tx(full0 + 8 * st, a.planes == 1 ? TILE_BYTES : 2 * TILE_BYTES);
                 __syncwarp();
                 produce_tile<D, BN>(s_tiles + st * 2 * TILE_BYTES, s_tiles + st * 2 * TILE_BYTES + TILE_BYTES,
-                                    full0 + 8 * st, tile * BN, lo, hi, pw, a.cache, head_base, page_stride, v_off, pd, lane,
-                                    0, a.planes == 1 ? 1 : 0);
+                                    full0 + 8 * st, (of_blocks ? tile - tile0 : tile) * BN, of_blocks ? 0 : lo, of_blocks ? blocks : hi, pw,
+                                    of_blocks ? a.pooled : a.cache, head_base, page_stride, v_off, pd, lane, 0, a.planes == 1 ? 1 : 0);
             }
-            if (pw.bad && a.status) atomicCAS(a.status, 0, VCB_STATUS_BAD_PAGE);
+            if ((pw.bad || bad) && a.status) atomicCAS(a.status, 0, VCB_STATUS_BAD_PAGE);
         } else {
             uint32_t qf[D / 16][4];
             load_q_frags<D>(qf, sq, 0);
@@ -385,7 +401,9 @@ attention_decode_kernel(MmaAttnArgs a) {
                 const int st = it % STAGES;
                 if (!cx_mbar_wait(full0 + 8 * st, (it / STAGES) & 1)) gave_up = true;
                 const uint32_t sk = s_tiles + st * 2 * TILE_BYTES, sv = a.planes == 1 ? sk : sk + TILE_BYTES;
-                const int kb = tile * BN + warp * 16;    // this warp's 16 keys
+                const bool of_blocks = POOLED && tile < tok0;
+                const int kt = (of_blocks ? tile - tile0 : tile) * BN, klo = of_blocks ? 0 : lo, khi = of_blocks ? blocks : hi;
+                const int kb = kt + warp * 16;           // this warp's 16 keys
                 float s[2][4];
 #pragma unroll
                 for (int i = 0; i < 2; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f; }
@@ -406,13 +424,13 @@ attention_decode_kernel(MmaAttnArgs a) {
                         }
                 }
                 // only a tile that crosses lo or hi has keys to mask (the same for the whole CTA)
-                if (tile * BN < lo || tile * BN + BN > hi) {
+                if (kt < klo || kt + BN > khi) {
 #pragma unroll
                     for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
                         for (int e = 0; e < 4; ++e) {
                             const int j = kb + nb * 8 + (lane & 3) * 2 + (e & 1);
-                            if (j < lo || j >= hi) s[nb][e] = -INFINITY;
+                            if (j < klo || j >= khi) s[nb][e] = -INFINITY;
                         }
                 }
                 // raw scores from here on; 2^(s * sl2 - m * sl2) is one multiply-add and one ex2.
@@ -552,15 +570,20 @@ attention_decode_kernel(MmaAttnArgs a) {
 }
 
 // ---------------------------------------------------------------- launchers
-template <int D>
-static int launch_decode(const MmaAttnArgs& a, int n_list, int nsplit, cudaStream_t s) {
+template <int D, bool POOLED>
+static int launch_decode_as(const MmaAttnArgs& a, int n_list, int nsplit, cudaStream_t s) {
     constexpr int STAGES = 3;
     const size_t smem = (size_t)STAGES * 2 * BN * D * 2 + 16 * D * 2 + 2 * STAGES * 8 + 64;   // tiles, Q, barriers
     static unsigned long long configured = 0;
-    if (int e = vcb_allow_dynamic_smem(attention_decode_kernel<D, STAGES>, (int)smem, &configured)) return e;
+    if (int e = vcb_allow_dynamic_smem(attention_decode_kernel<D, STAGES, POOLED>, (int)smem, &configured)) return e;
     dim3 grid(nsplit, a.nkv, n_list);
-    vcb_launch(attention_decode_kernel<D, STAGES>, grid, BLOCK_THREADS, smem, s, a);
+    vcb_launch(attention_decode_kernel<D, STAGES, POOLED>, grid, BLOCK_THREADS, smem, s, a);
     return vcb_last_error();
+}
+
+template <int D>
+static int launch_decode(const MmaAttnArgs& a, int n_list, int nsplit, cudaStream_t s) {
+    return a.pooled ? launch_decode_as<D, true>(a, n_list, nsplit, s) : launch_decode_as<D, false>(a, n_list, nsplit, s);
 }
 
 // ------------------------------------------------- prefill on tcgen05
@@ -690,7 +713,7 @@ __host__ __device__ constexpr uint32_t idesc(int n, bool b_mn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn ? (1u << 16) : 0u) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
 }
 
-template <int D, bool PRECISE>
+template <int D, bool PRECISE, bool POOLED>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_prefill_tc_kernel(MmaAttnArgs a) {
     // PRECISE (a template parameter of this kernel): the weights' rest after their rounding to bfloat16 goes into the second
@@ -755,7 +778,9 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
     const int last_row = min(row0 + BMT, rows_total) - 1;
     const int hi = ctx + last_row / G + 1;
     const int lo = a.window > 0 ? max(0, ctx + row0 / G + 1 - a.window) : 0;
-    const int tile0 = lo / TKT, tile1 = (hi + TKT - 1) / TKT;
+    // POOLED: tiles of block rows first (tiles tile0 .. tok0 - 1 of the run), as many rows as the last row of the tile sees
+    const int blocks = POOLED ? max(0, hi - a.window) / a.pool : 0;
+    const int tok0 = lo / TKT, tile0 = tok0 - (blocks + TKT - 1) / TKT, tile1 = (hi + TKT - 1) / TKT;
     const int n_tiles = *abort_flag ? 0 : tile1 - tile0;
 
     auto give_up = [&](int code) {
@@ -769,11 +794,21 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
         // tile j - 2 is.
         PageWindow pw;
         const PageDiv pd(a.page);
-        pw.init(bt, pd.div(tile0 * TKT), hi, a.page, lane, a.num_pages);
+        bool bad = false;
+        if (POOLED && tile0 < tok0) pw.init(a.pool_table + (size_t)r * a.pt_stride, 0, blocks, a.page, lane, a.pool_pages);
+        else pw.init(bt, pd.div(tile0 * TKT), hi, a.page, lane, a.num_pages);
         const size_t page_stride = (size_t)a.planes * a.nkv * a.page * D, head_base = (size_t)g * a.page * D,
                      v_off = (size_t)(a.planes - 1) * a.nkv * a.page * D;
         // a tile's addresses are worked out before its stage is waited for
-        TilePiece pc = tile_piece<D, TKT>(tile0 * TKT, lo, hi, pw, a.cache, head_base, page_stride, pd, lane);
+        auto piece_of = [&](int tile) {
+            if (POOLED && tile < tok0) return tile_piece<D, TKT>((tile - tile0) * TKT, 0, blocks, pw, a.pooled, head_base, page_stride, pd, lane);
+            if (POOLED && tile == tok0 && tile0 < tok0) {           // from the block rows to the tokens
+                bad = pw.bad;
+                pw.init(bt, pd.div(tile * TKT), hi, a.page, lane, a.num_pages);
+            }
+            return tile_piece<D, TKT>(tile * TKT, lo, hi, pw, a.cache, head_base, page_stride, pd, lane);
+        };
+        TilePiece pc = piece_of(tile0);
         if (warp == 0) {
             int ks = 0, kphase = 1;             // K stage of tile j and the parity its empty barrier is waited with
             for (int j = 0; j < n_tiles && !*abort_flag; ++j) {
@@ -782,7 +817,7 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
                 __syncwarp();
                 issue_piece(pc, sk0 + ks * KV_BYTES, 0, B(FULL_K + ks), v_off, lane, 0, 1);
                 if (++ks == K_STAGES) { ks = 0; kphase ^= 1; }
-                if (j + 1 < n_tiles) pc = tile_piece<D, TKT>((tile0 + j + 1) * TKT, lo, hi, pw, a.cache, head_base, page_stride, pd, lane);
+                if (j + 1 < n_tiles) pc = piece_of(tile0 + j + 1);
             }
         } else {
             int vs = 0, vphase = 1;
@@ -792,10 +827,10 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
                 __syncwarp();
                 issue_piece(pc, 0, sv0 + vs * KV_BYTES, 0, v_off, lane, B(FULL_V + vs), 2);
                 if (++vs == V_STAGES) { vs = 0; vphase ^= 1; }
-                if (j + 1 < n_tiles) pc = tile_piece<D, TKT>((tile0 + j + 1) * TKT, lo, hi, pw, a.cache, head_base, page_stride, pd, lane);
+                if (j + 1 < n_tiles) pc = piece_of(tile0 + j + 1);
             }
         }
-        if (pw.bad && a.status) atomicCAS(a.status, 0, VCB_STATUS_BAD_PAGE);
+        if ((pw.bad || bad) && a.status) atomicCAS(a.status, 0, VCB_STATUS_BAD_PAGE);
     } else if (warp == 2) {
         // ---- MMA issuer.  The whole warp walks the loop and waits, one elected lane issues: addresses and
         // descriptors are then the same in all lanes, which lets the compiler keep them in uniform
@@ -895,13 +930,15 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
         bool ok = true;
         for (int j = 0; j < n_tiles && !*abort_flag; ++j) {
             const int st = j & 1;
-            const int kb = (tile0 + j) * TKT;
+            const bool of_blocks = POOLED && tile0 + j < tok0;
+            const int kb = of_blocks ? j * TKT : (tile0 + j) * TKT;
             if (!cx_mbar_wait(B(S_FULL + st), (j >> 1) & 1)) { ok = false; break; }
             fence_after();
             const uint32_t s_addr = tm_s0 + st * TKT + lane_addr;
             // does any row of the tile mask any key of this tile? (the first row sees the fewest late keys,
             // the last row the fewest early ones)
-            const bool edge = kb + TKT - 1 > ctx + row0 / G || (a.window > 0 && kb < ctx + last_row / G + 1 - a.window);
+            const bool edge = of_blocks ? kb + TKT > max(0, ctx + row0 / G + 1 - a.window) / a.pool
+                                        : kb + TKT - 1 > ctx + row0 / G || (a.window > 0 && kb < ctx + last_row / G + 1 - a.window);
             float s[TKT];
             {
                 float t0[32], t1[32];
@@ -931,10 +968,11 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
                 }
             }
             if (edge) {
+                const int first = of_blocks ? 0 : row_lo, last = of_blocks ? row_lo / a.pool - 1 : pos;
 #pragma unroll
                 for (int i = 0; i < TKT; ++i) {
                     const int key = kb + i;
-                    if (!(key >= row_lo && key <= pos)) s[i] = -INFINITY;
+                    if (!(key >= first && key <= last)) s[i] = -INFINITY;
                 }
             }
             {
@@ -1033,17 +1071,18 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
 }
 }  // namespace tc
 
-template <int D, bool PRECISE>
+template <int D, bool PRECISE, bool POOLED>
 static int launch_prefill_tc_as(const MmaAttnArgs& a, int n_tiles, cudaStream_t s) {
     static unsigned long long configured = 0;
-    if (int e = vcb_allow_dynamic_smem(tc::attention_prefill_tc_kernel<D, PRECISE>, tc::smem_bytes<D>(), &configured)) return e;
-    vcb_launch(tc::attention_prefill_tc_kernel<D, PRECISE>, dim3((unsigned)n_tiles * a.nkv), tc::THREADS, (size_t)tc::smem_bytes<D>(), s, a);
+    if (int e = vcb_allow_dynamic_smem(tc::attention_prefill_tc_kernel<D, PRECISE, POOLED>, tc::smem_bytes<D>(), &configured)) return e;
+    vcb_launch(tc::attention_prefill_tc_kernel<D, PRECISE, POOLED>, dim3((unsigned)n_tiles * a.nkv), tc::THREADS, (size_t)tc::smem_bytes<D>(), s, a);
     return vcb_last_error();
 }
 
 template <int D>
 static int launch_prefill_tc(const MmaAttnArgs& a, int n_tiles, cudaStream_t s) {
-    return a.precise_weights ? launch_prefill_tc_as<D, true>(a, n_tiles, s) : launch_prefill_tc_as<D, false>(a, n_tiles, s);
+    if (a.pooled) return launch_prefill_tc_as<D, true, true>(a, n_tiles, s);        // with two-term weights only
+    return a.precise_weights ? launch_prefill_tc_as<D, true, false>(a, n_tiles, s) : launch_prefill_tc_as<D, false, false>(a, n_tiles, s);
 }
 
 // Both kernels copy a tile of 64 keys as at most eight runs of whole pages' rows (tile_piece: one lane
@@ -1178,6 +1217,45 @@ VCB_EXPORT int vcb_attention_prefill_tc(const void* q, const void* cache, void* 
                                         int* status, void* stream) {
     return vcb_attention_prefill_tc_planes(q, cache, out, q_start, ctx_lens, block_table, bt_stride, tile_req, tile_row0,
                                            n_tiles, nh, nkv, d, page, window, scale, num_pages, status, 2, stream);
+}
+
+// Attention over a window of tokens and the rows of the blocks before it (see MmaAttnArgs), two-term weights.
+static int check_pooled(const void* pooled, const int* pool_table, int pt_stride, int pool_pages, int pool, int window) {
+    return (!pooled || !pool_table || pt_stride <= 0 || pool_pages <= 0 || pool <= 0 || window <= 0) ? VCB_ERR_BAD_ARG : 0;
+}
+
+VCB_EXPORT int vcb_attention_decode_mma_pooled(const void* q, const void* cache, const void* pooled, void* out, const int* q_start,
+                                               const int* ctx_lens, const int* block_table, int bt_stride, const int* pool_table,
+                                               int pt_stride, int n_list, int nsplit, float* part_o, float* part_ml, int* counters,
+                                               const int* split_tiles, int nh, int nkv, int d, int page, int window, int pool, float scale,
+                                               int num_pages, int pool_pages, int* status, int kv_share, void* stream) {
+    if (n_list <= 0) return 0;
+    if (int c = check_common(nh, nkv, d, page, window, num_pages)) return c;
+    if (int c = check_pooled(pooled, pool_table, pt_stride, pool_pages, pool, window)) return c;
+    if (kv_share < 1 || nkv % kv_share || nsplit < 1 || nsplit > 32 || (nsplit > 1 && (!part_o || !part_ml || !counters))) return VCB_ERR_BAD_ARG;
+    MmaAttnArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, q_start, ctx_lens,
+                  block_table, nullptr, nullptr, part_o, part_ml, counters, status, split_tiles, bt_stride, nh, nkv,
+                  page, window, scale, num_pages, 2, kv_share};
+    a.precise_weights = 1;
+    a.pooled = (const __nv_bfloat16*)pooled; a.pool_table = pool_table; a.pt_stride = pt_stride; a.pool_pages = pool_pages; a.pool = pool;
+    cudaStream_t s = (cudaStream_t)stream;
+    return d == 64 ? launch_decode<64>(a, n_list, nsplit, s) : launch_decode<128>(a, n_list, nsplit, s);
+}
+
+VCB_EXPORT int vcb_attention_prefill_tc_pooled(const void* q, const void* cache, const void* pooled, void* out, const int* q_start,
+                                               const int* ctx_lens, const int* block_table, int bt_stride, const int* pool_table,
+                                               int pt_stride, const int* tile_req, const int* tile_row0, int n_tiles, int nh, int nkv,
+                                               int d, int page, int window, int pool, float scale, int num_pages, int pool_pages,
+                                               int* status, void* stream) {
+    if (n_tiles <= 0) return 0;
+    if (int c = check_common(nh, nkv, d, page, window, num_pages)) return c;
+    if (int c = check_pooled(pooled, pool_table, pt_stride, pool_pages, pool, window)) return c;
+    MmaAttnArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, q_start, ctx_lens,
+                  block_table, tile_req, tile_row0, nullptr, nullptr, nullptr, status, nullptr, bt_stride, nh, nkv, page,
+                  window, scale, num_pages, 2, 1};
+    a.precise_weights = 1;
+    a.pooled = (const __nv_bfloat16*)pooled; a.pool_table = pool_table; a.pt_stride = pt_stride; a.pool_pages = pool_pages; a.pool = pool;
+    return d == 64 ? launch_prefill_tc<64>(a, n_tiles, (cudaStream_t)stream) : launch_prefill_tc<128>(a, n_tiles, (cudaStream_t)stream);
 }
 
 // ------------------------------------------------ no-allocation entry point

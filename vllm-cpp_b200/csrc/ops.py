@@ -90,6 +90,8 @@ _SIGNATURES = {
     "vcb_conv_rope_cache_write": [_P, _L, _P, _P, _I, _P, _L, _P, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
     "vcb_pool_blocks": [_P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
     "vcb_attention_pooled": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _I, _P],
+    "vcb_attention_decode_mma_pooled": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _I, _P],
+    "vcb_attention_prefill_tc_pooled": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P],
     "vcb_selective_scan": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P],
     "vcb_general_delta": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _F, _F, _P, _I, _I, _P],
     "vcb_tanh_rows": [_P, _L, _P, _L, _I, _I, _I, _P],
@@ -1465,6 +1467,43 @@ def attention_pooled(q: torch.Tensor, cache: torch.Tensor, pooled: Optional[torc
                                       row, page_size, window, pool if with_pool else 0, float(scale), cache.shape[0],
                                       pooled.shape[0] if with_pool else 0, status_tensor(q.device).data_ptr(), dtype_code(q.dtype),
                                       _stream()), "attention_pooled")
+
+
+def _pooled_checks(q, cache, pooled, out, head_dim, page_size, what):
+    _need(q.dtype == cache.dtype == pooled.dtype == out.dtype == torch.bfloat16, f"{what} is a bfloat16 kernel")
+    _need(head_dim in MMA_HEAD_DIMS and page_size % 8 == 0, f"{what} takes head sizes {MMA_HEAD_DIMS} and pages of a multiple of 8 slots")
+    _need(cache.shape[1:] == pooled.shape[1:], f"{what}: one page layout for tokens and blocks")
+
+
+def attention_decode_mma_pooled(q, cache, pooled, out, q_start, ctx_lens, block_table, pool_table, n_list: int, nsplit: int, part_o, part_ml,
+                                counters, *, num_heads: int, num_kv_heads: int, head_dim: int, page_size: int, window: int, pool: int,
+                                scale: float, split_tiles=None, kv_share: int = 1) -> None:
+    """``attention_decode_mma`` over a window of tokens and, before it, the rows of the blocks of ``pool`` tokens (``pooled``
+    pages, ``pool_table``); the softmax weights enter the product with the values as two bfloat16 terms."""
+    _pooled_checks(q, cache, pooled, out, head_dim, page_size, "attention_decode_mma_pooled")
+    _need(nsplit == 1 or (part_o.numel() >= n_list * num_heads * nsplit * head_dim and part_ml.numel() >= n_list * num_heads * nsplit * 2
+                          and counters.numel() >= n_list * num_kv_heads), "attention_decode_mma_pooled: scratch for the split merge is too small")
+    opt = lambda t, name, dt: None if t is None else _dev(t, name, dt)
+    _check(lib().vcb_attention_decode_mma_pooled(
+        _dev(q, "q"), _dev(cache, "cache"), _dev(pooled, "pooled"), _dev(out, "out"), _dev(q_start, "q_start", torch.int32),
+        _dev(ctx_lens, "ctx_lens", torch.int32), _dev(block_table, "block_table", torch.int32), block_table.shape[1],
+        _dev(pool_table, "pool_table", torch.int32), pool_table.shape[1], n_list, nsplit, opt(part_o, "part_o", torch.float32),
+        opt(part_ml, "part_ml", torch.float32), opt(counters, "counters", torch.int32), opt(split_tiles, "split_tiles", torch.int32),
+        num_heads, num_kv_heads, head_dim, page_size, window, pool, float(scale), cache.shape[0], pooled.shape[0],
+        status_tensor(q.device).data_ptr(), kv_share, _stream()), "attention_decode_mma_pooled")
+
+
+def attention_prefill_tc_pooled(q, cache, pooled, out, q_start, ctx_lens, block_table, pool_table, tile_req, tile_row0, *, num_heads: int,
+                                num_kv_heads: int, head_dim: int, page_size: int, window: int, pool: int, scale: float) -> None:
+    """``attention_prefill_tc`` over a window of tokens and the rows of the blocks before it, two-term weights."""
+    _pooled_checks(q, cache, pooled, out, head_dim, page_size, "attention_prefill_tc_pooled")
+    _need(tile_row0.numel() == tile_req.numel(), "one first row per tile")
+    _check(lib().vcb_attention_prefill_tc_pooled(
+        _dev(q, "q"), _dev(cache, "cache"), _dev(pooled, "pooled"), _dev(out, "out"), _dev(q_start, "q_start", torch.int32),
+        _dev(ctx_lens, "ctx_lens", torch.int32), _dev(block_table, "block_table", torch.int32), block_table.shape[1],
+        _dev(pool_table, "pool_table", torch.int32), pool_table.shape[1], _dev(tile_req, "tile_req", torch.int32),
+        _dev(tile_row0, "tile_row0", torch.int32), tile_req.numel(), num_heads, num_kv_heads, head_dim, page_size, window, pool, float(scale),
+        cache.shape[0], pooled.shape[0], status_tensor(q.device).data_ptr(), _stream()), "attention_prefill_tc_pooled")
 
 
 # ------------------------------------------------- selective state space, generalised delta rule, joined results

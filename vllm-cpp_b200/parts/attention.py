@@ -32,8 +32,10 @@ class PagedAttentionKernels(Mixer):
     """What a mixer needs to run the engine's paged attention kernels on queries it has made: the per-step
     work lists, the kernels' scratch and the choice of kernel.  A subclass sets ``nh`` (query heads),
     ``nkv`` (heads of the cache), ``d`` (width of a cached row), ``window``, ``scale``, ``dtype`` and
-    ``planes`` (PagedKVSpec.planes: 2 for keys and values, 1 for rows that are both)."""
+    ``planes`` (PagedKVSpec.planes: 2 for keys and values, 1 for rows that are both); ``pool`` > 0 with a window: beside
+    the window's tokens a row per block of ``pool`` tokens that lies before it, in pages of its own (``attend``'s ``blocks``)."""
     planes = 2
+    pool = 0
 
     # -- work lists and kernel choice
     def _tensor_core_path(self) -> bool:
@@ -82,6 +84,8 @@ class PagedAttentionKernels(Mixer):
             hi = np.asarray(host.ctx_lens, dtype=np.int64) + 1
             lo = np.maximum(0, hi - self.window) if self.window > 0 else np.zeros_like(hi)
             n = -(-hi // tile) - lo // tile                     # key tiles of every request
+            if self.pool:
+                n = n + -(-(lo // self.pool) // tile)           # and those of the blocks before its window
             slots = self.decode_slots(len(n))
             low, high = max(1, -(-int(n.sum()) // slots)), int(n.max())
             while low < high:                                   # smallest count whose splits fit the slots
@@ -123,7 +127,7 @@ class PagedAttentionKernels(Mixer):
             ops.zeroed_ints("attn_tickets", n_reqs * self.decode_groups(), device)
 
     def _splits_key(self):
-        return f"attn_splits_kv{self.decode_groups()}_w{self.window}"
+        return f"attn_splits_kv{self.decode_groups()}_w{self.window}" + (f"_p{self.pool}" if self.pool else "")
 
     def score_shaping(self) -> dict:
         """What the tensor-core kernels do to a score beyond the scale: ``cap`` (cap * tanh(score / cap)) and ``bias_t``
@@ -131,13 +135,18 @@ class PagedAttentionKernels(Mixer):
         denominator once); empty for plain scaled scores."""
         return {}
 
-    def attend(self, q, attn, step, cache, block_table, head_gate=None):
-        """``head_gate`` (tensor-core kernels only): logits [tokens, heads]; a head's output is multiplied by their sigmoid."""
+    def attend(self, q, attn, step, cache, block_table, head_gate=None, blocks=None):
+        """``head_gate`` (tensor-core kernels only): logits [tokens, heads]; a head's output is multiplied by their sigmoid.
+        ``blocks`` (tensor-core kernels only): (pages, block table) of the rows of blocks, for mixers with a ``pool``."""
         if self._tensor_core_path():
             kw = dict(num_heads=self.nh, num_kv_heads=self.nkv, head_dim=self.d, page_size=cache.page_size,
                       window=self.window, scale=self.scale, planes=self.planes, **self.score_shaping())
             if head_gate is not None:
                 kw["head_gate"] = head_gate
+            pooled = ()
+            if blocks is not None:
+                kw = {name: kw[name] for name in ("num_heads", "num_kv_heads", "head_dim", "page_size", "window", "scale")}
+                kw["pool"], pooled = self.pool, blocks
             if step.decode_only:
                 nsplit = step.shapes.get(self._splits_key())
                 split_tiles = step.extras.get(self._splits_key())
@@ -145,7 +154,7 @@ class PagedAttentionKernels(Mixer):
                     # a step without the builder's arrays: every request in equal parts, as many as fill
                     # the device once, from the longest context's power-of-two bucket
                     longest = step.split_len or step.max_total_len
-                    if self.window > 0:
+                    if self.window > 0 and not self.pool:
                         longest = min(longest, self.window + 64)
                     nsplit = max(1, min(-(-longest // 64), 2 * ops.sm_count() // (step.n_reqs * self.decode_groups()),
                                         ops.DECODE_MAX_SPLITS))
@@ -157,11 +166,19 @@ class PagedAttentionKernels(Mixer):
                     part_ml = ops.scratch("attn_part_ml", need * 2, q.device)
                     counters = ops.zeroed_ints("attn_tickets", step.n_reqs * self.decode_groups(), q.device)
                 share = ops.decode_head_groups(self.nh, self.nkv)
+                kw = dict(kw, num_kv_heads=self.nkv * share, kv_share=share)
+                if pooled:
+                    ops.attention_decode_mma_pooled(q, cache.pages, pooled[0], attn, step.q_start, step.ctx_lens, block_table, pooled[1],
+                                                    step.n_reqs, nsplit, part_o, part_ml, counters, split_tiles=split_tiles, **kw)
+                    return
                 ops.attention_decode_mma(q, cache.pages, attn, step.q_start, step.ctx_lens, block_table, None,
-                                         step.n_reqs, nsplit, part_o, part_ml, counters, split_tiles=split_tiles,
-                                         **dict(kw, num_kv_heads=self.nkv * share, kv_share=share))
+                                         step.n_reqs, nsplit, part_o, part_ml, counters, split_tiles=split_tiles, **kw)
             else:
                 tiles = step.extras[f"attn_tiles_g{self.nh // self.nkv}"]
+                if pooled:
+                    ops.attention_prefill_tc_pooled(q, cache.pages, pooled[0], attn, step.q_start, step.ctx_lens, block_table, pooled[1],
+                                                    tiles[0], tiles[1], **kw)
+                    return
                 ops.attention_prefill_tc(q, cache.pages, attn, step.q_start, step.ctx_lens, block_table, tiles[0], tiles[1], **kw)
             return
         if head_gate is not None:

@@ -12,8 +12,10 @@ value per block of ``pool`` tokens:
 ``window`` 0: every token is seen; ``pool`` 0: nothing before the window is.  The mixer keeps three things per request: the
 window's pages (of which those of a block that is not complete yet are not given back, PagedKVSpec.keep_block), pages with a row
 per complete block (PagedKVSpec.stride), and the convolutions' last inputs in a state slot.  Convolution, rotation, the
-heads' factor and the cache write are one kernel, the means of the blocks a step completes a second, attention the third
-(csrc/attention_pooled.cu).  The reference's attention (src/layers/attention.cpp) has a rotation and none of the rest.
+heads' factor and the cache write are one kernel, the means of the blocks a step completes a second (csrc/attention_pooled.cu),
+attention the third: in bfloat16, with heads of 64 or 128 and keys as wide as values, the tensor-core kernels of
+csrc/attention_mma.cu, which walk the tiles of block rows before the tiles of tokens and take the softmax weights as two
+bfloat16 terms; else the plain kernel.  The reference's attention (src/layers/attention.cpp) has a rotation and none of the rest.
 """
 from __future__ import annotations
 
@@ -80,6 +82,8 @@ class PooledWindowAttention(PagedAttentionKernels):
         if self.temperature:
             self.temp = t["temp"].contiguous()
         self.w_o = t["o"].contiguous()
+        if self.dk == self.dv:
+            self.warn_if_plain()
 
     def tensors(self):
         return super().tensors() + self.position.tensors()
@@ -95,7 +99,12 @@ class PooledWindowAttention(PagedAttentionKernels):
         return CompositeSpec(tuple(parts))
 
     def _tensor_core_path(self) -> bool:
-        return False
+        # bfloat16 heads of 64 and 128 with keys as wide as values: the tcgen05 kernel for portions, split-KV for single tokens
+        return self.dk == self.dv and super()._tensor_core_path()
+
+    def score_shaping(self):
+        # the design wants its attention weights in 32-bit: the tensor-core kernels take them as two bfloat16 terms
+        return {"precise_weights": True}
 
     def workspace_bytes(self, n_tokens, n_reqs):
         return (workspace_piece((n_tokens, self.channels), self.dtype) + workspace_piece((n_tokens, self.nh * self.dk), self.dtype)
@@ -130,7 +139,10 @@ class PooledWindowAttention(PagedAttentionKernels):
         if blocks is not None:
             ops.pool_blocks(pages, pooled, step.q_start, step.ctx_lens, table, pool_table, step.n_reqs, step.max_q_len, pool=self.pool, **sizes)
         attn = ws.take((n, self.nh * self.dv), self.dtype)
-        ops.attention_pooled(q, pages, pooled, attn, step.positions, step.req_of_token, table, pool_table, num_heads=self.nh,
-                             window=self.window, pool=self.pool, scale=self.scale, **sizes)
+        if self._tensor_core_path() and tokens.page_size % 8 == 0:
+            self.attend(q, attn, step, tokens, table, blocks=None if blocks is None else (blocks.pages, pool_table))
+        else:
+            ops.attention_pooled(q, pages, pooled, attn, step.positions, step.req_of_token, table, pool_table, num_heads=self.nh,
+                                 window=self.window, pool=self.pool, scale=self.scale, **sizes)
         ops.linear(attn, self.w_o, out)
         ws.release(mark)
