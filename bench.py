@@ -714,7 +714,7 @@ def decode_step_bytes(model, cache, batch, context):
     el = model.embed.element_size()
     for spec in flatten_specs(model.cache_specs()):
         if isinstance(spec, PagedKVSpec):
-            keys = min(context, spec.window) if spec.window else context
+            keys = min(context, spec.window) if spec.window else context // spec.stride
             total += batch * keys * spec.planes * spec.num_kv_heads * spec.head_dim * el
         elif isinstance(spec, StateSpec):
             n = 4
@@ -1434,6 +1434,214 @@ REFERENCE_NOTES = ("the reference's own faults at these sizes, none of which cha
                    "layer 0's rotation table below position 336")
 
 
+# ------------------------------------------------------------------- the Kasuvik design beside Retodra
+# Layer sizes that resemble real models'.  Kasuvik: layers of the generalised delta rule in turn with layers of windowed
+# attention with block means beside a selective state space.  Retodra with dense feed-forwards (gated linear attention in turn
+# with windowed attention beside lightning attention, the same arrangement of norms) at equal width, heads, kv heads, head
+# size, window and feed-forward width is the nearest model the engine has.
+KASUVIK_SIZES = {"2k": dict(width=2048, heads=16, kv_heads=4, dim=128, ff=8192, layers=4),
+                 "4k": dict(width=4096, heads=32, kv_heads=8, dim=128, ff=14336, layers=4)}
+KASUVIK_VOCAB, KASUVIK_CONTEXT, KASUVIK_PROMPT, KASUVIK_WINDOW, KASUVIK_POOL, KASUVIK_STATE, KASUVIK_DELTA_DIM = 32000, 2048, 2048, 1024, 16, 16, 64
+
+
+def kasuvik_configs(size):
+    z = KASUVIK_SIZES[size]
+    w, h, d = z["width"], z["heads"], z["dim"]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    delta = {"type": "general_delta", "mixer": {"heads": w // KASUVIK_DELTA_DIM, "dim": KASUVIK_DELTA_DIM}, "mlp": mlp}
+    par = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": h, "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "conv": 4, "scale": d ** -0.5, "rot": {"base": 1e6, "dims": d},
+                 "mask": {"size": KASUVIK_WINDOW, "pool": KASUVIK_POOL}},
+        "right": {"inner": 2 * w, "state": KASUVIK_STATE, "dt_rank": w // 16, "conv": 4}}}
+    kasuvik = {"architecture": "Kasuvik", "vocab": KASUVIK_VOCAB, "width": w, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+               "layers": [delta if i % 2 == 0 else par for i in range(z["layers"])]}
+    retodra, _ = retodra_configs(size)
+    retodra = dict(retodra, vocab=KASUVIK_VOCAB, layers=[dict(l, mlp=mlp) for l in retodra["layers"]])
+    return kasuvik, retodra
+
+
+def run_kasuvik(a) -> int:
+    """Prefill and decode throughput of the Kasuvik design beside Retodra with dense feed-forwards at equal layer sizes (random
+    weights, synthetic cache contents), and the design's own kernels alone beside the like kernels of the engine's other models
+    with their share of the measured peaks.  One JSON line."""
+    import numpy as np
+    peaks = load_peaks()
+    steps, warmup = max(1, a.steps), max(3, a.warmup)
+    rng = np.random.default_rng(0)
+    sampler = ClockSampler()
+    sampler.start()
+    sampler.mark("decode")
+    out = {"metric": "prefill and decode tok/s of Kasuvik beside Retodra with dense feed-forwards at equal layer sizes (bf16, random weights)",
+           "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic", "sizes": {}, "peaks": peaks}
+    sizes = a.kasuvik.split(",") if a.kasuvik != "all" else sorted(KASUVIK_SIZES)
+    for size in sizes:
+        kasuvik, retodra = kasuvik_configs(size)
+        args = (steps, warmup, rng, peaks, KASUVIK_VOCAB, KASUVIK_CONTEXT, KASUVIK_PROMPT)
+        out["sizes"][size] = {"layers": KASUVIK_SIZES[size], "kasuvik": measure_design(kasuvik, (8, 64), *args),
+                              "retodra_dense": measure_design(retodra, (8, 64), *args)}
+    if not a.skip_points:
+        out["kernels"] = kasuvik_kernels(KASUVIK_SIZES[sizes[-1]], peaks)
+    out["clocks"] = sampler.stop()
+    big = out["sizes"][sizes[-1]]
+    out.update(value=big["kasuvik"]["decode"]["8"]["tok_s"], unit=f"tokens/s (Kasuvik, {sizes[-1]}-wide layers, batch 8)",
+               higher_is_better=True, gpu_launches=big["kasuvik"]["decode"]["8"]["launches_per_step"] * steps,
+               config={"sizes": KASUVIK_SIZES, "context": KASUVIK_CONTEXT, "prompt": KASUVIK_PROMPT, "window": KASUVIK_WINDOW,
+                       "pool": KASUVIK_POOL, "state": KASUVIK_STATE, "l2": "a step's weights exceed the 126 MB of L2"})
+    print(json.dumps(out))
+    return 0
+
+
+def kasuvik_kernels(z, peaks):
+    """The design's own kernels alone at one layer size, each beside the like kernel of another model of the engine:
+    [{kernel, like, us, GB/s or TFLOP/s, share of the measured peak}, ...] (CUDA graphs on rotating buffers)."""
+    import torch
+    from vllm_cpp_b200.csrc import ops
+    h, bf, dev = z["width"], torch.bfloat16, "cuda"
+    rows = []
+
+    def rnd(*shape, dtype=bf, scale=1.0):
+        return (torch.randn(*shape, device=dev) * scale).to(dtype)
+
+    def add(name, like, fn, copies, bytes_=0, flops=0, peak=None):
+        us = ops.time_in_graph(fn, reps=max(4, copies))
+        rate = bytes_ / us / 1e3 if bytes_ else flops / us / 1e6
+        row = {"kernel": name, "like": like, "us": round(us, 2), ("gb_s" if bytes_ else "tflop_s"): round(rate, 1)}
+        if bytes_ or peak != "none":
+            row["of_peak"] = round(rate / (peaks["hbm_gbs"] if bytes_ else peaks["bf16_tflops"]), 4)
+        rows.append(row)
+
+    # ---- rows: the two mixers' results joined into the stream, relu in the feed-forward
+    for t in (64, 2048):
+        c = 6 if t == 64 else 3
+        x = [rnd(t, h, dtype=torch.float32) for _ in range(c)]
+        ya, yb, o1 = ([rnd(t, h) for _ in range(c)] for _ in range(3))
+        gain = torch.ones(h, device=dev)
+        add(f"two results normed and joined + post norm + addition + next norm, {t} tokens", "", lambda i: ops.pair_norm(
+            ya[i % c], yb[i % c], gain, gain, 0.5, 0.5, 1e-6, o1[i % c], x=x[i % c], gain=gain, eps=1e-6, next_gain=gain, next_eps=1e-6), c, bytes_=t * h * 14)
+        add(f"Retodra: post norm + layer scale + addition + next norm, {t} tokens", "like the one above", lambda i: ops.norm_residual_norm(
+            ya[i % c], gain, x[i % c], 1e-6, next_gain=gain, next_out=o1[i % c], next_eps=1e-6), c, bytes_=t * h * 12)
+        gu, act = [rnd(t, 2 * z["ff"]) for _ in range(c)], torch.empty(t, z["ff"], dtype=bf, device=dev)
+        add(f"relu(gate) * up, width {z['ff']}, {t} tokens", "", lambda i: ops.relu_mul(gu[i % c], act), c, bytes_=t * z["ff"] * 6)
+        add(f"Retodra: silu(gate) * up, width {z['ff']}, {t} tokens", "like the one above", lambda i: ops.silu_mul(gu[i % c], act), c, bytes_=t * z["ff"] * 6)
+    # ---- the recurrences: single tokens of a batch, then a prompt
+    dk = KASUVIK_DELTA_DIM
+    H, I, N, J = h // dk, 2 * h, KASUVIK_STATE, 4
+    for n_reqs, per in ((8, 1), (64, 1), (1, KASUVIK_PROMPT)):
+        t, c = n_reqs * per, 3
+        what = f"decode, batch {n_reqs}" if per == 1 else f"prompt of {per}"
+        q_start = torch.arange(0, t + 1, per, dtype=torch.int32, device=dev)
+        slots = torch.arange(n_reqs, dtype=torch.int32, device=dev)
+        r, k, v, a, zz = (rnd(t, h) for _ in range(5))
+        o, zero = torch.empty(t, h, device=dev), torch.zeros(h, device=dev)
+        state = [torch.zeros(n_reqs, H, dk, dk, device=dev) for _ in range(c)]
+        work = torch.empty(ops.general_delta_work(t, H, dk, dk), device=dev)
+        moved = dict(bytes_=n_reqs * H * dk * dk * 8)
+        many = lambda f: moved if per == 1 else dict(flops=f * t * H * dk * dk, peak="none")
+        add(f"generalised delta rule, {H} heads of {dk} x {dk}, {what}", "", lambda i: ops.general_delta(
+            r, k, v, a, zz, zero, zero, state[i % c], o, q_start, slots, n_reqs, per, num_heads=H, rate=0.6, unit_eps=1e-6, work=work), c, **many(9.0))
+        qf, kf, vf = (rnd(t, h, dtype=torch.float32) for _ in range(3))
+        beta, al = rnd(t, H), torch.zeros(H, device=dev)
+        add(f"Lutodra: gated delta rule, {H} heads of {dk} x {dk}, {what}", "like the one above", lambda i: ops.gated_delta_scan(
+            qf, kf, vf, beta, zz, al, zero, state[i % c], o, q_start, slots, n_reqs, num_heads=H, num_qk_heads=H, q_scale=0.125, unit_eps=1e-6,
+            max_q_len=per), c, **many(7.0))
+        del r, k, v, a, qf, kf, vf, state, work
+        xz, dt, y = [rnd(t, 2 * I) for _ in range(c)], rnd(t, I, scale=0.5), torch.empty(t, I, dtype=bf, device=dev)
+        bc, taps = rnd(t, 2 * N), rnd(I, J, dtype=torch.float32)
+        a2, one = -torch.rand(I, N, device=dev) - 0.1, torch.ones(I, device=dev)
+        st = [torch.zeros(n_reqs, I, N, device=dev) for _ in range(c)]
+        window = torch.zeros(n_reqs, J - 1, I, device=dev)
+        add(f"causal convolution of {J} taps + silu, {I} channels, {what}", "Lutodra runs the same kernel", lambda i: ops.causal_conv(
+            xz[i % c][:, :I], taps, window, y, q_start, slots, n_reqs, per, bias=one, act="silu"), c, bytes_=t * I * 4 + 2 * n_reqs * (J - 1) * I * 4)
+        size = t * I * 8 + n_reqs * I * N * 8
+        add(f"selective state space, {I} channels of {N}, {what}", "", lambda i: ops.selective_scan(
+            xz[i % c][:, :I], dt, bc[:, :N], bc[:, N:], xz[i % c][:, I:], one, a2, one, st[i % c], y, q_start, slots, n_reqs, per), c, bytes_=size)
+        dec, drv = torch.rand(t, I, device=dev), rnd(t, I, dtype=torch.float32)
+        st1 = torch.zeros(n_reqs, I, device=dev)
+        add(f"Lutodra: linear recurrence + gelu branch, {I} channels of 1, {what}", "like the one above", lambda i: ops.linear_recurrence(
+            dec, drv, xz[i % c][:, :I], one, st1, y, q_start, slots, n_reqs, per), c, bytes_=t * I * 12 + n_reqs * I * 8)
+        del xz, dt, y, st, dec, drv
+    kasuvik_attention_kernels(z, add, rnd)
+    ops.check_status()
+    return rows
+
+
+def kasuvik_attention_kernels(z, add, rnd):
+    """Convolution + rotation + cache write, the means of blocks, and attention over a window and block means, beside Lutodra's
+    head norm + rotation + cache write and attention over a window alone (two-term weights in both)."""
+    import numpy as np
+    import torch
+    from vllm_cpp_b200.config.model_spec import PartSpec
+    from vllm_cpp_b200.csrc import ops
+    from vllm_cpp_b200.engine.runner import HostStep
+    from vllm_cpp_b200.parts.attention import PagedAttention
+    h, nh, nkv, d, page, bf, dev = z["width"], z["heads"], z["kv_heads"], z["dim"], 16, torch.bfloat16, "cuda"
+    W, P, J = KASUVIK_WINDOW, KASUVIK_POOL, 4
+    C = (nh + 2 * nkv) * d
+    ints = lambda a: torch.tensor(np.asarray(a), dtype=torch.int32, device=dev)
+    taps, bias, temp = rnd(C, J, dtype=torch.float32), torch.zeros(C, device=dev), torch.ones(nh, device=dev)
+    inv = torch.from_numpy((1e6 ** (-2.0 * np.arange(d // 2) / d)).astype(np.float32)).to(dev)
+    gain = torch.ones(d, device=dev)
+    sizes = dict(num_kv_heads=nkv, head_dim=d, v_head_dim=d, row=d, page_size=page)
+    for n_reqs, per in ((8, 1), (64, 1), (1, KASUVIK_PROMPT)):
+        t, c = n_reqs * per, 3
+        what = f"{t} single tokens" if per == 1 else f"prompt of {per}"
+        ctx = KASUVIK_CONTEXT if per == 1 else 0
+        blocks = (ctx + per) // page + 1
+        bt = ints(np.arange(n_reqs * blocks)).view(n_reqs, blocks)
+        pt = ints(np.arange(n_reqs * blocks)).view(n_reqs, blocks)
+        proj = [rnd(t, C) for _ in range(c)]
+        kv, pooled = rnd(n_reqs * blocks, 2, nkv, page * d), rnd(n_reqs * blocks, 2, nkv, page * d)
+        pages, rows_ = kv.view(kv.shape[0], -1), pooled.view(pooled.shape[0], -1)
+        q_start, pos, req, slots = ints(np.arange(0, t + 1, per)), ints(np.tile(np.arange(ctx, ctx + per), n_reqs)), ints(np.repeat(np.arange(n_reqs), per)), ints(np.arange(n_reqs))
+        state, q, ctxs = torch.zeros(n_reqs, J - 1, C, device=dev), torch.empty(t, nh * d, dtype=bf, device=dev), ints([ctx] * n_reqs)
+        add(f"convolution of {J} taps + rotation of {d} of {d} + cache write, {what}", "", lambda i: ops.conv_rope_cache_write(
+            proj[i % c], bias, taps, state, inv, temp, q, pages, q_start, pos, slots, bt, n_reqs, per, num_heads=nh, **sizes), c,
+            bytes_=t * C * 4 + 2 * n_reqs * (J - 1) * C * 4)
+        add(f"Lutodra: head norms + rotation of {d} of {d} + cache write, {what}", "like the one above", lambda i: ops.qk_head_rope_cache_write(
+            proj[i % c], 0, nh * d, (nh + nkv) * d, gain, gain, inv, q, pages, pos, req, bt, num_heads=nh, eps=1e-6, write_kv=True, **sizes), c, bytes_=t * C * 4)
+        full = ints([ctx // P * P + P - 1] * n_reqs) if per == 1 else ctxs
+        add(f"means of the blocks of {P} that end in {what}", "", lambda i: ops.pool_blocks(pages, rows_, q_start, full, bt, pt, n_reqs, per, pool=P, **sizes), c,
+            bytes_=max(n_reqs, t // P) * (P + 1) * 2 * nkv * d * 2)
+    # ---- attention: a prompt, then single tokens
+    t, G = KASUVIK_PROMPT, nh // nkv
+    n_pages = t // page + 2
+    bt = ints(np.arange(n_pages)).view(1, -1)
+    q_start, ctx = ints([0, t]), ints([0])
+    n_tiles = -(-t * G // ops.TC_ATTENTION_TILE_ROWS)
+    tile_req, tile_row0 = ints(np.zeros(n_tiles)), ints((np.arange(n_tiles) * ops.TC_ATTENTION_TILE_ROWS)[::-1].copy())
+    q, o = rnd(t, nh * d), torch.empty(t, nh * d, dtype=bf, device=dev)
+    kv, pooled = rnd(n_pages, 2, nkv, page * d, scale=0.5), rnd(n_pages, 2, nkv, page * d, scale=0.5)
+    kw = dict(num_heads=nh, num_kv_heads=nkv, head_dim=d, page_size=page, window=W, scale=d ** -0.5)
+    add(f"attention, window {W} and means of blocks of {P}, two-term weights, prompt of {t}", "", lambda i: ops.attention_prefill_tc_pooled(
+        q, kv, pooled, o, q_start, ctx, bt, bt, tile_req, tile_row0, pool=P, **kw), 4, flops=4.0 * nh * d * sum(min(i + 1, W) + max(0, i + 1 - W) // P for i in range(t)))
+    add(f"Lutodra's kernel: attention, window {W}, two-term weights, prompt of {t}", "like the one above", lambda i: ops.attention_prefill_tc(
+        q, kv, o, q_start, ctx, bt, tile_req, tile_row0, precise_weights=True, **kw), 4, flops=4.0 * nh * d * sum(min(i + 1, W) for i in range(t)))
+    part = PagedAttention(h, nh, nkv, d, True, False, W, PartSpec("none"), bf, dev)
+    for batch in (8, 64):
+        contexts, blocks = [KASUVIK_CONTEXT - 1] * batch, -(-KASUVIK_CONTEXT // page)
+        bt, q_start, ctx = ints(np.arange(batch * blocks)).view(batch, blocks), ints(np.arange(batch + 1)), ints(contexts)
+        q, o = rnd(batch, nh * d), torch.empty(batch, nh * d, dtype=bf, device=dev)
+        kv, pooled = rnd(batch * blocks + 1, 2, nkv, page * d, scale=0.5), rnd(batch * blocks + 1, 2, nkv, page * d, scale=0.5)
+        share = ops.decode_head_groups(nh, nkv)
+        for pool in (P, 0):
+            part.pool = pool
+            host = HostStep([1] * batch, contexts, page)
+            tiles = ints(part.step_arrays()[part._splits_key()](host))
+            ns = host.shapes[part._splits_key()]
+            scratch = (torch.empty(batch * nh * ns * d, device=dev), torch.empty(batch * nh * ns * 2, device=dev),
+                       torch.zeros(batch * nkv * share, dtype=torch.int32, device=dev))
+            kw = dict(num_heads=nh, num_kv_heads=nkv * share, head_dim=d, page_size=page, window=W, scale=d ** -0.5, split_tiles=tiles, kv_share=share)
+            keys = W + ((KASUVIK_CONTEXT - W) // pool if pool else 0)
+            if pool:
+                add(f"attention, window {W} and means of blocks of {P}, two-term weights, decode, batch {batch}, context {KASUVIK_CONTEXT}", "",
+                    lambda i: ops.attention_decode_mma_pooled(q, kv, pooled, o, q_start, ctx, bt, bt, batch, ns, *scratch, pool=pool, **kw), 4,
+                    bytes_=batch * keys * 2 * nkv * d * 2)
+            else:
+                add(f"Lutodra's kernel: attention, window {W}, two-term weights, decode, batch {batch}", "like the one above",
+                    lambda i: ops.attention_decode_mma(q, kv, o, q_start, ctx, bt, None, batch, ns, *scratch, precise_weights=True, **kw), 4,
+                    bytes_=batch * keys * 2 * nkv * d * 2)
+
+
 def unavailable(why: str) -> int:
     print(json.dumps({"impl": "reference", "unavailable": " ".join(str(why).split())[:600]}))
     return 0
@@ -1585,6 +1793,10 @@ def main() -> int:
                     help="instead of the benchmark's workload: prefill and decode throughput of the Gipinex design beside Lutodra's "
                          "attention layers at equal layer sizes, and the design's kernels alone: 'all' or a comma list of "
                          + ",".join(sorted(GIPINEX_SIZES)))
+    ap.add_argument("--kasuvik", default="", metavar="SIZES",
+                    help="instead of the benchmark's workload: prefill and decode throughput of the Kasuvik design beside Retodra "
+                         "with dense feed-forwards at equal layer sizes, and the design's kernels alone: 'all' or a comma list of "
+                         + ",".join(sorted(KASUVIK_SIZES)))
     ap.add_argument("--retodra", default="", metavar="SIZES",
                     help="instead of the benchmark's workload: prefill and decode throughput of the Retodra design beside Qwen2 "
                          f"at equal layer sizes ({','.join(sorted(RETODRA_SIZES))} or 'all'), and the design's kernels alone "
@@ -1628,6 +1840,8 @@ def main() -> int:
         return run_lutodra(a)
     if a.gipinex:
         return run_gipinex(a)
+    if a.kasuvik:
+        return run_kasuvik(a)
     if a.mix:
         return run_mix(cfg, a)
     if a.kernels:

@@ -240,8 +240,8 @@ struct PoolArgs {
 };
 
 // Grid (blocks a request can complete in this step, requests, kv heads): block ctx / P + blockIdx.x of the request, if this
-// step brings its last token.  Keys and then values; a thread per element, the block's tokens in order.
-template <typename T>
+// step brings its last token.  Keys and then values; a thread per VW neighbouring elements, the block's tokens in order.
+template <typename T, int VW>
 __global__ void __launch_bounds__(128) pool_blocks_kernel(PoolArgs a) {
     pdl_start();
     const int r = blockIdx.y, g = blockIdx.z;
@@ -256,22 +256,30 @@ __global__ void __launch_bounds__(128) pool_blocks_kernel(PoolArgs a) {
         if (a.status && threadIdx.x == 0) atomicCAS(a.status, 0, VCB_STATUS_BAD_PAGE);
         return;
     }
-    for (int e = threadIdx.x; e < a.dk + a.dv; e += blockDim.x) {
+    const int first = b * a.P, lp0 = first / a.page, slot0 = first - lp0 * a.page;
+    for (int e = threadIdx.x * VW; e < a.dk + a.dv; e += blockDim.x * VW) {
         const bool is_v = e >= a.dk;
         const int el = is_v ? e - a.dk : e;
         const size_t head = (size_t)(is_v ? a.nkv + g : g) * block;
-        float sum = 0.0f;
-#pragma unroll 4
+        float sum[VW];
+#pragma unroll
+        for (int i = 0; i < VW; ++i) sum[i] = 0.0f;
+#pragma unroll 8
         for (int k = 0; k < a.P; ++k) {
-            const int pos = b * a.P + k, lp = pos / a.page, slot = pos - lp * a.page;
+            const int at = slot0 + k, over = at / a.page, slot = at - over * a.page, lp = lp0 + over;
             const int pg = lp < a.bt_stride ? bt[lp] : -1;
             if ((unsigned)pg >= (unsigned)a.num_pages) {
                 if (a.status) atomicCAS(a.status, 0, VCB_STATUS_BAD_PAGE);
                 continue;
             }
-            sum += to_f32<T>(((const T*)a.cache)[(size_t)pg * page_elems + head + kv_pos(el, slot, a.row, a.page, (int)sizeof(T))]);
+            float v[VW];
+            conv_load<T, VW>((const T*)a.cache + (size_t)pg * page_elems + head + kv_pos(el, slot, a.row, a.page, (int)sizeof(T)), v);
+#pragma unroll
+            for (int i = 0; i < VW; ++i) sum[i] += v[i];
         }
-        ((T*)a.pooled)[(size_t)ppg * page_elems + head + kv_pos(el, pslot, a.row, a.page, (int)sizeof(T))] = from_f32<T>(sum / (float)a.P);
+        T* dst = (T*)a.pooled + (size_t)ppg * page_elems + head + kv_pos(el, pslot, a.row, a.page, (int)sizeof(T));
+#pragma unroll
+        for (int i = 0; i < VW; ++i) dst[i] = from_f32<T>(sum[i] / (float)a.P);
     }
 }
 
@@ -286,8 +294,11 @@ VCB_EXPORT int vcb_pool_blocks(const void* cache, void* pooled, const int* q_sta
     // a portion of n tokens completes at most ceil(n / P) blocks
     dim3 grid((max_q_len + P - 1) / P, n_reqs, nkv);
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == VCB_F32) vcb_launch(pool_blocks_kernel<float>, grid, 128, 0, s, a);
-    else if (dtype == VCB_BF16) vcb_launch(pool_blocks_kernel<__nv_bfloat16>, grid, 128, 0, s, a);
+    const bool pairs = !((dk | dv | row) & 1) && !(((uintptr_t)cache | (uintptr_t)pooled) & 7);
+    if (dtype == VCB_F32 && pairs) vcb_launch(pool_blocks_kernel<float, 2>, grid, 128, 0, s, a);
+    else if (dtype == VCB_F32) vcb_launch(pool_blocks_kernel<float, 1>, grid, 128, 0, s, a);
+    else if (dtype == VCB_BF16 && pairs) vcb_launch(pool_blocks_kernel<__nv_bfloat16, 2>, grid, 128, 0, s, a);
+    else if (dtype == VCB_BF16) vcb_launch(pool_blocks_kernel<__nv_bfloat16, 1>, grid, 128, 0, s, a);
     else return VCB_ERR_BAD_ARG;
     return vcb_last_error();
 }

@@ -198,66 +198,104 @@ __device__ __forceinline__ void gd_copy(float* smem, const float* gmem, int byte
     else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(gmem) : "memory");
 }
 
-// Grid (request, head, tile of DVT value channels), P lanes of a warp per column of S, DKP rows of the column in a thread.
-template <int DKP>
-__global__ void __launch_bounds__(128) general_delta_walk_kernel(GDeltaArgs A, const float* __restrict__ work, int P, int DVT) {
+// Two floats to a 64-bit register and packed arithmetic on them.
+__device__ __forceinline__ unsigned long long gd_pack(float a, float b) {
+    unsigned long long r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float gd_sum(unsigned long long v) {
+    float a, b;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+    return a + b;
+}
+__device__ __forceinline__ unsigned long long gd_fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ unsigned long long gd_mul2(unsigned long long a, unsigned long long b) {
+    unsigned long long r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
+// Grid (request, head, tile of DVT value channels).  P lanes of a warp share GD_COLS neighbouring columns of S, of which a
+// thread keeps DKP rows each, two rows to a register pair: a token's row values are read from shared memory once for all the
+// thread's columns (the walk is bound by those reads and by the chain sum -> update of one token after another).  The sums
+// u . S that the update waits for go round the lanes at once; the read-outs of four tokens wait and are summed together, each
+// round of shuffles handing half of them over.  Chunks of TC tokens' rows arrive by asynchronous copies a chunk ahead; tokens
+// beyond the portion's end are rows that leave S as it is.
+constexpr int GD_COLS = 2, GD_GROUP = 4, GD_WARPS = 2;
+
+template <int DKP, int P>
+__global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDeltaArgs A, const float* __restrict__ work) {
+    constexpr int CW = 32 / P * GD_COLS, DVT = CW * GD_WARPS, THREADS = 32 * GD_WARPS, PS = DKP + 4, TS = P * PS, V = GD_COLS * GD_GROUP;
     extern __shared__ __align__(16) float sm[];
     pdl_start();
     const int r = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * DVT;
-    const int tid = threadIdx.x, nthreads = blockDim.x;
-    const int part = tid % P, cl = tid / P, col = col0 + cl;
-    const bool col_ok = cl < DVT && col < A.dv;
-    const int pstride = DKP + 4, tstride = P * pstride, dk = A.dk, TC = A.chunk, wrow = gd_work_row(dk, A.dv);
-    // two buffers of a chunk's rows: [r, u, w, a: TC x tstride each][v: TC x DVT][scalars: TC x 4], then the outputs [TC x DVT]
-    const int buf_floats = TC * (4 * tstride + DVT + 4);
+    const int tid = threadIdx.x, lane = tid & 31, part = lane % P, cl = (tid >> 5) * CW + lane / P * GD_COLS, col = col0 + cl;
+    const int dk = A.dk, TC = A.chunk, wrow = gd_work_row(dk, A.dv);
+    // two buffers of a chunk's rows: [r, u, w, a: TC x TS each][v: TC x DVT][kn, r.(a u), r.k: TC x 4], then the outputs [TC x DVT]
+    const int buf_floats = TC * (4 * TS + DVT + 4);
     float* os = sm + 2 * buf_floats;
     const int row0 = A.q_start[r], row1 = A.q_start[r + 1];
+    if (row0 >= row1) return;
     float* st = A.state + (((size_t)A.state_slots[r] * A.H + h) * dk) * A.dv;
-    float S[DKP];
+    unsigned long long S[GD_COLS][DKP / 2];
 #pragma unroll
-    for (int i = 0; i < DKP; ++i) {
-        const int kr = part * DKP + i;
-        S[i] = (col_ok && kr < dk) ? st[(size_t)kr * A.dv + col] : 0.0f;
-    }
-    // key channels beyond dk, written once (the copies never touch them)
-    for (int idx = tid; idx < 2 * TC * P * DKP; idx += nthreads) {
+    for (int c = 0; c < GD_COLS; ++c)
+#pragma unroll
+        for (int i = 0; i < DKP / 2; ++i) {
+            const int kr = part * DKP + 2 * i;
+            const bool ok = col + c < A.dv;
+            S[c][i] = gd_pack(ok && kr < dk ? st[(size_t)kr * A.dv + col + c] : 0.0f, ok && kr + 1 < dk ? st[(size_t)(kr + 1) * A.dv + col + c] : 0.0f);
+        }
+    // the neutral row: r = u = a = 0, w = 1 (key channels beyond dk for good; whole tokens beyond the end in the last chunk)
+    auto neutral = [&](float* base, int tt, int i) {
+        float* at = base + tt * TS + (i / DKP) * PS + i % DKP;
+        at[0] = 0.0f;
+        at[TC * TS] = 0.0f;
+        at[2 * TC * TS] = 1.0f;
+        at[3 * TC * TS] = 0.0f;
+    };
+    for (int idx = tid; idx < 2 * TC * P * DKP; idx += THREADS) {
         const int b = idx / (TC * P * DKP), rest = idx - b * (TC * P * DKP);
         const int tt = rest / (P * DKP), i = rest - tt * (P * DKP);
-        if (i >= dk) {
-            float* base = sm + b * buf_floats + tt * tstride + (i / DKP) * pstride + i % DKP;
-            base[0] = 0.0f;
-            base[TC * tstride] = 0.0f;
-            base[2 * TC * tstride] = 1.0f;
-            base[3 * TC * tstride] = 0.0f;
-        }
+        if (i >= dk) neutral(sm + b * buf_floats, tt, i);
     }
     const bool wide = (dk & 3) == 0;
-    const int piece = wide ? 4 : 1, pieces = dk / piece;
     auto fetch = [&](int c0, int b) {
         const int tc = min(TC, row1 - c0);
         float* base = sm + b * buf_floats;
-        float* vs = base + 4 * TC * tstride;
+        float* vs = base + 4 * TC * TS;
         float* sc = vs + TC * DVT;
-        for (int idx = tid; idx < tc * pieces; idx += nthreads) {
-            const int tt = idx / pieces, i = (idx - tt * pieces) * piece;
-            const float* w = work + ((size_t)(c0 + tt) * A.H + h) * wrow + i;
-            float* at = base + tt * tstride + (i / DKP) * pstride + i % DKP;
-            gd_copy(at, w, 4 * piece);
-            gd_copy(at + TC * tstride, w + dk, 4 * piece);
-            gd_copy(at + 2 * TC * tstride, w + 2 * dk, 4 * piece);
-            gd_copy(at + 3 * TC * tstride, w + 3 * dk, 4 * piece);
+        for (int tt = 0; tt < tc; ++tt) {
+            const float* w = work + ((size_t)(c0 + tt) * A.H + h) * wrow;
+            float* at = base + tt * TS;
+            if (wide) {
+                for (int i = tid * 4; i < dk; i += THREADS * 4) {
+                    float* to = at + (i / DKP) * PS + i % DKP;
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) gd_copy(to + k * TC * TS, w + k * dk + i, 16);
+                }
+            } else {
+                for (int i = tid; i < dk; i += THREADS) {
+                    float* to = at + (i / DKP) * PS + i % DKP;
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) gd_copy(to + k * TC * TS, w + k * dk + i, 4);
+                }
+            }
+            for (int j = tid; j < DVT; j += THREADS)
+                if (col0 + j < A.dv) gd_copy(vs + tt * DVT + j, w + 4 * dk + col0 + j, 4);
+            if (tid < 3) gd_copy(sc + tt * 4 + tid, w + 4 * dk + A.dv + tid, 4);
         }
-        for (int idx = tid; idx < tc * DVT; idx += nthreads) {
-            const int tt = idx / DVT, j = idx - tt * DVT, c = col0 + j;
-            if (c < A.dv) gd_copy(vs + idx, work + ((size_t)(c0 + tt) * A.H + h) * wrow + 4 * dk + c, 4);
-        }
-        for (int idx = tid; idx < 3 * tc; idx += nthreads) {
-            const int tt = idx / 3, j = idx - tt * 3;
-            gd_copy(sc + tt * 4 + j, work + ((size_t)(c0 + tt) * A.H + h) * wrow + 4 * dk + A.dv + j, 4);
-        }
+        for (int idx = tid; idx < (TC - tc) * P * DKP; idx += THREADS) neutral(base, tc + idx / (P * DKP), idx % (P * DKP));
+        for (int idx = tc * DVT + tid; idx < TC * DVT; idx += THREADS) vs[idx] = 0.0f;
+        for (int idx = tc * 4 + tid; idx < TC * 4; idx += THREADS) sc[idx] = 0.0f;
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    if (row0 < row1) fetch(row0, 0);
+    fetch(row0, 0);
     int b = 0;
     for (int c0 = row0; c0 < row1; c0 += TC, b ^= 1) {
         const int tc = min(TC, row1 - c0);
@@ -268,87 +306,118 @@ __global__ void __launch_bounds__(128) general_delta_walk_kernel(GDeltaArgs A, c
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();                           // everybody's copies of this chunk have landed; the outputs before are stored
-        const float* base = sm + b * buf_floats;
-        const float* vs = base + 4 * TC * tstride;
+        const float* mine = sm + b * buf_floats + part * PS;
+        const float* vs = sm + b * buf_floats + 4 * TC * TS;
         const float* sc = vs + TC * DVT;
-        if (cl < DVT) {
-            // the rows of the token after this one are read while this one's sums run; two register sets take turns
-            struct Rows { float4 r[DKP / 4], u[DKP / 4], w[DKP / 4], a[DKP / 4]; float kn, ra, rk, v; };
-            const float* mine = base + part * pstride;
-            auto read = [&](Rows& x, int tt) {
-                const float* at = mine + tt * tstride;
+        for (int g = 0; g < tc; g += GD_GROUP) {
+            float q[V];
 #pragma unroll
-                for (int i = 0; i < DKP / 4; ++i) {
-                    x.r[i] = reinterpret_cast<const float4*>(at)[i];
-                    x.u[i] = reinterpret_cast<const float4*>(at + TC * tstride)[i];
-                    x.w[i] = reinterpret_cast<const float4*>(at + 2 * TC * tstride)[i];
-                    x.a[i] = reinterpret_cast<const float4*>(at + 3 * TC * tstride)[i];
-                }
-                x.kn = sc[4 * tt];
-                x.ra = sc[4 * tt + 1];
-                x.rk = sc[4 * tt + 2];
-                x.v = col_ok ? vs[tt * DVT + cl] : 0.0f;
-            };
-            auto token = [&](const Rows& x, Rows& next, int tt) {
-                if (tt + 1 < tc) read(next, tt + 1);
-                float p0 = 0.0f, p1 = 0.0f, p2 = 0.0f, p3 = 0.0f, q0 = 0.0f, q1 = 0.0f, q2 = 0.0f, q3 = 0.0f;
+            for (int k = 0; k < GD_GROUP; ++k) {
+                const int tt = g + k;
+                const float4 s4 = *reinterpret_cast<const float4*>(sc + tt * 4);
+                const float2 v2 = *reinterpret_cast<const float2*>(vs + tt * DVT + cl);
+                const float v[GD_COLS] = {col < A.dv ? v2.x : 0.0f, col + 1 < A.dv ? v2.y : 0.0f};
+                unsigned long long u[DKP / 2], w[DKP / 2], rv[DKP / 2], av[DKP / 2];
+                auto read = [&](unsigned long long (&x)[DKP / 2], int which) {
 #pragma unroll
-                for (int i = 0; i < DKP / 4; ++i) {
-                    p0 = fmaf(S[4 * i], x.u[i].x, p0);
-                    p1 = fmaf(S[4 * i + 1], x.u[i].y, p1);
-                    p2 = fmaf(S[4 * i + 2], x.u[i].z, p2);
-                    p3 = fmaf(S[4 * i + 3], x.u[i].w, p3);
-                    S[4 * i] *= x.w[i].x; S[4 * i + 1] *= x.w[i].y; S[4 * i + 2] *= x.w[i].z; S[4 * i + 3] *= x.w[i].w;
-                    q0 = fmaf(S[4 * i], x.r[i].x, q0);
-                    q1 = fmaf(S[4 * i + 1], x.r[i].y, q1);
-                    q2 = fmaf(S[4 * i + 2], x.r[i].z, q2);
-                    q3 = fmaf(S[4 * i + 3], x.r[i].w, q3);
-                }
-                float p = (p0 + p1) + (p2 + p3), q = (q0 + q1) + (q2 + q3);
-#pragma unroll
-                for (int o = 1; o < 32; o <<= 1) {
-                    if (o < P) {
-                        p += __shfl_xor_sync(0xffffffffu, p, o);
-                        q += __shfl_xor_sync(0xffffffffu, q, o);
+                    for (int i = 0; i < DKP / 4; ++i) {
+                        const float4 f = reinterpret_cast<const float4*>(mine + which * TC * TS + tt * TS)[i];
+                        x[2 * i] = gd_pack(f.x, f.y);
+                        x[2 * i + 1] = gd_pack(f.z, f.w);
                     }
-                }
-                const float knv = x.kn * x.v;
+                };
+                read(u, 1);
+                read(w, 2);
+                read(rv, 0);
+                read(av, 3);
+                float p[GD_COLS];
 #pragma unroll
-                for (int i = 0; i < DKP / 4; ++i) {
-                    S[4 * i] = fmaf(x.u[i].x, fmaf(-x.a[i].x, p, knv), S[4 * i]);
-                    S[4 * i + 1] = fmaf(x.u[i].y, fmaf(-x.a[i].y, p, knv), S[4 * i + 1]);
-                    S[4 * i + 2] = fmaf(x.u[i].z, fmaf(-x.a[i].z, p, knv), S[4 * i + 2]);
-                    S[4 * i + 3] = fmaf(x.u[i].w, fmaf(-x.a[i].w, p, knv), S[4 * i + 3]);
+                for (int c = 0; c < GD_COLS; ++c) {
+                    unsigned long long x = gd_mul2(S[c][0], u[0]), y = gd_mul2(S[c][1], u[1]);
+#pragma unroll
+                    for (int i = 2; i < DKP / 2; i += 2) { x = gd_fma2(S[c][i], u[i], x); y = gd_fma2(S[c][i + 1], u[i + 1], y); }
+                    p[c] = gd_sum(x) + gd_sum(y);
                 }
-                if (part == 0) os[tt * DVT + cl] = fmaf(x.rk, x.v, fmaf(-x.ra, p, q));
-            };
-            Rows even, odd;
-            read(even, 0);
-            for (int tt = 0; tt < tc; tt += 2) {
-                token(even, odd, tt);
-                if (tt + 1 < tc) token(odd, even, tt + 1);
+#pragma unroll
+                for (int o = 1; o < P; o <<= 1)
+#pragma unroll
+                    for (int c = 0; c < GD_COLS; ++c) p[c] += __shfl_xor_sync(0xffffffffu, p[c], o);
+#pragma unroll
+                for (int c = 0; c < GD_COLS; ++c) {
+                    unsigned long long x = gd_pack(0.0f, 0.0f), y = x;
+#pragma unroll
+                    for (int i = 0; i < DKP / 2; i += 2) {
+                        S[c][i] = gd_mul2(S[c][i], w[i]);
+                        S[c][i + 1] = gd_mul2(S[c][i + 1], w[i + 1]);
+                        x = gd_fma2(S[c][i], rv[i], x);
+                        y = gd_fma2(S[c][i + 1], rv[i + 1], y);
+                    }
+                    // the token's own terms join the sum in one of the lanes
+                    q[k * GD_COLS + c] = gd_sum(x) + gd_sum(y) + (part == 0 ? fmaf(s4.z, v[c], -s4.y * p[c]) : 0.0f);
+                    const unsigned long long mp = gd_pack(-p[c], -p[c]), kv = gd_pack(s4.x * v[c], s4.x * v[c]);
+#pragma unroll
+                    for (int i = 0; i < DKP / 2; ++i) S[c][i] = gd_fma2(u[i], gd_fma2(av[i], mp, kv), S[c][i]);
+                }
+            }
+            // V sums over P lanes: halve the values while there are several, then add up what is left
+            int first = 0;                          // which of the V values this lane's first one is
+            constexpr int ROUNDS_DEALT = P >= V ? V : P;
+            int left = V;
+#pragma unroll
+            for (int o = 1; o < ROUNDS_DEALT; o <<= 1) {
+                const bool upper = part & o;
+                left >>= 1;
+#pragma unroll
+                for (int i = 0; i < V / 2; ++i)
+                    if (i < left) {
+                        const float keep = upper ? q[i + left] : q[i], give = upper ? q[i] : q[i + left];
+                        q[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+                    }
+                if (upper) first += left;
+            }
+#pragma unroll
+            for (int o = ROUNDS_DEALT; o < P; o <<= 1) q[0] += __shfl_xor_sync(0xffffffffu, q[0], o);
+            constexpr int EACH = V / ROUNDS_DEALT;
+            if (part < ROUNDS_DEALT) {
+#pragma unroll
+                for (int i = 0; i < EACH; ++i) {
+                    const int which = first + i;
+                    os[(g + which / GD_COLS) * DVT + cl + which % GD_COLS] = q[i];
+                }
             }
         }
         __syncthreads();
-        for (int idx = tid; idx < tc * DVT; idx += nthreads) {
+        for (int idx = tid; idx < tc * DVT; idx += THREADS) {
             const int tt = idx / DVT, j = idx - tt * DVT, c = col0 + j;
             if (c < A.dv) A.out[(size_t)(c0 + tt) * A.ldo + h * A.dv + c] = os[idx];
         }
     }
 #pragma unroll
-    for (int i = 0; i < DKP; ++i) {
-        const int kr = part * DKP + i;
-        if (col_ok && kr < dk) st[(size_t)kr * A.dv + col] = S[i];
-    }
+    for (int c = 0; c < GD_COLS; ++c)
+#pragma unroll
+        for (int i = 0; i < DKP / 2; ++i) {
+            const int kr = part * DKP + 2 * i;
+            float x, y;
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(S[c][i]));
+            if (col + c < A.dv && kr < dk) st[(size_t)kr * A.dv + col + c] = x;
+            if (col + c < A.dv && kr + 1 < dk) st[(size_t)(kr + 1) * A.dv + col + c] = y;
+        }
 }
 
-constexpr int GD_WALK_SMEM = 80 * 1024;
+constexpr int GD_WALK_SMEM = 100 * 1024;
 
-template <int DKP>
-static int launch_gd_walk(const GDeltaArgs& A, dim3 grid, int threads, size_t bytes, const float* work, int P, int dvt, cudaStream_t s) {
+template <int DKP, int P>
+static int launch_gd_walk(GDeltaArgs A, int n_reqs, const float* work, cudaStream_t s) {
+    constexpr int DVT = 32 / P * GD_COLS * GD_WARPS;
+    auto bytes = [&](int tc) { return (size_t)tc * (2 * (4 * P * (DKP + 4) + DVT + 4) + DVT) * sizeof(float); };
+    int chunk = 16;
+    while (chunk > GD_GROUP && bytes(chunk) > GD_WALK_SMEM) chunk >>= 1;
+    if (bytes(chunk) > GD_WALK_SMEM) return VCB_ERR_UNSUPPORTED;
     static unsigned long long configured = 0;
-    if (int e = vcb_allow_dynamic_smem(general_delta_walk_kernel<DKP>, GD_WALK_SMEM, &configured)) return e;
-    vcb_launch(general_delta_walk_kernel<DKP>, grid, threads, bytes, s, A, work, P, dvt);
+    if (int e = vcb_allow_dynamic_smem(general_delta_walk_kernel<DKP, P>, GD_WALK_SMEM, &configured)) return e;
+    A.chunk = chunk;
+    dim3 grid(n_reqs, A.H, (A.dv + DVT - 1) / DVT);
+    vcb_launch(general_delta_walk_kernel<DKP, P>, grid, 32 * GD_WARPS, bytes(chunk), s, A, work);
     return vcb_last_error();
 }
 
@@ -374,23 +443,17 @@ static int launch_gd_scan(const GDeltaArgs& A, int n_reqs, cudaStream_t s) {
 
 template <typename T>
 static int launch_gd_portions(const GDeltaArgs& A, int n_reqs, int n_tokens, float* work, cudaStream_t s) {
-    const int dkp = A.dk > 256 ? 16 : 8;
-    int P = 1;
-    while (P * dkp < A.dk) P <<= 1;
-    const int dvt = 128 / P >= 32 ? 32 : 128 / P;
-    int chunk = 16;
-    auto bytes = [&](int tc) { return (size_t)tc * (2 * (4 * P * (dkp + 4) + dvt + 4) + dvt) * sizeof(float); };
-    while (chunk > 4 && bytes(chunk) > GD_WALK_SMEM) chunk >>= 1;
-    if (P > 32 || bytes(chunk) > GD_WALK_SMEM) return launch_gd_scan<T>(A, n_reqs, s);     // very long keys: the kernel above
+    if (A.dk > 512) return launch_gd_scan<T>(A, n_reqs, s);     // very long keys: the kernel above
     const long long items = (long long)n_tokens * A.H;
     vcb_launch(general_delta_prepare_kernel<T>, dim3((unsigned)((items + 3) / 4)), 128, 0, s, A, work, n_tokens);
     if (int e = vcb_last_error()) return e;
-    GDeltaArgs B = A;
-    B.chunk = chunk;
-    dim3 grid(n_reqs, A.H, (A.dv + dvt - 1) / dvt);
-    const int threads = dvt * P;
-    if (dkp == 8) return launch_gd_walk<8>(B, grid, threads, bytes(chunk), work, P, dvt, s);
-    return launch_gd_walk<16>(B, grid, threads, bytes(chunk), work, P, dvt, s);
+    if (A.dk <= 8) return launch_gd_walk<8, 1>(A, n_reqs, work, s);
+    if (A.dk <= 16) return launch_gd_walk<8, 2>(A, n_reqs, work, s);
+    if (A.dk <= 32) return launch_gd_walk<8, 4>(A, n_reqs, work, s);
+    if (A.dk <= 64) return launch_gd_walk<8, 8>(A, n_reqs, work, s);
+    if (A.dk <= 128) return launch_gd_walk<8, 16>(A, n_reqs, work, s);
+    if (A.dk <= 256) return launch_gd_walk<8, 32>(A, n_reqs, work, s);
+    return launch_gd_walk<16, 32>(A, n_reqs, work, s);
 }
 
 VCB_EXPORT int vcb_general_delta(const void* r, long long ldr, const void* k, long long ldk, const void* v, long long ldv,

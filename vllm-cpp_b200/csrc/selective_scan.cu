@@ -102,19 +102,59 @@ __global__ void __launch_bounds__(128) selective_step_kernel(SelectiveArgs a, in
     if (part == 0) ((T*)a.out)[row * a.ldo + c] = from_f32<T>(fmaf(dc, x, y) * ss_silu(z));
 }
 
-// Grid (tiles of CB channels, requests), CB * L threads.  TC tokens of a chunk; CB, L and TC are such that a thread stages
-// PER values of each kind: TC * CB = PER * threads for the channels' values.
+// Two floats to a 64-bit register and packed arithmetic on them.
+__device__ __forceinline__ unsigned long long ss_pack(float a, float b) {
+    unsigned long long r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ void ss_unpack(unsigned long long v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ unsigned long long ss_fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ unsigned long long ss_mul2(unsigned long long a, unsigned long long b) {
+    unsigned long long r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
+// v[k], k = 0 .. L - 1: every lane's share of the sum of token k over the L lanes of a channel.  Returns, in lane `part`, the
+// whole sum of token `part`: each round a lane keeps the half of its tokens that matches its bit and hands over the other.
+template <int L>
+__device__ __forceinline__ float ss_deal_sums(float (&v)[L], int part) {
+#pragma unroll
+    for (int half = L / 2; half > 0; half >>= 1) {
+        const bool upper = part & half;
+#pragma unroll
+        for (int k = 0; k < half; ++k) {
+            const float keep = upper ? v[k + half] : v[k], give = upper ? v[k] : v[k + half];
+            v[k] = keep + __shfl_xor_sync(0xffffffffu, give, half);
+        }
+    }
+    return v[0];
+}
+
+// Grid (tiles of CB channels, requests), CB * L threads; chunks of TC tokens.  Tokens beyond the portion's end are staged as
+// dt = 0 and dx = 0, which leave the state as it is, so a chunk is always walked whole.  L tokens are walked together: their
+// read-outs are independent of one another, and their sums over a channel's lanes are dealt out one token to a lane.
 template <typename T, int NPT, int L, int CB, int TC>
 __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a) {
     constexpr int THREADS = CB * L, PER = (TC * CB + THREADS - 1) / THREADS, NP = L * NPT, PERN = (TC * NP + THREADS - 1) / THREADS;
-    __shared__ __align__(16) float dts[TC][CB], dxs[TC][CB], ys[TC][CB + 1];
+    constexpr int GROUP = (L <= TC) ? L : 1;                  // tokens walked together
+    __shared__ __align__(16) float2 dts[TC][CB];              // dt, dt * x
     __shared__ __align__(16) float bs[TC][NP], cs[TC][NP];
+    __shared__ float ys[TC][CB + 1];
     const int tid = threadIdx.x, part = tid % L, cl = tid / L, c0 = blockIdx.x * CB;
     const int c = min(c0 + cl, a.I - 1), n0 = part * NPT;
     const bool there = c0 + cl < a.I, quads = (a.N & 3) == 0;
-    float A[NPT], S[NPT];
-    ss_load<NPT>(a.a2 + (size_t)c * a.N, n0, a.N, quads, A);
-    const int sc = tid % CB, st0 = tid / CB;                 // staging: channel sc, tokens st0, st0 + L, ...
+    float S[NPT];
+    unsigned long long A2[NPT / 2], S2[NPT / 2];
+    ss_load<NPT>(a.a2 + (size_t)c * a.N, n0, a.N, quads, S);
+#pragma unroll
+    for (int i = 0; i < NPT / 2; ++i) A2[i] = ss_pack(S[2 * i], S[2 * i + 1]);
+    const int sc = tid % CB, st0 = tid / CB;                  // staging: channel sc, tokens st0, st0 + L, ...
     const int scc = min(c0 + sc, a.I - 1);
     const float bias = a.dt_bias[scc], dc = a.d[scc];
     pdl_start();
@@ -123,27 +163,29 @@ __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a)
     if (len <= 0) return;
     float* st = a.state + ((size_t)a.state_slots[r] * a.I + c) * a.N;
     ss_load<NPT>(st, n0, a.N, quads, S);
+#pragma unroll
+    for (int i = 0; i < NPT / 2; ++i) S2[i] = ss_pack(S[2 * i], S[2 * i + 1]);
     const T* xp = (const T*)a.x + (size_t)row0 * a.ldx + scc;
     const T* dp = (const T*)a.dt_pre + (size_t)row0 * a.lddt + scc;
     const T* zp = (const T*)a.z + (size_t)row0 * a.ldz + scc;
     const T* bp = (const T*)a.b + (size_t)row0 * a.ldb;
     const T* cp = (const T*)a.c + (size_t)row0 * a.ldc;
     T* op = (T*)a.out + (size_t)row0 * a.ldo + scc;
-    float px[PER], pd[PER], pz[PER], pb[PERN], pc[PERN];     // the values of a chunk on their way
+    T px[PER], pd[PER], pz[PER], pb[PERN], pc[PERN];          // a chunk's values on their way, as they are stored
     auto fetch = [&](int t0) {
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
-            const int t = st0 + k * L, tt = min(t0 + t, len - 1);
-            px[k] = to_f32<T>(xp[(size_t)tt * a.ldx]);
-            pd[k] = to_f32<T>(dp[(size_t)tt * a.lddt]);
-            pz[k] = to_f32<T>(zp[(size_t)tt * a.ldz]);
+            const size_t tt = min(t0 + st0 + k * L, len - 1);
+            px[k] = xp[tt * a.ldx];
+            pd[k] = dp[tt * a.lddt];
+            pz[k] = zp[tt * a.ldz];
         }
 #pragma unroll
         for (int k = 0; k < PERN; ++k) {
-            const int idx = tid + k * THREADS, t = idx / NP, n = idx - t * NP, tt = min(t0 + t, len - 1);
-            const bool in = n < a.N && t < TC;
-            pb[k] = in ? to_f32<T>(bp[(size_t)tt * a.ldb + n]) : 0.0f;
-            pc[k] = in ? to_f32<T>(cp[(size_t)tt * a.ldc + n]) : 0.0f;
+            const int idx = tid + k * THREADS, t = idx / NP, n = min(idx - t * NP, a.N - 1);
+            const size_t tt = min(t0 + t, len - 1);
+            pb[k] = bp[tt * a.ldb + n];
+            pc[k] = cp[tt * a.ldc + n];
         }
     };
     fetch(0);
@@ -153,40 +195,54 @@ __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a)
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
             const int t = st0 + k * L;
+            xk[k] = to_f32<T>(px[k]);
+            zk[k] = to_f32<T>(pz[k]);
             if (t < TC) {
-                const float dt = ss_softplus(pd[k] + bias);
-                dts[t][sc] = dt;
-                dxs[t][sc] = dt * px[k];
+                const float dt = t < tc ? ss_softplus(to_f32<T>(pd[k]) + bias) : 0.0f;
+                dts[t][sc] = make_float2(dt, dt * xk[k]);
             }
-            zk[k] = pz[k];
-            xk[k] = px[k];
         }
 #pragma unroll
         for (int k = 0; k < PERN; ++k) {
             const int idx = tid + k * THREADS, t = idx / NP, n = idx - t * NP;
-            if (t < TC) { bs[t][n] = pb[k]; cs[t][n] = pc[k]; }
+            if (t < TC) {
+                bs[t][n] = n < a.N ? to_f32<T>(pb[k]) : 0.0f;
+                cs[t][n] = n < a.N ? to_f32<T>(pc[k]) : 0.0f;
+            }
         }
         __syncthreads();
         if (t0 + TC < len) fetch(t0 + TC);
-#pragma unroll 4
-        for (int t = 0; t < tc; ++t) {
-            const float dt = dts[t][cl], dx = dxs[t][cl];
-            float y = 0.0f;
 #pragma unroll
-            for (int i = 0; i < NPT; i += 4) {
-                const float4 b4 = *reinterpret_cast<const float4*>(&bs[t][n0 + i]), c4 = *reinterpret_cast<const float4*>(&cs[t][n0 + i]);
-                S[i] = fmaf(ss_exp2(dt * A[i]), S[i], dx * b4.x);
-                S[i + 1] = fmaf(ss_exp2(dt * A[i + 1]), S[i + 1], dx * b4.y);
-                S[i + 2] = fmaf(ss_exp2(dt * A[i + 2]), S[i + 2], dx * b4.z);
-                S[i + 3] = fmaf(ss_exp2(dt * A[i + 3]), S[i + 3], dx * b4.w);
-                y = fmaf(S[i], c4.x, y);
-                y = fmaf(S[i + 1], c4.y, y);
-                y = fmaf(S[i + 2], c4.z, y);
-                y = fmaf(S[i + 3], c4.w, y);
+        for (int g = 0; g < TC; g += GROUP) {
+            float y[GROUP];
+#pragma unroll
+            for (int k = 0; k < GROUP; ++k) {
+                const float2 d = dts[g + k][cl];
+                const unsigned long long dt2 = ss_pack(d.x, d.x), dx2 = ss_pack(d.y, d.y);
+                unsigned long long y2 = ss_pack(0.0f, 0.0f);
+#pragma unroll
+                for (int i = 0; i < NPT / 4; ++i) {
+                    const float4 b4 = *reinterpret_cast<const float4*>(&bs[g + k][n0 + 4 * i]), c4 = *reinterpret_cast<const float4*>(&cs[g + k][n0 + 4 * i]);
+                    float e0, e1, e2, e3;
+                    ss_unpack(ss_mul2(dt2, A2[2 * i]), e0, e1);
+                    ss_unpack(ss_mul2(dt2, A2[2 * i + 1]), e2, e3);
+                    S2[2 * i] = ss_fma2(ss_pack(ss_exp2(e0), ss_exp2(e1)), S2[2 * i], ss_mul2(dx2, ss_pack(b4.x, b4.y)));
+                    S2[2 * i + 1] = ss_fma2(ss_pack(ss_exp2(e2), ss_exp2(e3)), S2[2 * i + 1], ss_mul2(dx2, ss_pack(b4.z, b4.w)));
+                    y2 = ss_fma2(S2[2 * i], ss_pack(c4.x, c4.y), y2);
+                    y2 = ss_fma2(S2[2 * i + 1], ss_pack(c4.z, c4.w), y2);
+                }
+                float u, v;
+                ss_unpack(y2, u, v);
+                y[k] = u + v;
             }
+            if constexpr (GROUP == L) {
+                ys[g + part][cl] = ss_deal_sums<L>(y, part);
+            } else {
+                float v = y[0];
 #pragma unroll
-            for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (part == 0) ys[t][cl] = y;
+                for (int o = 1; o < L; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+                if (part == 0) ys[g][cl] = v;
+            }
         }
         __syncthreads();
 #pragma unroll
@@ -196,6 +252,8 @@ __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a)
         }
         // ys is written again only after the next chunk's first barrier
     }
+#pragma unroll
+    for (int i = 0; i < NPT / 2; ++i) ss_unpack(S2[i], S[2 * i], S[2 * i + 1]);
     if (there) ss_store<NPT>(st, n0, a.N, quads, S);
 }
 
