@@ -12,9 +12,9 @@
 // so a token costs one round of shuffles for two sums.
 //
 //   general_delta_scan_kernel      steps of single tokens and short portions: inputs made and walked in one kernel
-//   general_delta_prepare_kernel   steps with portions: per token and head a row of floats [r | u | w | a | v | kn, r.(a u), r.k, 0]
+//   general_delta_prepare_kernel   steps with portions: per token and head a row of floats [r | u | w | a | kn, r.(a u), r.k, 0 | v]
 //   general_delta_walk_kernel      the walk over the tokens, whose rows arrive by asynchronous copies a chunk ahead
-#include "common.cuh"
+#include "fast_math.cuh"
 
 struct GDeltaArgs {
     const void* r;              // [n, H * dk] rows of T
@@ -35,11 +35,21 @@ struct GDeltaArgs {
     int chunk;                  // tokens staged in shared memory at a time
 };
 
-__device__ __forceinline__ float gd_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+// One or two neighbouring elements of a row.
+template <typename T, int VW> __device__ __forceinline__ void gd_load(const T* p, float (&v)[VW]) {
+    if constexpr (VW == 2 && sizeof(T) == 2) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+        v[0] = f.x;
+        v[1] = f.y;
+    } else {
+#pragma unroll
+        for (int e = 0; e < VW; ++e) v[e] = to_f32<T>(p[e]);
+    }
+}
 
-// A warp makes one token's inputs of one head: calls put(i, r, u, w, a) for its channels i (lane, lane + 32, ...) and returns
-// the three sums to every lane.
-template <typename T, typename Put>
+// A warp makes one token's inputs of one head: calls put(i, r, u, w, a) for its channels i (VW neighbours at a time, from
+// VW * lane on) and returns the three sums to every lane.
+template <typename T, int VW, typename Put>
 __device__ __forceinline__ void gd_inputs(const GDeltaArgs& A, size_t row, int h, int lane, Put put, float& kn, float& ra, float& rk) {
     const T* rp = (const T*)A.r + row * A.ldr + h * A.dk;
     const T* kp = (const T*)A.k + row * A.ldk + h * A.dk;
@@ -48,20 +58,37 @@ __device__ __forceinline__ void gd_inputs(const GDeltaArgs& A, size_t row, int h
     const float* ab = A.a_bias ? A.a_bias + h * A.dk : nullptr;
     const float* zb = A.z_bias ? A.z_bias + h * A.dk : nullptr;
     float ss = 0.0f;
-    for (int i = lane; i < A.dk; i += 32) { const float x = to_f32<T>(kp[i]); ss = fmaf(x, x, ss); }
+    for (int i = lane * VW; i < A.dk; i += 32 * VW) {
+        float x[VW];
+        gd_load<T, VW>(kp + i, x);
+#pragma unroll
+        for (int e = 0; e < VW; ++e) ss = fmaf(x[e], x[e], ss);
+    }
     kn = sqrtf(warp_sum(ss) + A.unit_eps);
-    const float inv = 1.0f / kn;
+    const float inv = 1.0f / kn, rate2 = -A.rate * FM_LOG2E;
     float sa = 0.0f, sk = 0.0f;
-    for (int i = lane; i < A.dk; i += 32) {
-        const float x = to_f32<T>(kp[i]), r = to_f32<T>(rp[i]), u = x * inv;
-        const float a = gd_sigmoid(to_f32<T>(ap[i]) + (ab ? ab[i] : 0.0f));
-        const float w = expf(-A.rate * gd_sigmoid(to_f32<T>(zp[i]) + (zb ? zb[i] : 0.0f)));
-        sa = fmaf(r, a * u, sa);
-        sk = fmaf(r, x, sk);
-        put(i, r, u, w, a);
+    for (int i = lane * VW; i < A.dk; i += 32 * VW) {
+        float x[VW], r[VW], a[VW], z[VW];
+        gd_load<T, VW>(kp + i, x);
+        gd_load<T, VW>(rp + i, r);
+        gd_load<T, VW>(ap + i, a);
+        gd_load<T, VW>(zp + i, z);
+#pragma unroll
+        for (int e = 0; e < VW; ++e) {
+            const float u = x[e] * inv, av = fm_sigmoid(a[e] + (ab ? ab[i + e] : 0.0f));
+            const float w = fm_ex2(rate2 * fm_sigmoid(z[e] + (zb ? zb[i + e] : 0.0f)));
+            sa = fmaf(r[e], av * u, sa);
+            sk = fmaf(r[e], x[e], sk);
+            put(i + e, r[e], u, w, av);
+        }
     }
     ra = warp_sum(sa);
     rk = warp_sum(sk);
+}
+
+// Pairs of channels may be read together: even head sizes and strides, aligned rows.
+static bool gd_pairs(const GDeltaArgs& A) {
+    return !(A.dk & 1) && !((A.ldr | A.ldk | A.lda | A.ldz) & 1) && !(((uintptr_t)A.r | (uintptr_t)A.k | (uintptr_t)A.a_pre | (uintptr_t)A.z) & 3);
 }
 
 // Grid (request, head, tile of DVT value channels).  A thread keeps DKP rows of one column of S in registers; the P threads
@@ -103,7 +130,7 @@ __global__ void general_delta_scan_kernel(GDeltaArgs A, int P, int DVT) {
         __syncthreads();                          // the chunk before has been read
         for (int tt = warp; tt < tc; tt += nwarps) {
             float kn, ra, rk;
-            gd_inputs<T>(A, (size_t)(c0 + tt), h, lane, [&](int i, float rv, float u, float w, float a) {
+            gd_inputs<T, 1>(A, (size_t)(c0 + tt), h, lane, [&](int i, float rv, float u, float w, float a) {
                 const int at = tt * tstride + (i / DKP) * pstride + i % DKP;
                 rs[at] = rv;
                 us[at] = u;
@@ -168,56 +195,37 @@ __global__ void general_delta_scan_kernel(GDeltaArgs A, int P, int DVT) {
     }
 }
 
-// Floats of a (token, head) row of the prepared inputs, a multiple of 4 (ops.py has the same formula).
-__host__ __device__ static inline int gd_work_row(int dk, int dv) { return (4 * dk + dv + 4 + 3) / 4 * 4; }
+// A (token, head) row of the prepared inputs: r, u, w and a of dk channels each, padded to a multiple of 4 by channels that do
+// nothing, then kn, r.(a u), r.k, 0, then v, padded.  Its size in floats (ops.py has the same formula).
+__host__ __device__ static inline int gd_pad4(int n) { return (n + 3) / 4 * 4; }
+__host__ __device__ static inline int gd_work_row(int dk, int dv) { return 4 * gd_pad4(dk) + 4 + gd_pad4(dv); }
 
-template <typename T>
+template <typename T, int VW>
 __global__ void __launch_bounds__(128) general_delta_prepare_kernel(GDeltaArgs A, float* __restrict__ work, int n) {
     pdl_start();
     const int lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
     if (item >= (long long)n * A.H) return;
-    const size_t row = (size_t)(item / A.H);
-    const int h = (int)(item % A.H), dk = A.dk;
+    const int row = (int)(item / A.H), h = (int)(item - (long long)row * A.H), dk = A.dk, d4 = gd_pad4(dk);
     float* w = work + (size_t)item * gd_work_row(dk, A.dv);
     float kn, ra, rk;
-    gd_inputs<T>(A, row, h, lane, [&](int i, float rv, float u, float wv, float a) {
+    gd_inputs<T, VW>(A, (size_t)row, h, lane, [&](int i, float rv, float u, float wv, float a) {
         w[i] = rv;
-        w[dk + i] = u;
-        w[2 * dk + i] = wv;
-        w[3 * dk + i] = a;
+        w[d4 + i] = u;
+        w[2 * d4 + i] = wv;
+        w[3 * d4 + i] = a;
     }, kn, ra, rk);
-    const T* vp = (const T*)A.v + row * A.ldv + h * A.dv;
-    for (int i = lane; i < A.dv; i += 32) w[4 * dk + i] = to_f32<T>(vp[i]);
-    if (lane < 4) w[4 * dk + A.dv + lane] = lane == 0 ? kn : lane == 1 ? ra : lane == 2 ? rk : 0.0f;
+    if (lane < d4 - dk) {
+        w[dk + lane] = w[d4 + dk + lane] = w[3 * d4 + dk + lane] = 0.0f;
+        w[2 * d4 + dk + lane] = 1.0f;
+    }
+    if (lane < 4) w[4 * d4 + lane] = lane == 0 ? kn : lane == 1 ? ra : lane == 2 ? rk : 0.0f;
+    const T* vp = (const T*)A.v + (size_t)row * A.ldv + h * A.dv;
+    for (int i = lane; i < gd_pad4(A.dv); i += 32) w[4 * d4 + 4 + i] = i < A.dv ? to_f32<T>(vp[i]) : 0.0f;
 }
 
-__device__ __forceinline__ void gd_copy(float* smem, const float* gmem, int bytes) {
-    const uint32_t dst = (uint32_t)__cvta_generic_to_shared(smem);
-    if (bytes == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(gmem) : "memory");
-    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(gmem) : "memory");
-}
-
-// Two floats to a 64-bit register and packed arithmetic on them.
-__device__ __forceinline__ unsigned long long gd_pack(float a, float b) {
-    unsigned long long r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-    return r;
-}
-__device__ __forceinline__ float gd_sum(unsigned long long v) {
-    float a, b;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
-    return a + b;
-}
-__device__ __forceinline__ unsigned long long gd_fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
-    unsigned long long r;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-    return r;
-}
-__device__ __forceinline__ unsigned long long gd_mul2(unsigned long long a, unsigned long long b) {
-    unsigned long long r;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-    return r;
+__device__ __forceinline__ void gd_copy16(uint32_t dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
 
 // Grid (request, head, tile of DVT value channels).  P lanes of a warp share GD_COLS neighbouring columns of S, of which a
@@ -242,16 +250,17 @@ __global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDelt
     const int row0 = A.q_start[r], row1 = A.q_start[r + 1];
     if (row0 >= row1) return;
     float* st = A.state + (((size_t)A.state_slots[r] * A.H + h) * dk) * A.dv;
-    unsigned long long S[GD_COLS][DKP / 2];
+    f32x2 S[GD_COLS][DKP / 2];
 #pragma unroll
     for (int c = 0; c < GD_COLS; ++c)
 #pragma unroll
         for (int i = 0; i < DKP / 2; ++i) {
             const int kr = part * DKP + 2 * i;
             const bool ok = col + c < A.dv;
-            S[c][i] = gd_pack(ok && kr < dk ? st[(size_t)kr * A.dv + col + c] : 0.0f, ok && kr + 1 < dk ? st[(size_t)(kr + 1) * A.dv + col + c] : 0.0f);
+            S[c][i] = pack2f(ok && kr < dk ? st[(size_t)kr * A.dv + col + c] : 0.0f, ok && kr + 1 < dk ? st[(size_t)(kr + 1) * A.dv + col + c] : 0.0f);
         }
-    // the neutral row: r = u = a = 0, w = 1 (key channels beyond dk for good; whole tokens beyond the end in the last chunk)
+    // Channels beyond the padded head (r = u = a = 0, w = 1) are written once; whole tokens beyond the end in the last chunk.
+    const int d4 = gd_pad4(dk);
     auto neutral = [&](float* base, int tt, int i) {
         float* at = base + tt * TS + (i / DKP) * PS + i % DKP;
         at[0] = 0.0f;
@@ -259,40 +268,68 @@ __global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDelt
         at[2 * TC * TS] = 1.0f;
         at[3 * TC * TS] = 0.0f;
     };
-    for (int idx = tid; idx < 2 * TC * P * DKP; idx += THREADS) {
-        const int b = idx / (TC * P * DKP), rest = idx - b * (TC * P * DKP);
-        const int tt = rest / (P * DKP), i = rest - tt * (P * DKP);
-        if (i >= dk) neutral(sm + b * buf_floats, tt, i);
+    if (d4 < P * DKP) {
+        for (int idx = tid; idx < 2 * TC * P * DKP; idx += THREADS) {
+            const int b = idx / (TC * P * DKP), rest = idx - b * (TC * P * DKP);
+            const int tt = rest / (P * DKP), i = rest - tt * (P * DKP);
+            if (i >= d4) neutral(sm + b * buf_floats, tt, i);
+        }
     }
-    const bool wide = (dk & 3) == 0;
+    // A token's pieces of 16 bytes: four vectors of P * DKP / 4, the scalars, DVT / 4 of v.  Every thread has fixed pieces of
+    // every token and walks their addresses from token to token.
+    constexpr int VEC_PIECES = P * DKP, PIECES = VEC_PIECES + 1 + DVT / 4, MINE = (PIECES + THREADS - 1) / THREADS;
+    const float* src[MINE];
+    int dst[MINE], step[MINE];
+#pragma unroll
+    for (int k = 0; k < MINE; ++k) {
+        const int piece = tid + k * THREADS;
+        src[k] = nullptr;
+        dst[k] = step[k] = 0;
+        const float* w = work + ((size_t)row0 * A.H + h) * wrow;
+        if (piece < VEC_PIECES) {
+            const int which = piece / (P * DKP / 4), i = (piece - which * (P * DKP / 4)) * 4;
+            if (i < d4) {
+                src[k] = w + which * d4 + i;
+                dst[k] = which * TC * TS + (i / DKP) * PS + i % DKP;
+                step[k] = TS;
+            }
+        } else if (piece == VEC_PIECES) {
+            src[k] = w + 4 * d4;
+            dst[k] = TC * (4 * TS + DVT);
+            step[k] = 4;
+        } else if (piece < PIECES) {
+            const int j = (piece - VEC_PIECES - 1) * 4;
+            if (col0 + j < A.dv) {
+                src[k] = w + 4 * d4 + 4 + col0 + j;
+                dst[k] = 4 * TC * TS + j;
+                step[k] = DVT;
+            }
+        }
+    }
+    const uint32_t sm0 = (uint32_t)__cvta_generic_to_shared(sm);
+    const size_t token = (size_t)A.H * wrow;
     auto fetch = [&](int c0, int b) {
         const int tc = min(TC, row1 - c0);
         float* base = sm + b * buf_floats;
-        float* vs = base + 4 * TC * TS;
-        float* sc = vs + TC * DVT;
-        for (int tt = 0; tt < tc; ++tt) {
-            const float* w = work + ((size_t)(c0 + tt) * A.H + h) * wrow;
-            float* at = base + tt * TS;
-            if (wide) {
-                for (int i = tid * 4; i < dk; i += THREADS * 4) {
-                    float* to = at + (i / DKP) * PS + i % DKP;
 #pragma unroll
-                    for (int k = 0; k < 4; ++k) gd_copy(to + k * TC * TS, w + k * dk + i, 16);
-                }
-            } else {
-                for (int i = tid; i < dk; i += THREADS) {
-                    float* to = at + (i / DKP) * PS + i % DKP;
-#pragma unroll
-                    for (int k = 0; k < 4; ++k) gd_copy(to + k * TC * TS, w + k * dk + i, 4);
-                }
+        for (int k = 0; k < MINE; ++k) {
+            if (!src[k]) continue;
+            uint32_t to = sm0 + 4u * (uint32_t)(b * buf_floats + dst[k]);
+            const float* from = src[k];
+            for (int tt = 0; tt < tc; ++tt) {
+                gd_copy16(to, from);
+                to += 4u * (uint32_t)step[k];
+                from += token;
             }
-            for (int j = tid; j < DVT; j += THREADS)
-                if (col0 + j < A.dv) gd_copy(vs + tt * DVT + j, w + 4 * dk + col0 + j, 4);
-            if (tid < 3) gd_copy(sc + tt * 4 + tid, w + 4 * dk + A.dv + tid, 4);
+            src[k] = from;
         }
-        for (int idx = tid; idx < (TC - tc) * P * DKP; idx += THREADS) neutral(base, tc + idx / (P * DKP), idx % (P * DKP));
-        for (int idx = tc * DVT + tid; idx < TC * DVT; idx += THREADS) vs[idx] = 0.0f;
-        for (int idx = tc * 4 + tid; idx < TC * 4; idx += THREADS) sc[idx] = 0.0f;
+        if (tc < TC) {
+            float* vs = base + 4 * TC * TS;
+            float* sc = vs + TC * DVT;
+            for (int idx = tid; idx < (TC - tc) * P * DKP; idx += THREADS) neutral(base, tc + idx / (P * DKP), idx % (P * DKP));
+            for (int idx = tc * DVT + tid; idx < TC * DVT; idx += THREADS) vs[idx] = 0.0f;
+            for (int idx = tc * 4 + tid; idx < TC * 4; idx += THREADS) sc[idx] = 0.0f;
+        }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     fetch(row0, 0);
@@ -317,13 +354,13 @@ __global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDelt
                 const float4 s4 = *reinterpret_cast<const float4*>(sc + tt * 4);
                 const float2 v2 = *reinterpret_cast<const float2*>(vs + tt * DVT + cl);
                 const float v[GD_COLS] = {col < A.dv ? v2.x : 0.0f, col + 1 < A.dv ? v2.y : 0.0f};
-                unsigned long long u[DKP / 2], w[DKP / 2], rv[DKP / 2], av[DKP / 2];
-                auto read = [&](unsigned long long (&x)[DKP / 2], int which) {
+                f32x2 u[DKP / 2], w[DKP / 2], rv[DKP / 2], av[DKP / 2];
+                auto read = [&](f32x2 (&x)[DKP / 2], int which) {
 #pragma unroll
                     for (int i = 0; i < DKP / 4; ++i) {
                         const float4 f = reinterpret_cast<const float4*>(mine + which * TC * TS + tt * TS)[i];
-                        x[2 * i] = gd_pack(f.x, f.y);
-                        x[2 * i + 1] = gd_pack(f.z, f.w);
+                        x[2 * i] = pack2f(f.x, f.y);
+                        x[2 * i + 1] = pack2f(f.z, f.w);
                     }
                 };
                 read(u, 1);
@@ -333,10 +370,10 @@ __global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDelt
                 float p[GD_COLS];
 #pragma unroll
                 for (int c = 0; c < GD_COLS; ++c) {
-                    unsigned long long x = gd_mul2(S[c][0], u[0]), y = gd_mul2(S[c][1], u[1]);
+                    f32x2 x = mul2f(S[c][0], u[0]), y = mul2f(S[c][1], u[1]);
 #pragma unroll
-                    for (int i = 2; i < DKP / 2; i += 2) { x = gd_fma2(S[c][i], u[i], x); y = gd_fma2(S[c][i + 1], u[i + 1], y); }
-                    p[c] = gd_sum(x) + gd_sum(y);
+                    for (int i = 2; i < DKP / 2; i += 2) { x = fma2f(S[c][i], u[i], x); y = fma2f(S[c][i + 1], u[i + 1], y); }
+                    p[c] = sum2f(x) + sum2f(y);
                 }
 #pragma unroll
                 for (int o = 1; o < P; o <<= 1)
@@ -344,19 +381,19 @@ __global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDelt
                     for (int c = 0; c < GD_COLS; ++c) p[c] += __shfl_xor_sync(0xffffffffu, p[c], o);
 #pragma unroll
                 for (int c = 0; c < GD_COLS; ++c) {
-                    unsigned long long x = gd_pack(0.0f, 0.0f), y = x;
+                    f32x2 x = pack2f(0.0f, 0.0f), y = x;
 #pragma unroll
                     for (int i = 0; i < DKP / 2; i += 2) {
-                        S[c][i] = gd_mul2(S[c][i], w[i]);
-                        S[c][i + 1] = gd_mul2(S[c][i + 1], w[i + 1]);
-                        x = gd_fma2(S[c][i], rv[i], x);
-                        y = gd_fma2(S[c][i + 1], rv[i + 1], y);
+                        S[c][i] = mul2f(S[c][i], w[i]);
+                        S[c][i + 1] = mul2f(S[c][i + 1], w[i + 1]);
+                        x = fma2f(S[c][i], rv[i], x);
+                        y = fma2f(S[c][i + 1], rv[i + 1], y);
                     }
                     // the token's own terms join the sum in one of the lanes
-                    q[k * GD_COLS + c] = gd_sum(x) + gd_sum(y) + (part == 0 ? fmaf(s4.z, v[c], -s4.y * p[c]) : 0.0f);
-                    const unsigned long long mp = gd_pack(-p[c], -p[c]), kv = gd_pack(s4.x * v[c], s4.x * v[c]);
+                    q[k * GD_COLS + c] = sum2f(x) + sum2f(y) + (part == 0 ? fmaf(s4.z, v[c], -s4.y * p[c]) : 0.0f);
+                    const f32x2 mp = pack2f(-p[c], -p[c]), kv = pack2f(s4.x * v[c], s4.x * v[c]);
 #pragma unroll
-                    for (int i = 0; i < DKP / 2; ++i) S[c][i] = gd_fma2(u[i], gd_fma2(av[i], mp, kv), S[c][i]);
+                    for (int i = 0; i < DKP / 2; ++i) S[c][i] = fma2f(u[i], fma2f(av[i], mp, kv), S[c][i]);
                 }
             }
             // V sums over P lanes: halve the values while there are several, then add up what is left
@@ -398,7 +435,7 @@ __global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDelt
         for (int i = 0; i < DKP / 2; ++i) {
             const int kr = part * DKP + 2 * i;
             float x, y;
-            asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(S[c][i]));
+            unpack2f(S[c][i], x, y);
             if (col + c < A.dv && kr < dk) st[(size_t)kr * A.dv + col + c] = x;
             if (col + c < A.dv && kr + 1 < dk) st[(size_t)(kr + 1) * A.dv + col + c] = y;
         }
@@ -445,7 +482,8 @@ template <typename T>
 static int launch_gd_portions(const GDeltaArgs& A, int n_reqs, int n_tokens, float* work, cudaStream_t s) {
     if (A.dk > 512) return launch_gd_scan<T>(A, n_reqs, s);     // very long keys: the kernel above
     const long long items = (long long)n_tokens * A.H;
-    vcb_launch(general_delta_prepare_kernel<T>, dim3((unsigned)((items + 3) / 4)), 128, 0, s, A, work, n_tokens);
+    if (gd_pairs(A)) vcb_launch(general_delta_prepare_kernel<T, 2>, dim3((unsigned)((items + 3) / 4)), 128, 0, s, A, work, n_tokens);
+    else vcb_launch(general_delta_prepare_kernel<T, 1>, dim3((unsigned)((items + 3) / 4)), 128, 0, s, A, work, n_tokens);
     if (int e = vcb_last_error()) return e;
     if (A.dk <= 8) return launch_gd_walk<8, 1>(A, n_reqs, work, s);
     if (A.dk <= 16) return launch_gd_walk<8, 2>(A, n_reqs, work, s);

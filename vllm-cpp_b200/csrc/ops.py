@@ -1533,7 +1533,8 @@ def selective_scan(x: torch.Tensor, dt_pre: torch.Tensor, b: torch.Tensor, c: to
 
 def general_delta_work(n: int, num_heads: int, head_dim: int, v_head_dim: int) -> int:
     """Floats of the prepared inputs of ``n`` tokens (csrc/general_delta.cu, gd_work_row)."""
-    return n * num_heads * ((4 * head_dim + v_head_dim + 4 + 3) // 4 * 4)
+    pad = lambda d: (d + 3) // 4 * 4
+    return n * num_heads * (4 * pad(head_dim) + 4 + pad(v_head_dim))
 
 
 def general_delta(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a_pre: torch.Tensor, z: torch.Tensor, a_bias: Optional[torch.Tensor],

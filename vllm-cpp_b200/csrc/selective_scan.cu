@@ -11,8 +11,8 @@
 //   selective_scan_kernel    portions: the same threads walk the request's tokens, whose step sizes, drives, B and C are made
 //                            once per chunk in shared memory while the values of the chunk after are on their way
 //
-// Exponentials are ex2.approx (2^-22 relative) of dt * A log2(e).  The reference has no recurrent mixer.
-#include "common.cuh"
+// Exponentials are ex2.approx (2^-22 relative) of dt * A log2(e); softplus and the gate are those of fast_math.cuh.  The reference has no recurrent mixer.
+#include "fast_math.cuh"
 
 struct SelectiveArgs {
     const void* x;              // [n, I] rows of T
@@ -31,14 +31,6 @@ struct SelectiveArgs {
     const int* state_slots;
     int I, N;
 };
-
-__device__ __forceinline__ float ss_exp2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ float ss_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
-__device__ __forceinline__ float ss_silu(float z) { return z / (1.0f + expf(-z)); }
 
 // NPT consecutive floats of a row of N (those beyond N: zero); quads where the row allows.
 template <int NPT>
@@ -83,7 +75,7 @@ __global__ void __launch_bounds__(128) selective_step_kernel(SelectiveArgs a, in
     float S[NPT];
     ss_load<NPT>(st, n0, a.N, quads, S);
     const float x = to_f32<T>(((const T*)a.x)[row * a.ldx + c]);
-    const float dt = ss_softplus(to_f32<T>(((const T*)a.dt_pre)[row * a.lddt + c]) + bias);
+    const float dt = fm_softplus(to_f32<T>(((const T*)a.dt_pre)[row * a.lddt + c]) + bias);
     const float z = to_f32<T>(((const T*)a.z)[row * a.ldz + c]);
     const T* bp = (const T*)a.b + row * a.ldb;
     const T* cp = (const T*)a.c + row * a.ldc;
@@ -93,31 +85,13 @@ __global__ void __launch_bounds__(128) selective_step_kernel(SelectiveArgs a, in
     for (int i = 0; i < NPT; ++i) {
         const bool in = n0 + i < a.N;
         const float bn = in ? to_f32<T>(bp[n0 + i]) : 0.0f, cn = in ? to_f32<T>(cp[n0 + i]) : 0.0f;
-        S[i] = fmaf(ss_exp2(dt * A[i]), S[i], dx * bn);
+        S[i] = fmaf(fm_ex2(dt * A[i]), S[i], dx * bn);
         y = fmaf(S[i], cn, y);
     }
     for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
     if (!there) return;
     ss_store<NPT>(st, n0, a.N, quads, S);
-    if (part == 0) ((T*)a.out)[row * a.ldo + c] = from_f32<T>(fmaf(dc, x, y) * ss_silu(z));
-}
-
-// Two floats to a 64-bit register and packed arithmetic on them.
-__device__ __forceinline__ unsigned long long ss_pack(float a, float b) {
-    unsigned long long r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-    return r;
-}
-__device__ __forceinline__ void ss_unpack(unsigned long long v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
-__device__ __forceinline__ unsigned long long ss_fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
-    unsigned long long r;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-    return r;
-}
-__device__ __forceinline__ unsigned long long ss_mul2(unsigned long long a, unsigned long long b) {
-    unsigned long long r;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-    return r;
+    if (part == 0) ((T*)a.out)[row * a.ldo + c] = from_f32<T>(fmaf(dc, x, y) * fm_silu(z));
 }
 
 // v[k], k = 0 .. L - 1: every lane's share of the sum of token k over the L lanes of a channel.  Returns, in lane `part`, the
@@ -143,6 +117,7 @@ template <typename T, int NPT, int L, int CB, int TC>
 __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a) {
     constexpr int THREADS = CB * L, PER = (TC * CB + THREADS - 1) / THREADS, NP = L * NPT, PERN = (TC * NP + THREADS - 1) / THREADS;
     constexpr int GROUP = (L <= TC) ? L : 1;                  // tokens walked together
+    static_assert(THREADS % NP == 0 && (TC % L == 0 || L > TC) && TC % (THREADS / NP) == 0, "whole rounds of staging");
     __shared__ __align__(16) float2 dts[TC][CB];              // dt, dt * x
     __shared__ __align__(16) float bs[TC][NP], cs[TC][NP];
     __shared__ float ys[TC][CB + 1];
@@ -150,10 +125,10 @@ __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a)
     const int c = min(c0 + cl, a.I - 1), n0 = part * NPT;
     const bool there = c0 + cl < a.I, quads = (a.N & 3) == 0;
     float S[NPT];
-    unsigned long long A2[NPT / 2], S2[NPT / 2];
+    f32x2 A2[NPT / 2], S2[NPT / 2];
     ss_load<NPT>(a.a2 + (size_t)c * a.N, n0, a.N, quads, S);
 #pragma unroll
-    for (int i = 0; i < NPT / 2; ++i) A2[i] = ss_pack(S[2 * i], S[2 * i + 1]);
+    for (int i = 0; i < NPT / 2; ++i) A2[i] = pack2f(S[2 * i], S[2 * i + 1]);
     const int sc = tid % CB, st0 = tid / CB;                  // staging: channel sc, tokens st0, st0 + L, ...
     const int scc = min(c0 + sc, a.I - 1);
     const float bias = a.dt_bias[scc], dc = a.d[scc];
@@ -164,31 +139,48 @@ __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a)
     float* st = a.state + ((size_t)a.state_slots[r] * a.I + c) * a.N;
     ss_load<NPT>(st, n0, a.N, quads, S);
 #pragma unroll
-    for (int i = 0; i < NPT / 2; ++i) S2[i] = ss_pack(S[2 * i], S[2 * i + 1]);
-    const T* xp = (const T*)a.x + (size_t)row0 * a.ldx + scc;
-    const T* dp = (const T*)a.dt_pre + (size_t)row0 * a.lddt + scc;
-    const T* zp = (const T*)a.z + (size_t)row0 * a.ldz + scc;
-    const T* bp = (const T*)a.b + (size_t)row0 * a.ldb;
-    const T* cp = (const T*)a.c + (size_t)row0 * a.ldc;
-    T* op = (T*)a.out + (size_t)row0 * a.ldo + scc;
+    for (int i = 0; i < NPT / 2; ++i) S2[i] = pack2f(S[2 * i], S[2 * i + 1]);
+    // every thread's own pointers to the values it stages next; a chunk advances them
+    const T* xp = (const T*)a.x + (size_t)(row0 + st0) * a.ldx + scc;
+    const T* dp = (const T*)a.dt_pre + (size_t)(row0 + st0) * a.lddt + scc;
+    const T* zp = (const T*)a.z + (size_t)(row0 + st0) * a.ldz + scc;
+    T* op = (T*)a.out + (size_t)(row0 + st0) * a.ldo + scc;
+    const int nb = min(tid % NP, a.N - 1), tb = tid / NP;        // B and C: state nb, tokens tb, tb + THREADS / NP, ...
+    const bool in = tid % NP < a.N;
+    constexpr int TB = THREADS / NP;
+    const T* bp = (const T*)a.b + (size_t)(row0 + tb) * a.ldb + nb;
+    const T* cp = (const T*)a.c + (size_t)(row0 + tb) * a.ldc + nb;
+    constexpr int ROWS = L < TC ? L : TC;                        // token rows the staging threads cover at once
+    const long long sx = (long long)ROWS * a.ldx, sd = (long long)ROWS * a.lddt, sz = (long long)ROWS * a.ldz, so = (long long)ROWS * a.ldo,
+                    sb = (long long)TB * a.ldb, scs = (long long)TB * a.ldc;
     T px[PER], pd[PER], pz[PER], pb[PERN], pc[PERN];          // a chunk's values on their way, as they are stored
-    auto fetch = [&](int t0) {
+#pragma unroll
+    for (int k = 0; k < PER; ++k) px[k] = pd[k] = pz[k] = from_f32<T>(0.0f);
+#pragma unroll
+    for (int k = 0; k < PERN; ++k) pb[k] = pc[k] = from_f32<T>(0.0f);
+    auto fetch = [&](int left) {                              // left: tokens from the chunk's first one on
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
-            const size_t tt = min(t0 + st0 + k * L, len - 1);
-            px[k] = xp[tt * a.ldx];
-            pd[k] = dp[tt * a.lddt];
-            pz[k] = zp[tt * a.ldz];
+            if (st0 + k * L < min(left, TC)) {
+                px[k] = *xp;
+                pd[k] = *dp;
+                pz[k] = *zp;
+            }
+            xp += sx;
+            dp += sd;
+            zp += sz;
         }
 #pragma unroll
         for (int k = 0; k < PERN; ++k) {
-            const int idx = tid + k * THREADS, t = idx / NP, n = min(idx - t * NP, a.N - 1);
-            const size_t tt = min(t0 + t, len - 1);
-            pb[k] = bp[tt * a.ldb + n];
-            pc[k] = cp[tt * a.ldc + n];
+            if (tb + k * TB < min(left, TC)) {
+                pb[k] = *bp;
+                pc[k] = *cp;
+            }
+            bp += sb;
+            cp += scs;
         }
     };
-    fetch(0);
+    fetch(len);
     for (int t0 = 0; t0 < len; t0 += TC) {
         const int tc = min(TC, len - t0);
         float zk[PER], xk[PER];
@@ -198,41 +190,41 @@ __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a)
             xk[k] = to_f32<T>(px[k]);
             zk[k] = to_f32<T>(pz[k]);
             if (t < TC) {
-                const float dt = t < tc ? ss_softplus(to_f32<T>(pd[k]) + bias) : 0.0f;
+                const float dt = t < tc ? fm_softplus(to_f32<T>(pd[k]) + bias) : 0.0f;
                 dts[t][sc] = make_float2(dt, dt * xk[k]);
             }
         }
 #pragma unroll
         for (int k = 0; k < PERN; ++k) {
-            const int idx = tid + k * THREADS, t = idx / NP, n = idx - t * NP;
+            const int t = tb + k * TB;
             if (t < TC) {
-                bs[t][n] = n < a.N ? to_f32<T>(pb[k]) : 0.0f;
-                cs[t][n] = n < a.N ? to_f32<T>(pc[k]) : 0.0f;
+                bs[t][tid % NP] = in ? to_f32<T>(pb[k]) : 0.0f;
+                cs[t][tid % NP] = in ? to_f32<T>(pc[k]) : 0.0f;
             }
         }
         __syncthreads();
-        if (t0 + TC < len) fetch(t0 + TC);
+        if (t0 + TC < len) fetch(len - t0 - TC);
 #pragma unroll
         for (int g = 0; g < TC; g += GROUP) {
             float y[GROUP];
 #pragma unroll
             for (int k = 0; k < GROUP; ++k) {
                 const float2 d = dts[g + k][cl];
-                const unsigned long long dt2 = ss_pack(d.x, d.x), dx2 = ss_pack(d.y, d.y);
-                unsigned long long y2 = ss_pack(0.0f, 0.0f);
+                const f32x2 dt2 = pack2f(d.x, d.x), dx2 = pack2f(d.y, d.y);
+                f32x2 y2 = pack2f(0.0f, 0.0f);
 #pragma unroll
                 for (int i = 0; i < NPT / 4; ++i) {
                     const float4 b4 = *reinterpret_cast<const float4*>(&bs[g + k][n0 + 4 * i]), c4 = *reinterpret_cast<const float4*>(&cs[g + k][n0 + 4 * i]);
                     float e0, e1, e2, e3;
-                    ss_unpack(ss_mul2(dt2, A2[2 * i]), e0, e1);
-                    ss_unpack(ss_mul2(dt2, A2[2 * i + 1]), e2, e3);
-                    S2[2 * i] = ss_fma2(ss_pack(ss_exp2(e0), ss_exp2(e1)), S2[2 * i], ss_mul2(dx2, ss_pack(b4.x, b4.y)));
-                    S2[2 * i + 1] = ss_fma2(ss_pack(ss_exp2(e2), ss_exp2(e3)), S2[2 * i + 1], ss_mul2(dx2, ss_pack(b4.z, b4.w)));
-                    y2 = ss_fma2(S2[2 * i], ss_pack(c4.x, c4.y), y2);
-                    y2 = ss_fma2(S2[2 * i + 1], ss_pack(c4.z, c4.w), y2);
+                    unpack2f(mul2f(dt2, A2[2 * i]), e0, e1);
+                    unpack2f(mul2f(dt2, A2[2 * i + 1]), e2, e3);
+                    S2[2 * i] = fma2f(pack2f(fm_ex2(e0), fm_ex2(e1)), S2[2 * i], mul2f(dx2, pack2f(b4.x, b4.y)));
+                    S2[2 * i + 1] = fma2f(pack2f(fm_ex2(e2), fm_ex2(e3)), S2[2 * i + 1], mul2f(dx2, pack2f(b4.z, b4.w)));
+                    y2 = fma2f(S2[2 * i], pack2f(c4.x, c4.y), y2);
+                    y2 = fma2f(S2[2 * i + 1], pack2f(c4.z, c4.w), y2);
                 }
                 float u, v;
-                ss_unpack(y2, u, v);
+                unpack2f(y2, u, v);
                 y[k] = u + v;
             }
             if constexpr (GROUP == L) {
@@ -248,12 +240,13 @@ __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a)
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
             const int t = st0 + k * L;
-            if (t < tc && c0 + sc < a.I) op[(size_t)(t0 + t) * a.ldo] = from_f32<T>(fmaf(dc, xk[k], ys[t][sc]) * ss_silu(zk[k]));
+            if (t < tc && c0 + sc < a.I) *op = from_f32<T>(fmaf(dc, xk[k], ys[t][sc]) * fm_silu(zk[k]));
+            op += so;
         }
         // ys is written again only after the next chunk's first barrier
     }
 #pragma unroll
-    for (int i = 0; i < NPT / 2; ++i) ss_unpack(S2[i], S[2 * i], S[2 * i + 1]);
+    for (int i = 0; i < NPT / 2; ++i) unpack2f(S2[i], S[2 * i], S[2 * i + 1]);
     if (there) ss_store<NPT>(st, n0, a.N, quads, S);
 }
 
@@ -275,8 +268,8 @@ static int launch_selective(const SelectiveArgs& a, int n_reqs, int max_q_len, c
         return vcb_last_error();
     }
     if (npt == 16) {
-        if (L == 16) launch_scan<T, 16, 16, 8>(a, n_reqs, s);
-        else launch_scan<T, 16, 32, 8>(a, n_reqs, s);
+        if (L == 16) launch_scan<T, 16, 16, 16>(a, n_reqs, s);
+        else launch_scan<T, 16, 32, 16>(a, n_reqs, s);
         return vcb_last_error();
     }
     switch (L) {
