@@ -201,13 +201,12 @@ __host__ __device__ static inline int gd_pad4(int n) { return (n + 3) / 4 * 4; }
 __host__ __device__ static inline int gd_work_row(int dk, int dv) { return 4 * gd_pad4(dk) + 4 + gd_pad4(dv); }
 
 template <typename T, int VW>
-__global__ void __launch_bounds__(128) general_delta_prepare_kernel(GDeltaArgs A, float* __restrict__ work, int n) {
-    pdl_start();
-    const int lane = threadIdx.x & 31;
-    const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-    if (item >= (long long)n * A.H) return;
-    const int row = (int)(item / A.H), h = (int)(item - (long long)row * A.H), dk = A.dk, d4 = gd_pad4(dk);
-    float* w = work + (size_t)item * gd_work_row(dk, A.dv);
+__global__ void __launch_bounds__(128) general_delta_prepare_kernel(GDeltaArgs A, float* __restrict__ work) {
+    // The walk's CTAs come when all of these have ended: placed while these fill the SMs, they would crowd on a few.
+    pdl_wait();
+    const int lane = threadIdx.x & 31, row = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), dk = A.dk, d4 = gd_pad4(dk);
+    if (h >= A.H) return;
+    float* w = work + ((size_t)row * A.H + h) * gd_work_row(dk, A.dv);
     float kn, ra, rk;
     gd_inputs<T, VW>(A, (size_t)row, h, lane, [&](int i, float rv, float u, float wv, float a) {
         w[i] = rv;
@@ -229,12 +228,11 @@ __device__ __forceinline__ void gd_copy16(uint32_t dst, const float* src) {
 }
 
 // Grid (request, head, tile of DVT value channels).  P lanes of a warp share GD_COLS neighbouring columns of S, of which a
-// thread keeps DKP rows each, two rows to a register pair: a token's row values are read from shared memory once for all the
-// thread's columns (the walk is bound by those reads and by the chain sum -> update of one token after another).  The sums
-// u . S that the update waits for go round the lanes at once; the read-outs of four tokens wait and are summed together, each
+// thread keeps DKP rows each, two rows to a register pair.  (The walk is bound by the chain sum -> update of one token after
+// another and by the reads of the token's rows.)  The sums u . S that the update waits for go round the lanes at once; the read-outs of four tokens wait and are summed together, each
 // round of shuffles handing half of them over.  Chunks of TC tokens' rows arrive by asynchronous copies a chunk ahead; tokens
 // beyond the portion's end are rows that leave S as it is.
-constexpr int GD_COLS = 2, GD_GROUP = 4, GD_WARPS = 2;
+constexpr int GD_COLS = 1, GD_GROUP = 4, GD_WARPS = 4 / GD_COLS;      // two columns a thread, with half the warps, measured slower
 
 template <int DKP, int P>
 __global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDeltaArgs A, const float* __restrict__ work) {
@@ -352,8 +350,9 @@ __global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDelt
             for (int k = 0; k < GD_GROUP; ++k) {
                 const int tt = g + k;
                 const float4 s4 = *reinterpret_cast<const float4*>(sc + tt * 4);
-                const float2 v2 = *reinterpret_cast<const float2*>(vs + tt * DVT + cl);
-                const float v[GD_COLS] = {col < A.dv ? v2.x : 0.0f, col + 1 < A.dv ? v2.y : 0.0f};
+                float v[GD_COLS];
+#pragma unroll
+                for (int c = 0; c < GD_COLS; ++c) v[c] = col + c < A.dv ? vs[tt * DVT + cl + c] : 0.0f;
                 f32x2 u[DKP / 2], w[DKP / 2], rv[DKP / 2], av[DKP / 2];
                 auto read = [&](f32x2 (&x)[DKP / 2], int which) {
 #pragma unroll
@@ -481,9 +480,8 @@ static int launch_gd_scan(const GDeltaArgs& A, int n_reqs, cudaStream_t s) {
 template <typename T>
 static int launch_gd_portions(const GDeltaArgs& A, int n_reqs, int n_tokens, float* work, cudaStream_t s) {
     if (A.dk > 512) return launch_gd_scan<T>(A, n_reqs, s);     // very long keys: the kernel above
-    const long long items = (long long)n_tokens * A.H;
-    if (gd_pairs(A)) vcb_launch(general_delta_prepare_kernel<T, 2>, dim3((unsigned)((items + 3) / 4)), 128, 0, s, A, work, n_tokens);
-    else vcb_launch(general_delta_prepare_kernel<T, 1>, dim3((unsigned)((items + 3) / 4)), 128, 0, s, A, work, n_tokens);
+    if (gd_pairs(A)) vcb_launch(general_delta_prepare_kernel<T, 2>, dim3(n_tokens, (A.H + 3) / 4), 128, 0, s, A, work);
+    else vcb_launch(general_delta_prepare_kernel<T, 1>, dim3(n_tokens, (A.H + 3) / 4), 128, 0, s, A, work);
     if (int e = vcb_last_error()) return e;
     if (A.dk <= 8) return launch_gd_walk<8, 1>(A, n_reqs, work, s);
     if (A.dk <= 16) return launch_gd_walk<8, 2>(A, n_reqs, work, s);

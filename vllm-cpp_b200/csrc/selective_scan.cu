@@ -35,9 +35,9 @@ struct SelectiveArgs {
 // NPT consecutive floats of a row of N (those beyond N: zero); quads where the row allows.
 template <int NPT>
 __device__ __forceinline__ void ss_load(const float* p, int n0, int N, bool quads, float (&v)[NPT]) {
-    if (quads && n0 + NPT <= N) {
+    if (NPT >= 4 && quads && n0 + NPT <= N) {
 #pragma unroll
-        for (int i = 0; i < NPT; i += 4) {
+        for (int i = 0; i + 3 < NPT; i += 4) {
             const float4 q = *reinterpret_cast<const float4*>(p + n0 + i);
             v[i] = q.x; v[i + 1] = q.y; v[i + 2] = q.z; v[i + 3] = q.w;
         }
@@ -48,9 +48,9 @@ __device__ __forceinline__ void ss_load(const float* p, int n0, int N, bool quad
 }
 template <int NPT>
 __device__ __forceinline__ void ss_store(float* p, int n0, int N, bool quads, const float (&v)[NPT]) {
-    if (quads && n0 + NPT <= N) {
+    if (NPT >= 4 && quads && n0 + NPT <= N) {
 #pragma unroll
-        for (int i = 0; i < NPT; i += 4) *reinterpret_cast<float4*>(p + n0 + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+        for (int i = 0; i + 3 < NPT; i += 4) *reinterpret_cast<float4*>(p + n0 + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
         return;
     }
 #pragma unroll
@@ -213,15 +213,12 @@ __global__ void __launch_bounds__(CB * L) selective_scan_kernel(SelectiveArgs a)
                 const f32x2 dt2 = pack2f(d.x, d.x), dx2 = pack2f(d.y, d.y);
                 f32x2 y2 = pack2f(0.0f, 0.0f);
 #pragma unroll
-                for (int i = 0; i < NPT / 4; ++i) {
-                    const float4 b4 = *reinterpret_cast<const float4*>(&bs[g + k][n0 + 4 * i]), c4 = *reinterpret_cast<const float4*>(&cs[g + k][n0 + 4 * i]);
-                    float e0, e1, e2, e3;
-                    unpack2f(mul2f(dt2, A2[2 * i]), e0, e1);
-                    unpack2f(mul2f(dt2, A2[2 * i + 1]), e2, e3);
-                    S2[2 * i] = fma2f(pack2f(fm_ex2(e0), fm_ex2(e1)), S2[2 * i], mul2f(dx2, pack2f(b4.x, b4.y)));
-                    S2[2 * i + 1] = fma2f(pack2f(fm_ex2(e2), fm_ex2(e3)), S2[2 * i + 1], mul2f(dx2, pack2f(b4.z, b4.w)));
-                    y2 = fma2f(S2[2 * i], pack2f(c4.x, c4.y), y2);
-                    y2 = fma2f(S2[2 * i + 1], pack2f(c4.z, c4.w), y2);
+                for (int i = 0; i < NPT / 2; ++i) {
+                    const float2 b2 = *reinterpret_cast<const float2*>(&bs[g + k][n0 + 2 * i]), c2 = *reinterpret_cast<const float2*>(&cs[g + k][n0 + 2 * i]);
+                    float e0, e1;
+                    unpack2f(mul2f(dt2, A2[i]), e0, e1);
+                    S2[i] = fma2f(pack2f(fm_ex2(e0), fm_ex2(e1)), S2[i], mul2f(dx2, pack2f(b2.x, b2.y)));
+                    y2 = fma2f(S2[i], pack2f(c2.x, c2.y), y2);
                 }
                 float u, v;
                 unpack2f(y2, u, v);
@@ -272,11 +269,17 @@ static int launch_selective(const SelectiveArgs& a, int n_reqs, int max_q_len, c
         else launch_scan<T, 16, 32, 16>(a, n_reqs, s);
         return vcb_last_error();
     }
+    // two states a thread where the channels alone leave the SMs with few warps
+    if (a.N <= 32 && a.N > 1) {
+        if (a.N <= 2) launch_scan<T, 2, 1, 32>(a, n_reqs, s);
+        else if (a.N <= 4) launch_scan<T, 2, 2, 32>(a, n_reqs, s);
+        else if (a.N <= 8) launch_scan<T, 2, 4, 32>(a, n_reqs, s);
+        else if (a.N <= 16) launch_scan<T, 2, 8, 16>(a, n_reqs, s);
+        else launch_scan<T, 2, 16, 8>(a, n_reqs, s);
+        return vcb_last_error();
+    }
     switch (L) {
         case 1: launch_scan<T, 4, 1, 32>(a, n_reqs, s); break;
-        case 2: launch_scan<T, 4, 2, 32>(a, n_reqs, s); break;
-        case 4: launch_scan<T, 4, 4, 32>(a, n_reqs, s); break;
-        case 8: launch_scan<T, 4, 8, 16>(a, n_reqs, s); break;
         case 16: launch_scan<T, 4, 16, 8>(a, n_reqs, s); break;
         default: launch_scan<T, 4, 32, 8>(a, n_reqs, s); break;
     }
