@@ -201,7 +201,8 @@ def windowed_attention(h, w, p, m, eps):
 
 
 def selective_scan_core(x, dt, A, B, C, D, S=None):
-    """S[c, n] <- exp(dt_c A[c, n]) S + dt_c x_c B_n;  y_c = S[c] . C + D_c x_c.  Returns (y, S)."""
+    """A token's step: every channel's row of S decays by e^(dt * its row of A), takes in (dt * x) B and is read by C; the token's
+    own x joins times D.  Returns (y, S)."""
     S = np.zeros(A.shape) if S is None else S.copy()
     y = np.empty_like(x)
     for t in range(x.shape[0]):

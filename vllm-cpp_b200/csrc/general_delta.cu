@@ -228,11 +228,12 @@ __device__ __forceinline__ void gd_copy16(uint32_t dst, const float* src) {
 }
 
 // Grid (request, head, tile of DVT value channels).  P lanes of a warp share GD_COLS neighbouring columns of S, of which a
-// thread keeps DKP rows each, two rows to a register pair.  (The walk is bound by the chain sum -> update of one token after
-// another and by the reads of the token's rows.)  The sums u . S that the update waits for go round the lanes at once; the read-outs of four tokens wait and are summed together, each
-// round of shuffles handing half of them over.  Chunks of TC tokens' rows arrive by asynchronous copies a chunk ahead; tokens
+// thread keeps DKP rows each, two rows to a register pair: a token's row values are read from shared memory once for both
+// columns.  (The walk is bound by the chain sum -> update of one token after another; one column a thread with twice the warps
+// measured a tenth slower.)  The sums u . S that the update waits for go round the lanes at once; the read-outs of four tokens
+// wait and are summed together, each round of shuffles handing half of them over.  Chunks of TC tokens' rows arrive by asynchronous copies a chunk ahead; tokens
 // beyond the portion's end are rows that leave S as it is.
-constexpr int GD_COLS = 1, GD_GROUP = 4, GD_WARPS = 4 / GD_COLS;      // two columns a thread, with half the warps, measured slower
+constexpr int GD_COLS = 2, GD_GROUP = 4, GD_WARPS = 4 / GD_COLS;
 
 template <int DKP, int P>
 __global__ void __launch_bounds__(32 * GD_WARPS) general_delta_walk_kernel(GDeltaArgs A, const float* __restrict__ work) {

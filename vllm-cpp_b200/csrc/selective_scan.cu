@@ -1,9 +1,10 @@
 // A selective state space: per channel c a state of N numbers that decays and is driven by the token, with step sizes,
 // drive and read-out made from the token itself,
 //
-//   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,     y_c = sum_n S[c, n] C_n + D_c x_c,     out_c = y_c * silu(z_c)
+//   s_n <- e^(dt a_n) s_n + (dt x) b_n  for n < N,     y = b'.s + d x  with read-out weights b' of the token,     out = silu(z) y
 //
-// dt = softplus(dt_pre + dt_bias).  x, dt_pre, B, C and z are rows of the activations' type; step sizes, exponentials, state,
+// (the channel's own a and d; b and b' are the same for all channels of a token: B and C below; dt = softplus(dt_pre + dt_bias)).
+// x, dt_pre, B, C and z are rows of the activations' type; step sizes, exponentials, state,
 // sums and the gate are float.  The state lives in the request's slot ([slots][I][N]), is read at the start of a request's
 // portion and left there at its end.
 //

@@ -2,7 +2,7 @@
 key channel, from which it removes, at a rate per key channel, what S holds under the token's unit key, and to which it adds
 the outer product of its plain key and value:
 
-    r = W_r h, k = W_k h, v = W_v h;   w = exp(-decay_rate * sigmoid(W_w2 tanh(W_w1 h) + w0));   a = sigmoid(W_a h + b_a)
+    [r; k; v] = [W_r; W_k; W_v] h;   w = exp(-decay_rate * sigmoid(W_w2 tanh(W_w1 h) + w0));   a = sigmoid(W_a h + b_a)
     u = k / sqrt(sum k^2 + 1e-6) per head;   S <- diag(w) S - (a * u) (u^T S) + k v^T  (both terms of the old S);   o = S^T r
     out = W_o (rms_head(o) * norm * sigmoid(W_g h))            a gain per channel of all heads
 

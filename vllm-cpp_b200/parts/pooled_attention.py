@@ -1,12 +1,12 @@
 """Grouped-query attention over a sliding window of tokens plus, for what lies before the window, one mean key and one mean
 value per block of ``pool`` tokens:
 
-    q = conv(W_q h + b_q), k = conv(W_k h + b_k), v = conv(W_v h + b_v)       a causal convolution over time per channel (``taps``)
+    (q, k, v) = conv([W_q; W_k; W_v] h + b)                                  a causal convolution over time per channel (``taps``)
     q, k rotated by position on the first ``rotary_dim`` coordinates of a head (interleaved pairs; "none": no rotation)
     score = (q . k) * scale * temp[head]
     position i sees the tokens j with 0 <= i - j < window, and the block b of the positions b P .. b P + P - 1 if
-    b P + P - 1 <= i - window; a block's key and value are the means of its tokens' keys and values as the cache holds them;
-    tokens that have left the window and whose block is not seen yet are not seen.  One softmax over tokens and blocks.
+    b P + P - 1 <= i - window; a block's key and value are the means of its tokens' cached keys and values.  Between the two
+    lies a gap of fewer than P tokens that nothing shows.  One softmax over tokens and blocks.
     out = W_o concat_heads(.)
 
 ``window`` 0: every token is seen; ``pool`` 0: nothing before the window is.  The mixer keeps three things per request: the

@@ -1,8 +1,8 @@
 """A selective state space as a mixer: per channel a vector of ``state`` numbers whose decay, drive and read-out follow the token.
 
     [x | z] = W_in h (``inner`` channels each);   x = silu(conv(x) + b)          a causal convolution over time per channel (``taps``)
-    [low | B | C] = W_x x (``dt_rank``, ``state``, ``state``);   dt = softplus(W_dt low + b_dt);   A = -exp(A_log)
-    S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n;   y_c = sum_n S[c, n] C_n + D_c x_c
+    [low | b | b'] = W_x x (``dt_rank``, ``state``, ``state``);   dt = softplus(W_dt low + b_dt), a step size per channel
+    per channel, with its row a = -e^(A_log) and its number d:   s <- e^(dt a) * s + (dt x) b  (elementwise);   y = b'.s + d x
     out = W_o (y * silu(z))
 
 The state S (float32 [inner, state]) and the convolution's last taps - 1 inputs live in slots of the cache manager, zero at
