@@ -82,11 +82,11 @@ struct GemmArgs {
     int ldr, sumsq_ld;
     // Gated feed-forward (swapped products on a gated tile image only): > 0 = the number of gate features.
     // Tile t holds gate rows 64 t .. and, in its upper half, the matching up rows;
-    // out[token, 64 t + r] = act(gate) * up, act 0: silu, 1: relu.
-    int gated, gated_act;
+    // out[token, 64 t + r] = act(gate) * up, act silu or relu (the kernel's parameter).
+    int gated;
 };
 
-__device__ __forceinline__ float gate_activation(int act, float z) { return act == 1 ? fmaxf(z, 0.0f) : z / (1.0f + expf(-z)); }
+template <bool RELU> __device__ __forceinline__ float gate_activation(float z) { return RELU ? fmaxf(z, 0.0f) : z / (1.0f + expf(-z)); }
 
 // The segments of one CTA's run of (tile, slab) units.
 struct Segments {
@@ -210,7 +210,7 @@ struct Units {
     }
 };
 
-template <int BN, int STAGES>
+template <int BN, int STAGES, bool RELU>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant__ CUtensorMap map_q, GemmArgs a) {
     constexpr int Q_BYTES = BN * BK * 2;
@@ -379,7 +379,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
                             const float f = a.scale_sumsq ? rstd_s[j] : 1.0f;
                             const float z = v[g8 + e] * f, u = xch[r * 8 + e] * f;
                             reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)j * a.ldc + feature] =
-                                __float2bfloat16_rn(gate_activation(a.gated_act, z) * u);
+                                __float2bfloat16_rn(gate_activation<RELU>(z) * u);
                         }
                     }
                     asm volatile("bar.sync 1, 128;" ::: "memory");   // the halves are read before the next group overwrites them
@@ -481,7 +481,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
                                 const float z = (is_gate ? __uint_as_float(lo[e]) : from_gate[e * 64 + half_row]) * f;
                                 const float u = (is_gate ? from_up[e * 64 + half_row] : __uint_as_float(hi[e])) * f;
                                 reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)j * a.ldc + feature] =
-                                    __float2bfloat16_rn(gate_activation(a.gated_act, z) * u);
+                                    __float2bfloat16_rn(gate_activation<RELU>(z) * u);
                             }
                         }
                         asm volatile("bar.sync 1, 128;" ::: "memory");   // read before the next round overwrites
@@ -657,14 +657,22 @@ int make_map(CUtensorMap* map, const void* base, int rows, int k, int ld, int bo
     return r == CUDA_SUCCESS ? 0 : VCB_ERR_BAD_ARG;
 }
 
-template <int BN, int STAGES>
-int launch(const CUtensorMap& mp, const CUtensorMap& mq, const GemmArgs& a, int ctas, cudaStream_t s) {
+template <int BN, int STAGES, bool RELU>
+int launch_as(const CUtensorMap& mp, const CUtensorMap& mq, const GemmArgs& a, int ctas, cudaStream_t s) {
     // stages, 1 KB to align them, barriers with the epilogue's factor and exchange areas (2 KB, 8 KB for wide tiles)
     constexpr size_t smem = (size_t)STAGES * (P_BYTES + BN * BK * 2) + 1024 + (BN >= 32 ? 9216 : 3072);
     static unsigned long long configured = 0;
-    if (int e = vcb_allow_dynamic_smem(gemm_tcgen05_kernel<BN, STAGES>, (int)smem, &configured)) return e;
-    vcb_launch(gemm_tcgen05_kernel<BN, STAGES>, ctas, GEMM_THREADS, smem, s, mp, mq, a);
+    if (int e = vcb_allow_dynamic_smem(gemm_tcgen05_kernel<BN, STAGES, RELU>, (int)smem, &configured)) return e;
+    vcb_launch(gemm_tcgen05_kernel<BN, STAGES, RELU>, ctas, GEMM_THREADS, smem, s, mp, mq, a);
     return vcb_last_error();
+}
+
+// relu: the activation of a gated product (tiles of up to 128 columns); other products do not look at it
+template <int BN, int STAGES>
+int launch(const CUtensorMap& mp, const CUtensorMap& mq, const GemmArgs& a, int ctas, bool relu, cudaStream_t s) {
+    if constexpr (BN <= 128)
+        if (relu) return launch_as<BN, STAGES, true>(mp, mq, a, ctas, s);
+    return launch_as<BN, STAGES, false>(mp, mq, a, ctas, s);
 }
 
 }  // namespace
@@ -774,14 +782,15 @@ VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused_act(const void* p, int rows_p, int ld
     GemmArgs a{out, partial, tickets, status, (const uint8_t*)p_tiled, ldc, out_f32, swapped, rows_p, rows_q,
                k_slabs, tiles_p, per, (int)total,
                scale_sumsq, scale_parts, scale_ld, scale_sumsq ? 1.0f / (float)scale_width : 0.0f, scale_eps,
-               residual, gain, sumsq_out, ldr, sumsq_ld, gated, gated_act};
+               residual, gain, sumsq_out, ldr, sumsq_ld, gated};
+    const bool relu = gated && gated_act == 1;
     cudaStream_t s = (cudaStream_t)stream;
     switch (bn) {
-        case 16: return launch<16, 6>(mp, mq, a, ctas, s);
-        case 32: return launch<32, 5>(mp, mq, a, ctas, s);
-        case 64: return max_ctas > vcb_sm_count() ? launch<64, 4>(mp, mq, a, ctas, s) : launch<64, 8>(mp, mq, a, ctas, s);
-        case 128: return launch<128, 6>(mp, mq, a, ctas, s);
-        default: return launch<256, 4>(mp, mq, a, ctas, s);
+        case 16: return launch<16, 6>(mp, mq, a, ctas, relu, s);
+        case 32: return launch<32, 5>(mp, mq, a, ctas, relu, s);
+        case 64: return max_ctas > vcb_sm_count() ? launch<64, 4>(mp, mq, a, ctas, relu, s) : launch<64, 8>(mp, mq, a, ctas, relu, s);
+        case 128: return launch<128, 6>(mp, mq, a, ctas, relu, s);
+        default: return launch<256, 4>(mp, mq, a, ctas, relu, s);
     }
 }
 
