@@ -15,7 +15,8 @@ a request holds ``n`` tokens no later query reads a key at or below n - window.
 A group whose rows stand for ``stride`` tokens each (PagedKVSpec.stride) hands out pages
 for n // stride rows; its pool is sized so that whatever fits a group of one row per
 token fits it too.  A windowed group that such rows are made from (``keep_block``)
-keeps the tokens of the block that is not complete yet.
+keeps the tokens of the block that is not complete yet, and one whose first tokens stay visible
+(``keep_first``) keeps the pages that hold them.
 Layers that declare a StateSpec get one slot per live request in a tensor of
 their own; the slot is zeroed when the request is admitted.  A request always
 gets a slot id, even if no layer has state.
@@ -228,6 +229,8 @@ class CacheManager:
                 dead = min(dead, rc.num_tokens // g.spec.keep_block * g.spec.keep_block)
             dead_blocks = max(0, dead // self.page_size)
             table = rc.tables[gi]
+            # the pages of the first tokens stay
+            rc.released[gi] = max(rc.released[gi], cdiv(g.spec.keep_first, self.page_size))
             for b in range(rc.released[gi], min(dead_blocks, len(table))):
                 g.pool.release(table[b])
                 table[b] = RELEASED

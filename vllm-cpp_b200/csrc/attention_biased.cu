@@ -5,8 +5,8 @@
 //                                (all heads at once, one gain per channel), the normed keys and the values into
 //                                the token's slot of the cache, the normed queries out
 //   attention_biased_kernel      score(i, j) = cap * tanh(scale * (q_i . k_j) / cap) + bias[min(i - j, L - 1), head]
-//                                over the keys j <= i (window > 0: i - j < window), softmax, sum of values, and a
-//                                sigmoid gate on the result
+//                                over the keys j <= i (window > 0: i - j < window, or j < keep), softmax, sum of values,
+//                                and a sigmoid gate on the result
 //
 // The cache block of a (page, k|v, kv head) holds `page` rows of `row` elements in the layout of kv_pos
 // (common.cuh); keys fill the first dk elements of a row of the key plane, values the first dv of the value
@@ -29,7 +29,14 @@ struct QkNormArgs {
     int bt_stride, H, G, dk, dv, row, page, num_pages, write_kv;
     float eps;
     int* status;
+    // queries grow with the position: times 1 + temp_coef * ln((position + 1) / temp_every + 1), the quotient whole (temp_every 0: no)
+    float temp_coef;
+    int temp_every;
 };
+
+__device__ __forceinline__ float query_temperature(const QkNormArgs& a, int pos) {
+    return a.temp_every > 0 ? fmaf(a.temp_coef, logf((float)((pos + 1) / a.temp_every + 1)), 1.0f) : 1.0f;
+}
 
 template <typename T>
 __global__ void qk_norm_cache_write_kernel(QkNormArgs a) {
@@ -50,6 +57,7 @@ __global__ void qk_norm_cache_write_kernel(QkNormArgs a) {
         rk = 1.0f / sqrtf(block_sum(ss, scratch) / (float)nk + a.eps);
     }
     T* qo = (T*)a.q_out + (size_t)t * nq;
+    rq *= query_temperature(a, a.positions[t]);
     for (int i = threadIdx.x; i < nq; i += blockDim.x)
         qo[i] = from_f32<T>(to_f32<T>(src[a.q_off + i]) * rq * (a.wq ? a.wq[i] : 1.0f));
     if (!a.write_kv) return;
@@ -133,7 +141,8 @@ __global__ void qk_norm_cache_write_bf16x8_kernel(QkNormArgs a) {
         }
         __syncthreads();
     }
-    const float rq = a.wq ? 1.0f / sqrtf(both[0][32] / (float)(nq8 * 8) + a.eps) : 1.0f;
+    const int pos = a.positions[t];
+    const float rq = (a.wq ? 1.0f / sqrtf(both[0][32] / (float)(nq8 * 8) + a.eps) : 1.0f) * query_temperature(a, pos);
     const float rk = a.wk ? 1.0f / sqrtf(both[1][32] / (float)(nk8 * 8) + a.eps) : 1.0f;
     auto normed = [](const uint4& raw, float r, const float* w) {
         float f[8];
@@ -145,6 +154,9 @@ __global__ void qk_norm_cache_write_bf16x8_kernel(QkNormArgs a) {
             const float g[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
 #pragma unroll
             for (int e = 0; e < 4; ++e) p[e] = __floats2bfloat162_rn(f[2 * e] * r * g[2 * e], f[2 * e + 1] * r * g[2 * e + 1]);
+        } else if (r != 1.0f) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) p[e] = __floats2bfloat162_rn(f[2 * e] * r, f[2 * e + 1] * r);
         } else {
             out = raw;
         }
@@ -158,7 +170,6 @@ __global__ void qk_norm_cache_write_bf16x8_kernel(QkNormArgs a) {
     }
     for (int c = threadIdx.x + KEEP * blockDim.x; c < nq8; c += blockDim.x) qo[c] = normed(qsrc[c], rq, a.wq ? a.wq + c * 8 : nullptr);
     if (!a.write_kv) return;
-    const int pos = a.positions[t];
     const int lp = pos / a.page, slot = pos - lp * a.page;
     const int pg = lp < a.bt_stride ? a.block_table[(size_t)a.req_of_token[t] * a.bt_stride + lp] : -1;
     if ((unsigned)pg >= (unsigned)a.num_pages) {
@@ -178,16 +189,16 @@ __global__ void qk_norm_cache_write_bf16x8_kernel(QkNormArgs a) {
     }
 }
 
-VCB_EXPORT int vcb_qk_norm_cache_write(const void* proj, long long ld, int q_off, int k_off, int v_off, const float* wq,
-                                       const float* wk, void* q_out, void* cache, const int* positions,
-                                       const int* req_of_token, const int* block_table, int bt_stride, int n_tokens,
-                                       int H, int G, int dk, int dv, int row, int page, int num_pages, int write_kv,
-                                       float eps, int* status, int dtype, void* stream) {
+VCB_EXPORT int vcb_qk_norm_cache_write_temp(const void* proj, long long ld, int q_off, int k_off, int v_off, const float* wq,
+                                            const float* wk, void* q_out, void* cache, const int* positions,
+                                            const int* req_of_token, const int* block_table, int bt_stride, int n_tokens,
+                                            int H, int G, int dk, int dv, int row, int page, int num_pages, int write_kv,
+                                            float eps, float temp_coef, int temp_every, int* status, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
-    if (!proj || !q_out || !cache || H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || row < dk || row < dv || page <= 0)
+    if (!proj || !q_out || !cache || H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || row < dk || row < dv || page <= 0 || temp_every < 0)
         return VCB_ERR_BAD_ARG;
     QkNormArgs a{proj, ld, q_off, k_off, v_off, wq, wk, q_out, cache, positions, req_of_token, block_table, bt_stride,
-                 H, G, dk, dv, row, page, num_pages, write_kv, eps, status};
+                 H, G, dk, dv, row, page, num_pages, write_kv, eps, status, temp_coef, temp_every};
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = H * dk >= 2048 ? 512 : 256;
     const uintptr_t addrs = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache | (uintptr_t)wq | (uintptr_t)wk;
@@ -200,6 +211,16 @@ VCB_EXPORT int vcb_qk_norm_cache_write(const void* proj, long long ld, int q_off
     else if (dtype == VCB_BF16) vcb_launch(qk_norm_cache_write_kernel<__nv_bfloat16>, n_tokens, threads, 0, s, a);
     else return VCB_ERR_BAD_ARG;
     return vcb_last_error();
+}
+
+// Queries that do not grow with the position.
+VCB_EXPORT int vcb_qk_norm_cache_write(const void* proj, long long ld, int q_off, int k_off, int v_off, const float* wq,
+                                       const float* wk, void* q_out, void* cache, const int* positions,
+                                       const int* req_of_token, const int* block_table, int bt_stride, int n_tokens,
+                                       int H, int G, int dk, int dv, int row, int page, int num_pages, int write_kv,
+                                       float eps, int* status, int dtype, void* stream) {
+    return vcb_qk_norm_cache_write_temp(proj, ld, q_off, k_off, v_off, wq, wk, q_out, cache, positions, req_of_token, block_table, bt_stride,
+                                        n_tokens, H, G, dk, dv, row, page, num_pages, write_kv, eps, 0.0f, 0, status, dtype, stream);
 }
 
 // ------------------------------------------------------------- norm per head, rotation, cache write
@@ -332,6 +353,7 @@ struct BiasedAttnArgs {
     int* status;
     const float* sink;          // [nh] or null: a logit per head that joins the softmax's denominator and has no value
     int gate_per_head;          // 1: the gate holds one number per head ([n, nh]) instead of one per channel
+    int keep;                   // with a window: the sequence's first `keep` tokens are seen wherever the window is
 };
 
 template <typename T>
@@ -360,10 +382,13 @@ __global__ void attention_biased_kernel(BiasedAttnArgs a) {
     for (int k = 0; k < ATB_MAX_DV / 32; ++k) o[k] = 0.0f;
     float m = -INFINITY, l = 0.0f;
     const int kstart = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    // the keys seen, one after the other: the kept ones before the window, then the window's
+    const int kept = min(a.keep, kstart), seen = kept + pos - kstart + 1;
+    auto key_of = [&](int v) { return v < kept ? v : v - kept + kstart; };
 
-    for (int kb = kstart; kb <= pos; kb += 32) {
-        const int j = kb + lane;
-        bool valid = j <= pos;
+    for (int kb = 0; kb < seen; kb += 32) {
+        const int j = key_of(kb + lane);
+        bool valid = kb + lane < seen;
         float s = -INFINITY;
         unsigned long long koff = 0;
         if (valid) {
@@ -391,12 +416,12 @@ __global__ void attention_biased_kernel(BiasedAttnArgs a) {
         l = l * corr + warp_sum(p);
 #pragma unroll
         for (int k = 0; k < ATB_MAX_DV / 32; ++k) o[k] *= corr;
-        const int nvalid = min(32, pos - kb + 1);
+        const int nvalid = min(32, seen - kb);
         for (int jj = 0; jj < nvalid; ++jj) {
             const float pj = __shfl_sync(0xffffffffu, p, jj);
             const unsigned long long off = __shfl_sync(0xffffffffu, koff, jj);
             const T* vr = cache + off + v_off;
-            const int slot = (kb + jj) % a.page;
+            const int slot = key_of(kb + jj) % a.page;
 #pragma unroll
             for (int k = 0; k < ATB_MAX_DV / 32; ++k) {
                 const int dim = lane + 32 * k;
@@ -427,17 +452,17 @@ __global__ void attention_biased_kernel(BiasedAttnArgs a) {
     }
 }
 
-VCB_EXPORT int vcb_attention_biased(const void* q, const void* cache, void* out, const void* gate, long long ldg,
-                                    const int* positions, const int* req_of_token, const int* block_table, int bt_stride,
-                                    const float* bias, int bias_len, int n_tokens, int nh, int nkv, int dk, int dv, int row,
-                                    int page, int window, float scale, float cap, int num_pages, int* status,
-                                    const float* sink, int gate_per_head, int dtype, void* stream) {
+VCB_EXPORT int vcb_attention_biased_kept(const void* q, const void* cache, void* out, const void* gate, long long ldg,
+                                         const int* positions, const int* req_of_token, const int* block_table, int bt_stride,
+                                         const float* bias, int bias_len, int n_tokens, int nh, int nkv, int dk, int dv, int row,
+                                         int page, int window, int keep, float scale, float cap, int num_pages, int* status,
+                                         const float* sink, int gate_per_head, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
     if (dk <= 0 || dv <= 0 || dv > ATB_MAX_DV || dk > 1024 || row < dk || row < dv || nh <= 0 || nkv <= 0 || nh % nkv ||
-        page <= 0 || window < 0 || num_pages < 0 || (bias && bias_len <= 0))
+        page <= 0 || window < 0 || keep < 0 || num_pages < 0 || (bias && bias_len <= 0))
         return VCB_ERR_BAD_ARG;
     BiasedAttnArgs a{q, cache, out, gate, ldg, positions, req_of_token, block_table, bias, bias_len, bt_stride, n_tokens,
-                     nh, nkv, dk, dv, row, page, window, scale, cap, num_pages, status, sink, gate_per_head};
+                     nh, nkv, dk, dv, row, page, window, scale, cap, num_pages, status, sink, gate_per_head, keep};
     const long long items = (long long)n_tokens * nh;
     const int blocks = (int)((items + ATB_WARPS - 1) / ATB_WARPS);
     const size_t smem = (size_t)ATB_WARPS * dk * sizeof(float);
@@ -446,4 +471,14 @@ VCB_EXPORT int vcb_attention_biased(const void* q, const void* cache, void* out,
     else if (dtype == VCB_BF16) vcb_launch(attention_biased_kernel<__nv_bfloat16>, blocks, ATB_WARPS * 32, smem, s, a);
     else return VCB_ERR_BAD_ARG;
     return vcb_last_error();
+}
+
+// A window alone.
+VCB_EXPORT int vcb_attention_biased(const void* q, const void* cache, void* out, const void* gate, long long ldg,
+                                    const int* positions, const int* req_of_token, const int* block_table, int bt_stride,
+                                    const float* bias, int bias_len, int n_tokens, int nh, int nkv, int dk, int dv, int row,
+                                    int page, int window, float scale, float cap, int num_pages, int* status,
+                                    const float* sink, int gate_per_head, int dtype, void* stream) {
+    return vcb_attention_biased_kept(q, cache, out, gate, ldg, positions, req_of_token, block_table, bt_stride, bias, bias_len, n_tokens, nh,
+                                     nkv, dk, dv, row, page, window, 0, scale, cap, num_pages, status, sink, gate_per_head, dtype, stream);
 }

@@ -70,13 +70,19 @@ struct MmaAttnArgs {
     // Nonzero: the softmax weights enter the P V product as two bfloat16 terms, p = hi + lo with hi the rounding of p and lo
     // that of the rest (16 bits of mantissa instead of 8), for designs that want their attention weights in 32-bit.
     int precise_weights;
-    // Rows for blocks of `pool` tokens beside the window's tokens (the POOLED forms of both kernels; window > 0): pages of the
+    // Rows for blocks of `pool` tokens beside the window's tokens (the BEFORE_BLOCKS forms of both kernels; window > 0): pages of the
     // same layout in which row b of a request is the mean key and value of its tokens b pool .. b pool + pool - 1.  A query at
     // position i sees the rows b with (b + 1) pool - 1 <= i - window.
     const __nv_bfloat16* pooled;
     const int* pool_table;         // [n_reqs, pt_stride]
     int pt_stride, pool_pages, pool;
+    // The sequence's first `keep` tokens, seen wherever the window is (the BEFORE_KEPT forms; window > 0).
+    int keep;
 };
+
+// What a query sees before its window, as key tiles that come before the tiles of the window: nothing, rows of blocks, or the
+// first tokens of the sequence.
+enum { BEFORE_NONE = 0, BEFORE_BLOCKS = 1, BEFORE_KEPT = 2 };
 
 // 1 / (l + e^(sink - m)) * sigmoid(gate): what an output row is multiplied by.  m2: the reference of l in units of log2.
 __device__ __forceinline__ float epilogue_factor(const MmaAttnArgs& a, float l, float m2, size_t token, int head) {
@@ -292,10 +298,11 @@ __device__ __forceinline__ void load_q_frags(uint32_t (&qf)[D / 16][4], uint32_t
 }
 
 // ------------------------------------------------------------------ decode
-template <int D, int STAGES, bool POOLED>
+template <int D, int STAGES, int BEFORE>
 __global__ void __launch_bounds__(BLOCK_THREADS, 2)
 attention_decode_kernel(MmaAttnArgs a) {
     extern __shared__ __align__(1024) unsigned char smem[];
+    constexpr bool POOLED = BEFORE == BEFORE_BLOCKS, KEPT = BEFORE == BEFORE_KEPT;
     constexpr int TILE_BYTES = BN * D * 2;
     // The step's index arrays were copied in before its first kernel, and every cache row below the
     // request's newest position was written by an earlier step: both are read before
@@ -322,7 +329,8 @@ attention_decode_kernel(MmaAttnArgs a) {
     // (A number that would need more splits than the grid has falls back to equal parts.)
     // POOLED: the tiles of block rows come before the tiles of tokens, as tiles tile0 .. tok0 - 1 of the same run.  (A block that
     // this step completes ends at pos, inside the window: every visible row was written by an earlier step.)
-    const int blocks = POOLED ? lo / a.pool : 0;
+    // KEPT: the same with the tiles of the kept tokens that lie before the window, under their own positions.
+    const int blocks = POOLED ? lo / a.pool : KEPT ? min(a.keep, lo) : 0;
     const int tok0 = lo / BN, tile0 = tok0 - (blocks + BN - 1) / BN, tile1 = (hi + BN - 1) / BN;
     const int grid_splits = gridDim.x;
     int per = (tile1 - tile0 + grid_splits - 1) / grid_splits, nsplit = grid_splits;
@@ -373,14 +381,15 @@ attention_decode_kernel(MmaAttnArgs a) {
             const PageDiv pd(a.page);
             bool bad = false;
             if (POOLED && my0 < tok0) pw.init(a.pool_table + (size_t)r * a.pt_stride, pd.div((my0 - tile0) * BN), blocks, a.page, lane, a.pool_pages);
+            else if (KEPT && my0 < tok0) pw.init(bt, pd.div((my0 - tile0) * BN), blocks, a.page, lane, a.num_pages);
             else pw.init(bt, pd.div(my0 * BN), hi, a.page, lane, a.num_pages);
             const int cache_heads = a.nkv / a.kv_share;
             const size_t page_stride = (size_t)a.planes * cache_heads * a.page * D, head_base = (size_t)(g / a.kv_share) * a.page * D,
                          v_off = (size_t)(a.planes - 1) * cache_heads * a.page * D;
             for (int tile = my0; tile < my1; ++tile, ++it) {
                 const int st = it % STAGES;
-                const bool of_blocks = POOLED && tile < tok0;
-                if (POOLED && tile == tok0 && my0 < tok0) {          // from the block rows to the tokens
+                const bool of_blocks = BEFORE != BEFORE_NONE && tile < tok0;
+                if (BEFORE != BEFORE_NONE && tile == tok0 && my0 < tok0) {          // from the rows before the window to its tokens
                     bad = pw.bad;
                     pw.init(bt, pd.div(tile * BN), hi, a.page, lane, a.num_pages);
                 }
@@ -391,7 +400,7 @@ attention_decode_kernel(MmaAttnArgs a) {
                 __syncwarp();
                 produce_tile<D, BN>(s_tiles + st * 2 * TILE_BYTES, s_tiles + st * 2 * TILE_BYTES + TILE_BYTES,
                                     full0 + 8 * st, (of_blocks ? tile - tile0 : tile) * BN, of_blocks ? 0 : lo, of_blocks ? blocks : hi, pw,
-                                    of_blocks ? a.pooled : a.cache, head_base, page_stride, v_off, pd, lane, 0, a.planes == 1 ? 1 : 0);
+                                    POOLED && of_blocks ? a.pooled : a.cache, head_base, page_stride, v_off, pd, lane, 0, a.planes == 1 ? 1 : 0);
             }
             if ((pw.bad || bad) && a.status) atomicCAS(a.status, 0, VCB_STATUS_BAD_PAGE);
         } else {
@@ -401,7 +410,7 @@ attention_decode_kernel(MmaAttnArgs a) {
                 const int st = it % STAGES;
                 if (!cx_mbar_wait(full0 + 8 * st, (it / STAGES) & 1)) gave_up = true;
                 const uint32_t sk = s_tiles + st * 2 * TILE_BYTES, sv = a.planes == 1 ? sk : sk + TILE_BYTES;
-                const bool of_blocks = POOLED && tile < tok0;
+                const bool of_blocks = BEFORE != BEFORE_NONE && tile < tok0;
                 const int kt = (of_blocks ? tile - tile0 : tile) * BN, klo = of_blocks ? 0 : lo, khi = of_blocks ? blocks : hi;
                 const int kb = kt + warp * 16;           // this warp's 16 keys
                 float s[2][4];
@@ -570,20 +579,21 @@ attention_decode_kernel(MmaAttnArgs a) {
 }
 
 // ---------------------------------------------------------------- launchers
-template <int D, bool POOLED>
+template <int D, int BEFORE>
 static int launch_decode_as(const MmaAttnArgs& a, int n_list, int nsplit, cudaStream_t s) {
     constexpr int STAGES = 3;
     const size_t smem = (size_t)STAGES * 2 * BN * D * 2 + 16 * D * 2 + 2 * STAGES * 8 + 64;   // tiles, Q, barriers
     static unsigned long long configured = 0;
-    if (int e = vcb_allow_dynamic_smem(attention_decode_kernel<D, STAGES, POOLED>, (int)smem, &configured)) return e;
+    if (int e = vcb_allow_dynamic_smem(attention_decode_kernel<D, STAGES, BEFORE>, (int)smem, &configured)) return e;
     dim3 grid(nsplit, a.nkv, n_list);
-    vcb_launch(attention_decode_kernel<D, STAGES, POOLED>, grid, BLOCK_THREADS, smem, s, a);
+    vcb_launch(attention_decode_kernel<D, STAGES, BEFORE>, grid, BLOCK_THREADS, smem, s, a);
     return vcb_last_error();
 }
 
 template <int D>
 static int launch_decode(const MmaAttnArgs& a, int n_list, int nsplit, cudaStream_t s) {
-    return a.pooled ? launch_decode_as<D, true>(a, n_list, nsplit, s) : launch_decode_as<D, false>(a, n_list, nsplit, s);
+    if (a.pooled) return launch_decode_as<D, BEFORE_BLOCKS>(a, n_list, nsplit, s);
+    return a.keep > 0 && a.window > 0 ? launch_decode_as<D, BEFORE_KEPT>(a, n_list, nsplit, s) : launch_decode_as<D, BEFORE_NONE>(a, n_list, nsplit, s);
 }
 
 // ------------------------------------------------- prefill on tcgen05
@@ -713,11 +723,12 @@ __host__ __device__ constexpr uint32_t idesc(int n, bool b_mn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn ? (1u << 16) : 0u) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
 }
 
-template <int D, bool PRECISE, bool POOLED>
+template <int D, bool PRECISE, int BEFORE>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_prefill_tc_kernel(MmaAttnArgs a) {
     // PRECISE (a template parameter of this kernel): the weights' rest after their rounding to bfloat16 goes into the second
     // half of the S buffer, whose scores have been read by then, and a second P V product adds it.
+    constexpr bool POOLED = BEFORE == BEFORE_BLOCKS, KEPT = BEFORE == BEFORE_KEPT;
     static_assert(D == 64 || D == 128, "one or two planes of 64 elements; S, S and O fit 256 columns");
     constexpr int Q_BYTES = BMT * D * 2, KV_BYTES = TKT * D * 2, K_STAGES = k_stages<D>(), V_STAGES = v_stages<D>();
     extern __shared__ __align__(1024) unsigned char smem[];
@@ -779,7 +790,8 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
     const int hi = ctx + last_row / G + 1;
     const int lo = a.window > 0 ? max(0, ctx + row0 / G + 1 - a.window) : 0;
     // POOLED: tiles of block rows first (tiles tile0 .. tok0 - 1 of the run), as many rows as the last row of the tile sees
-    const int blocks = POOLED ? max(0, hi - a.window) / a.pool : 0;
+    // KEPT: the same with the tiles of the kept tokens before the last row's window
+    const int blocks = POOLED ? max(0, hi - a.window) / a.pool : KEPT ? min(a.keep, max(0, hi - a.window)) : 0;
     const int tok0 = lo / TKT, tile0 = tok0 - (blocks + TKT - 1) / TKT, tile1 = (hi + TKT - 1) / TKT;
     const int n_tiles = *abort_flag ? 0 : tile1 - tile0;
 
@@ -796,13 +808,15 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
         const PageDiv pd(a.page);
         bool bad = false;
         if (POOLED && tile0 < tok0) pw.init(a.pool_table + (size_t)r * a.pt_stride, 0, blocks, a.page, lane, a.pool_pages);
+        else if (KEPT && tile0 < tok0) pw.init(bt, 0, blocks, a.page, lane, a.num_pages);
         else pw.init(bt, pd.div(tile0 * TKT), hi, a.page, lane, a.num_pages);
         const size_t page_stride = (size_t)a.planes * a.nkv * a.page * D, head_base = (size_t)g * a.page * D,
                      v_off = (size_t)(a.planes - 1) * a.nkv * a.page * D;
         // a tile's addresses are worked out before its stage is waited for
         auto piece_of = [&](int tile) {
-            if (POOLED && tile < tok0) return tile_piece<D, TKT>((tile - tile0) * TKT, 0, blocks, pw, a.pooled, head_base, page_stride, pd, lane);
-            if (POOLED && tile == tok0 && tile0 < tok0) {           // from the block rows to the tokens
+            if (BEFORE != BEFORE_NONE && tile < tok0)
+                return tile_piece<D, TKT>((tile - tile0) * TKT, 0, blocks, pw, POOLED ? a.pooled : a.cache, head_base, page_stride, pd, lane);
+            if (BEFORE != BEFORE_NONE && tile == tok0 && tile0 < tok0) {           // from the rows before the window to its tokens
                 bad = pw.bad;
                 pw.init(bt, pd.div(tile * TKT), hi, a.page, lane, a.num_pages);
             }
@@ -930,14 +944,14 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
         bool ok = true;
         for (int j = 0; j < n_tiles && !*abort_flag; ++j) {
             const int st = j & 1;
-            const bool of_blocks = POOLED && tile0 + j < tok0;
+            const bool of_blocks = BEFORE != BEFORE_NONE && tile0 + j < tok0;
             const int kb = of_blocks ? j * TKT : (tile0 + j) * TKT;
             if (!cx_mbar_wait(B(S_FULL + st), (j >> 1) & 1)) { ok = false; break; }
             fence_after();
             const uint32_t s_addr = tm_s0 + st * TKT + lane_addr;
             // does any row of the tile mask any key of this tile? (the first row sees the fewest late keys,
             // the last row the fewest early ones)
-            const bool edge = of_blocks ? kb + TKT > max(0, ctx + row0 / G + 1 - a.window) / a.pool
+            const bool edge = of_blocks ? kb + TKT > (KEPT ? min(a.keep, max(0, ctx + row0 / G + 1 - a.window)) : max(0, ctx + row0 / G + 1 - a.window) / a.pool)
                                         : kb + TKT - 1 > ctx + row0 / G || (a.window > 0 && kb < ctx + last_row / G + 1 - a.window);
             float s[TKT];
             {
@@ -968,7 +982,7 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
                 }
             }
             if (edge) {
-                const int first = of_blocks ? 0 : row_lo, last = of_blocks ? row_lo / a.pool - 1 : pos;
+                const int first = of_blocks ? 0 : row_lo, last = of_blocks ? (KEPT ? min(a.keep, row_lo) : row_lo / a.pool) - 1 : pos;
 #pragma unroll
                 for (int i = 0; i < TKT; ++i) {
                     const int key = kb + i;
@@ -1071,18 +1085,19 @@ attention_prefill_tc_kernel(MmaAttnArgs a) {
 }
 }  // namespace tc
 
-template <int D, bool PRECISE, bool POOLED>
+template <int D, bool PRECISE, int BEFORE>
 static int launch_prefill_tc_as(const MmaAttnArgs& a, int n_tiles, cudaStream_t s) {
     static unsigned long long configured = 0;
-    if (int e = vcb_allow_dynamic_smem(tc::attention_prefill_tc_kernel<D, PRECISE, POOLED>, tc::smem_bytes<D>(), &configured)) return e;
-    vcb_launch(tc::attention_prefill_tc_kernel<D, PRECISE, POOLED>, dim3((unsigned)n_tiles * a.nkv), tc::THREADS, (size_t)tc::smem_bytes<D>(), s, a);
+    if (int e = vcb_allow_dynamic_smem(tc::attention_prefill_tc_kernel<D, PRECISE, BEFORE>, tc::smem_bytes<D>(), &configured)) return e;
+    vcb_launch(tc::attention_prefill_tc_kernel<D, PRECISE, BEFORE>, dim3((unsigned)n_tiles * a.nkv), tc::THREADS, (size_t)tc::smem_bytes<D>(), s, a);
     return vcb_last_error();
 }
 
 template <int D>
 static int launch_prefill_tc(const MmaAttnArgs& a, int n_tiles, cudaStream_t s) {
-    if (a.pooled) return launch_prefill_tc_as<D, true, true>(a, n_tiles, s);        // with two-term weights only
-    return a.precise_weights ? launch_prefill_tc_as<D, true, false>(a, n_tiles, s) : launch_prefill_tc_as<D, false, false>(a, n_tiles, s);
+    if (a.pooled) return launch_prefill_tc_as<D, true, BEFORE_BLOCKS>(a, n_tiles, s);        // with two-term weights only
+    if (a.keep > 0 && a.window > 0) return launch_prefill_tc_as<D, true, BEFORE_KEPT>(a, n_tiles, s);      // likewise
+    return a.precise_weights ? launch_prefill_tc_as<D, true, BEFORE_NONE>(a, n_tiles, s) : launch_prefill_tc_as<D, false, BEFORE_NONE>(a, n_tiles, s);
 }
 
 // Both kernels copy a tile of 64 keys as at most eight runs of whole pages' rows (tile_piece: one lane
@@ -1118,7 +1133,30 @@ VCB_EXPORT int vcb_attention_decode_mma_planes(const void* q, const void* cache,
     return d == 64 ? launch_decode<64>(a, n_list, nsplit, s) : launch_decode<128>(a, n_list, nsplit, s);
 }
 
-// The same with shaped scores and an epilogue (see MmaAttnArgs): cap <= 0 no cap; bias_t, sink, gate null: none.
+// The same with shaped scores and an epilogue (see MmaAttnArgs): cap <= 0 no cap; bias_t, sink, gate null: none; keep > 0 with a
+// window: the first tokens of the sequence stay visible (two-term weights in the portions' kernel).
+VCB_EXPORT int vcb_attention_decode_mma_shaped_kept(const void* q, const void* cache, void* out, const int* q_start,
+                                               const int* ctx_lens, const int* block_table, int bt_stride,
+                                               const int* req_list, int n_list, int nsplit, float* part_o,
+                                               float* part_ml, int* counters, const int* split_tiles, int nh, int nkv,
+                                               int d, int page, int window, float scale, int num_pages, int* status,
+                                               int kv_share, float cap, const float* bias_t, int bias_len, const float* sink,
+                                               const void* gate, long long ldg, int precise_weights, int planes, int keep, void* stream) {
+    if (n_list <= 0) return 0;
+    int c = check_common(nh, nkv, d, page, window, num_pages);
+    if (c) return c;
+    if (kv_share < 1 || nkv % kv_share || (bias_t && bias_len <= 0) || (planes != 1 && planes != 2) || keep < 0) return VCB_ERR_BAD_ARG;
+    if (nsplit < 1 || nsplit > 32 || (nsplit > 1 && (!part_o || !part_ml || !counters))) return VCB_ERR_BAD_ARG;
+    MmaAttnArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, q_start, ctx_lens,
+                  block_table, req_list, nullptr, part_o, part_ml, counters, status, split_tiles, bt_stride, nh, nkv,
+                  page, window, scale, num_pages, planes, kv_share, cap, bias_t, bias_len, sink, (const __nv_bfloat16*)gate, ldg,
+                  precise_weights};
+    a.keep = keep;
+    cudaStream_t s = (cudaStream_t)stream;
+    return d == 64 ? launch_decode<64>(a, n_list, nsplit, s) : launch_decode<128>(a, n_list, nsplit, s);
+}
+
+// A window alone.
 VCB_EXPORT int vcb_attention_decode_mma_shaped_planes(const void* q, const void* cache, void* out, const int* q_start,
                                                const int* ctx_lens, const int* block_table, int bt_stride,
                                                const int* req_list, int n_list, int nsplit, float* part_o,
@@ -1126,17 +1164,7 @@ VCB_EXPORT int vcb_attention_decode_mma_shaped_planes(const void* q, const void*
                                                int d, int page, int window, float scale, int num_pages, int* status,
                                                int kv_share, float cap, const float* bias_t, int bias_len, const float* sink,
                                                const void* gate, long long ldg, int precise_weights, int planes, void* stream) {
-    if (n_list <= 0) return 0;
-    int c = check_common(nh, nkv, d, page, window, num_pages);
-    if (c) return c;
-    if (kv_share < 1 || nkv % kv_share || (bias_t && bias_len <= 0) || (planes != 1 && planes != 2)) return VCB_ERR_BAD_ARG;
-    if (nsplit < 1 || nsplit > 32 || (nsplit > 1 && (!part_o || !part_ml || !counters))) return VCB_ERR_BAD_ARG;
-    MmaAttnArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, q_start, ctx_lens,
-                  block_table, req_list, nullptr, part_o, part_ml, counters, status, split_tiles, bt_stride, nh, nkv,
-                  page, window, scale, num_pages, planes, kv_share, cap, bias_t, bias_len, sink, (const __nv_bfloat16*)gate, ldg,
-                  precise_weights};
-    cudaStream_t s = (cudaStream_t)stream;
-    return d == 64 ? launch_decode<64>(a, n_list, nsplit, s) : launch_decode<128>(a, n_list, nsplit, s);
+    return vcb_attention_decode_mma_shaped_kept(q, cache, out, q_start, ctx_lens, block_table, bt_stride, req_list, n_list, nsplit, part_o, part_ml, counters, split_tiles, nh, nkv, d, page, window, scale, num_pages, status, kv_share, cap, bias_t, bias_len, sink, gate, ldg, precise_weights, planes, 0, stream);
 }
 
 // Keys and values in planes of their own.
@@ -1182,20 +1210,31 @@ VCB_EXPORT int vcb_attention_prefill_tc_planes(const void* q, const void* cache,
 }
 
 // The same with shaped scores and an epilogue (see MmaAttnArgs).
+VCB_EXPORT int vcb_attention_prefill_tc_shaped_kept(const void* q, const void* cache, void* out, const int* q_start,
+                                               const int* ctx_lens, const int* block_table, int bt_stride,
+                                               const int* tile_req, const int* tile_row0, int n_tiles, int nh,
+                                               int nkv, int d, int page, int window, float scale, int num_pages,
+                                               int* status, float cap, const float* bias_t, int bias_len, const float* sink,
+                                               const void* gate, long long ldg, int precise_weights, int planes, int keep, void* stream) {
+    if (n_tiles <= 0) return 0;
+    int c = check_common(nh, nkv, d, page, window, num_pages);
+    if (c) return c;
+    if ((bias_t && bias_len <= 0) || (planes != 1 && planes != 2) || keep < 0) return VCB_ERR_BAD_ARG;
+    MmaAttnArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, q_start, ctx_lens,
+                  block_table, tile_req, tile_row0, nullptr, nullptr, nullptr, status, nullptr, bt_stride, nh, nkv, page,
+                  window, scale, num_pages, planes, 1, cap, bias_t, bias_len, sink, (const __nv_bfloat16*)gate, ldg, precise_weights};
+    a.keep = keep;
+    return d == 64 ? launch_prefill_tc<64>(a, n_tiles, (cudaStream_t)stream) : launch_prefill_tc<128>(a, n_tiles, (cudaStream_t)stream);
+}
+
+// A window alone.
 VCB_EXPORT int vcb_attention_prefill_tc_shaped_planes(const void* q, const void* cache, void* out, const int* q_start,
                                                const int* ctx_lens, const int* block_table, int bt_stride,
                                                const int* tile_req, const int* tile_row0, int n_tiles, int nh,
                                                int nkv, int d, int page, int window, float scale, int num_pages,
                                                int* status, float cap, const float* bias_t, int bias_len, const float* sink,
                                                const void* gate, long long ldg, int precise_weights, int planes, void* stream) {
-    if (n_tiles <= 0) return 0;
-    int c = check_common(nh, nkv, d, page, window, num_pages);
-    if (c) return c;
-    if ((bias_t && bias_len <= 0) || (planes != 1 && planes != 2)) return VCB_ERR_BAD_ARG;
-    MmaAttnArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, q_start, ctx_lens,
-                  block_table, tile_req, tile_row0, nullptr, nullptr, nullptr, status, nullptr, bt_stride, nh, nkv, page,
-                  window, scale, num_pages, planes, 1, cap, bias_t, bias_len, sink, (const __nv_bfloat16*)gate, ldg, precise_weights};
-    return d == 64 ? launch_prefill_tc<64>(a, n_tiles, (cudaStream_t)stream) : launch_prefill_tc<128>(a, n_tiles, (cudaStream_t)stream);
+    return vcb_attention_prefill_tc_shaped_kept(q, cache, out, q_start, ctx_lens, block_table, bt_stride, tile_req, tile_row0, n_tiles, nh, nkv, d, page, window, scale, num_pages, status, cap, bias_t, bias_len, sink, gate, ldg, precise_weights, planes, 0, stream);
 }
 
 // Keys and values in planes of their own.

@@ -31,6 +31,7 @@ struct AttnArgs {
     int num_pages;              // a table entry outside [0, num_pages) is not read through: the key is left
     int* status;                // out and VCB_STATUS_BAD_PAGE is recorded here (may be null)
     int planes;
+    const float* sink;          // [nh] or null: a logit per head that joins the softmax's denominator once, unscaled, and has no value
 };
 
 template <typename T, int MAXD>
@@ -102,7 +103,12 @@ __global__ void attention_simt_kernel(AttnArgs a) {
         m = m_new;
     }
     T* orow = (T*)a.out + ((size_t)t * a.nh + h) * a.d;
-    const float inv = 1.0f / l;
+    float inv = 1.0f / l;
+    if (a.sink) {
+        // the reference of the exponents moves if the sink is the largest
+        const float sk = a.sink[h], mf = fmaxf(m, sk), keep = expf(m - mf);
+        inv = keep / (l * keep + expf(sk - mf));
+    }
 #pragma unroll
     for (int k = 0; k < MAXD / 32; ++k) {
         const int dim = lane + 32 * k;
@@ -110,16 +116,16 @@ __global__ void attention_simt_kernel(AttnArgs a) {
     }
 }
 
-VCB_EXPORT int vcb_attention_simt_planes(const void* q, const void* cache, void* out, const int* positions,
-                                  const int* req_of_token, const int* block_table, int bt_stride,
-                                  int n_tokens, int nh, int nkv, int d, int page, int window,
-                                  float scale, int num_pages, int* status, int planes, int dtype, void* stream) {
+VCB_EXPORT int vcb_attention_simt_sink(const void* q, const void* cache, void* out, const int* positions,
+                                       const int* req_of_token, const int* block_table, int bt_stride,
+                                       int n_tokens, int nh, int nkv, int d, int page, int window,
+                                       float scale, int num_pages, int* status, int planes, const float* sink, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
     if (d <= 0 || d > ATT_MAX_D || nh <= 0 || nkv <= 0 || nh % nkv || page <= 0 || window < 0 || num_pages < 0 ||
         (planes != 1 && planes != 2))
         return VCB_ERR_BAD_ARG;
     AttnArgs a{q, cache, out, positions, req_of_token, block_table, bt_stride, n_tokens, nh, nkv, d,
-               page, window, scale, num_pages, status, planes};
+               page, window, scale, num_pages, status, planes, sink};
     const long long items = (long long)n_tokens * nh;
     const int blocks = (int)((items + ATT_WARPS - 1) / ATT_WARPS);
     const size_t smem = (size_t)ATT_WARPS * d * sizeof(float);
@@ -133,6 +139,14 @@ VCB_EXPORT int vcb_attention_simt_planes(const void* q, const void* cache, void*
         else vcb_launch(attention_simt_kernel<__nv_bfloat16, 256>, blocks, ATT_WARPS * 32, smem, s, a);
     } else return VCB_ERR_BAD_ARG;
     return vcb_last_error();
+}
+
+VCB_EXPORT int vcb_attention_simt_planes(const void* q, const void* cache, void* out, const int* positions,
+                                  const int* req_of_token, const int* block_table, int bt_stride,
+                                  int n_tokens, int nh, int nkv, int d, int page, int window,
+                                  float scale, int num_pages, int* status, int planes, int dtype, void* stream) {
+    return vcb_attention_simt_sink(q, cache, out, positions, req_of_token, block_table, bt_stride, n_tokens, nh, nkv, d, page, window, scale,
+                                   num_pages, status, planes, nullptr, dtype, stream);
 }
 
 // Keys and values in planes of their own (planes = 2), the form every cache with separate keys and values has.

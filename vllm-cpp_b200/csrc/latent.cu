@@ -338,7 +338,8 @@ VCB_EXPORT int vcb_rows_rmsnorm(const void* x, int ldx, const float* gain, void*
 // key part of `rot` coordinates, turned by the token's position, that every head scores against the rotated part of
 // its query.  The same kernel turns the rotated part of every head's query in place: head h of q holds it at
 // q[t, h * q_stride + q_off .. + rot).  Pair j of a rotated part is (2j, 2j + 1) (pairing 1) or (j, j + rot / 2)
-// (pairing 0); its angle is position * inv_freq[j] in float; (u, v) -> (u cos - v sin, v cos + u sin).
+// (pairing 0); its angle is position * inv_freq[j] in float; (u, v) -> (u cos - v sin, v cos + u sin), cosine and sine
+// times `magnitude`.
 // A CTA per token.
 struct LatentRopeArgs {
     const void* raw;            // [n, ld]: the latent's columns, then the rot columns of the shared key part
@@ -357,6 +358,7 @@ struct LatentRopeArgs {
     int n_tokens, rank, page, num_pages, write_kv;
     float eps;
     int* status;
+    float magnitude;            // factor of cosine and sine
 };
 
 template <typename T>
@@ -374,6 +376,8 @@ __global__ void latent_rope_cache_write_kernel(LatentRopeArgs a) {
             const int h = idx / half, j = idx - h * half;
             float sn, cs;
             sincosf((float)pos * a.inv_freq[j], &sn, &cs);
+            sn *= a.magnitude;
+            cs *= a.magnitude;
             T* part = q + (size_t)h * a.q_stride + a.q_off;
             const int iu = a.pairing ? 2 * j : j, iv = a.pairing ? 2 * j + 1 : j + half;
             const float u = to_f32<T>(part[iu]), v = to_f32<T>(part[iv]);
@@ -402,6 +406,8 @@ __global__ void latent_rope_cache_write_kernel(LatentRopeArgs a) {
     for (int j = threadIdx.x; j < half; j += blockDim.x) {
         float sn, cs;
         sincosf((float)pos * a.inv_freq[j], &sn, &cs);
+        sn *= a.magnitude;
+        cs *= a.magnitude;
         const int iu = a.pairing ? 2 * j : j, iv = a.pairing ? 2 * j + 1 : j + half;
         const float u = to_f32<T>(row[a.rank + iu]), v = to_f32<T>(row[a.rank + iv]);
         dst[kv_pos(a.rank + iu, slot, row_w, a.page, (int)sizeof(T))] = from_f32<T>(u * cs - v * sn);
@@ -409,21 +415,32 @@ __global__ void latent_rope_cache_write_kernel(LatentRopeArgs a) {
     }
 }
 
-VCB_EXPORT int vcb_latent_rope_cache_write(const void* raw, int ld, const float* gain, void* q, int ldq, int heads, int q_stride,
+VCB_EXPORT int vcb_latent_rope_cache_write_scaled(const void* raw, int ld, const float* gain, void* q, int ldq, int heads, int q_stride,
                                            int q_off, const float* inv_freq, int rot, int pairing, const int* positions,
                                            const int* req_of_token, const int* block_table, int bt_stride, void* cache,
                                            long long page_stride, int n_tokens, int rank, int page, float eps, int num_pages,
-                                           int write_kv, int* status, int dtype, void* stream) {
+                                           int write_kv, float magnitude, int* status, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
     if (rank <= 0 || rot < 0 || (rot & 1) || (rot && !inv_freq) || page <= 0 || ld < rank + rot ||
         page_stride < (long long)page * (rank + rot) || num_pages <= 0 || (pairing != 0 && pairing != 1))
         return VCB_ERR_BAD_ARG;
     if (q && (heads <= 0 || q_off < 0 || q_stride < q_off + rot || ldq < heads * q_stride)) return VCB_ERR_BAD_ARG;
     LatentRopeArgs a{raw, ld, gain, q, ldq, heads, q_stride, q_off, inv_freq, rot, pairing, positions, req_of_token, block_table,
-                     bt_stride, cache, (size_t)page_stride, n_tokens, rank, page, num_pages, write_kv, eps, status};
+                     bt_stride, cache, (size_t)page_stride, n_tokens, rank, page, num_pages, write_kv, eps, status, magnitude};
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == VCB_F32) vcb_launch(latent_rope_cache_write_kernel<float>, n_tokens, 128, 0, s, a);
     else if (dtype == VCB_BF16) vcb_launch(latent_rope_cache_write_kernel<__nv_bfloat16>, n_tokens, 128, 0, s, a);
     else return VCB_ERR_BAD_ARG;
     return vcb_last_error();
+}
+
+// Cosine and sine as they are.
+VCB_EXPORT int vcb_latent_rope_cache_write(const void* raw, int ld, const float* gain, void* q, int ldq, int heads, int q_stride,
+                                           int q_off, const float* inv_freq, int rot, int pairing, const int* positions,
+                                           const int* req_of_token, const int* block_table, int bt_stride, void* cache,
+                                           long long page_stride, int n_tokens, int rank, int page, float eps, int num_pages,
+                                           int write_kv, int* status, int dtype, void* stream) {
+    return vcb_latent_rope_cache_write_scaled(raw, ld, gain, q, ldq, heads, q_stride, q_off, inv_freq, rot, pairing, positions, req_of_token,
+                                              block_table, bt_stride, cache, page_stride, n_tokens, rank, page, eps, num_pages, write_kv, 1.0f,
+                                              status, dtype, stream);
 }

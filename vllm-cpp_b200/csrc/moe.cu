@@ -9,9 +9,11 @@
 //   moe_expert_gemm_kernel   one product per tile against that expert's matrix; the first product gathers the
 //                            tokens' rows, computes gate and up together and applies the experts' activation
 //                              g = min(gate, limit), u = clamp(up, -limit, limit), y = g * sigmoid(alpha * g) * (u + up_shift)
-//                            (limit = inf, alpha = 1, up_shift = 0: silu(gate) * up)
+//                            (limit = inf, alpha = 1, up_shift = 0: silu(gate) * up); or, for experts without a gate, one
+//                            matrix and y = gelu(s * x), gelu by its definition through erf and s a number per row: the
+//                            pair's weight, for designs in which it multiplies what the expert reads
 //   moe_combine_kernel       out[t] = sum over the token's choices of weight * (the expert's row, or h[t] itself for a
-//                            router output beyond the experts: an identity expert)
+//                            router output beyond the experts: an identity expert); without weights the plain sum
 //
 // Grids are sized for the most tiles a step can have; a block beyond the step's count leaves at once, so the
 // same launches serve every routing (and a captured step).  Router, softmax, weights and all sums are float.
@@ -224,8 +226,9 @@ VCB_EXPORT int vcb_moe_router(const void* h, long long ldh, const float* wr, con
 // --------------------------------------------------------------------------------------------- sort
 // One CTA.  ids: [pairs] router outputs; outputs >= n_experts are identity experts and get no row (pos = -1).
 // meta[0] = number of tiles.  Rows of one expert are in no particular order; every row is computed by itself.
-__global__ void moe_sort_kernel(const int* __restrict__ ids, int pairs, int top, int n_experts, int tm,
-                                int* __restrict__ sorted_token, int* __restrict__ pos, int* __restrict__ tile_expert,
+// wts, sorted_weight (both or neither): the pairs' weights in the order of the sorted rows.
+__global__ void moe_sort_kernel(const int* __restrict__ ids, const float* __restrict__ wts, float* __restrict__ sorted_weight, int pairs, int top,
+                                int n_experts, int tm, int* __restrict__ sorted_token, int* __restrict__ pos, int* __restrict__ tile_expert,
                                 int* __restrict__ tile_row0, int* __restrict__ tile_rows, int* __restrict__ meta) {
     extern __shared__ int smi[];
     int* count = smi;                   // [n_experts]
@@ -258,6 +261,7 @@ __global__ void moe_sort_kernel(const int* __restrict__ ids, int pairs, int top,
         if ((unsigned)e < (unsigned)n_experts) {
             const int dst = atomicAdd(&cursor[e], 1);
             sorted_token[dst] = p / top;
+            if (wts) sorted_weight[dst] = wts[p];
             pos[p] = dst;
         } else {
             pos[p] = -1;
@@ -265,29 +269,39 @@ __global__ void moe_sort_kernel(const int* __restrict__ ids, int pairs, int top,
     }
 }
 
+VCB_EXPORT int vcb_moe_sort_weighted(const int* ids, const float* wts, float* sorted_weight, int pairs, int top, int n_experts, int tm,
+                                     int* sorted_token, int* pos, int* tile_expert, int* tile_row0, int* tile_rows, int* meta, void* stream) {
+    if (pairs <= 0) return 0;
+    if (!wts != !sorted_weight || n_experts <= 0 || top <= 0 || tm <= 0 || (size_t)n_experts * 2 * sizeof(int) > 48 * 1024) return VCB_ERR_BAD_ARG;
+    vcb_launch(moe_sort_kernel, 1, 1024, (size_t)n_experts * 2 * sizeof(int), (cudaStream_t)stream, ids, wts, sorted_weight, pairs, top,
+               n_experts, tm, sorted_token, pos, tile_expert, tile_row0, tile_rows, meta);
+    return vcb_last_error();
+}
+
 VCB_EXPORT int vcb_moe_sort(const int* ids, int pairs, int top, int n_experts, int tm, int* sorted_token, int* pos,
                             int* tile_expert, int* tile_row0, int* tile_rows, int* meta, void* stream) {
-    if (pairs <= 0) return 0;
-    if (n_experts <= 0 || top <= 0 || tm <= 0 || (size_t)n_experts * 2 * sizeof(int) > 48 * 1024) return VCB_ERR_BAD_ARG;
-    vcb_launch(moe_sort_kernel, 1, 1024, (size_t)n_experts * 2 * sizeof(int), (cudaStream_t)stream, ids, pairs, top, n_experts,
-               tm, sorted_token, pos, tile_expert, tile_row0, tile_rows, meta);
-    return vcb_last_error();
+    return vcb_moe_sort_weighted(ids, nullptr, nullptr, pairs, top, n_experts, tm, sorted_token, pos, tile_expert, tile_row0, tile_rows, meta,
+                                 stream);
 }
 
 // ------------------------------------------------------------------------------------ expert products
 // C[row, n] = sum_k A[src(row), k] * W_e[n, k] for the rows of one tile, W_e the tile's expert's matrix.
-// GATED: W_e = [gate rows; up rows] ([2 * N, K]), rows are gathered through sorted_token, and C (type T) receives
-// the activation of (gate, up).  Otherwise A is the sorted list itself and C is float.
+// MG_GATED: W_e = [gate rows; up rows] ([2 * N, K]), rows are gathered through sorted_token, and C (type T) receives
+// the activation of (gate, up).  MG_GELU: W_e [N, K], rows gathered too, C (type T) = gelu(row_scale[row] * the sum).
+// MG_PLAIN: A is the sorted list itself and C is float.
 // 64 output columns per CTA, TM rows, 16-deep k slices in shared memory, float accumulation (FMA).
 #define MG_N 64
 #define MG_K 16
+enum { MG_PLAIN = 0, MG_GATED = 1, MG_GELU = 2 };
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 
-template <typename T, int TM, bool GATED>
+template <typename T, int TM, int MODE>
 __global__ void __launch_bounds__(256)
 moe_expert_gemm_kernel(const T* __restrict__ A, long long lda, const T* __restrict__ W, void* __restrict__ Cv, long long ldc,
                        int N, int K, const int* __restrict__ sorted_token, const int* __restrict__ tile_expert,
                        const int* __restrict__ tile_row0, const int* __restrict__ tile_rows, const int* __restrict__ meta,
-                       float limit, float alpha, float up_shift) {
+                       float limit, float alpha, float up_shift, const float* __restrict__ row_scale) {
+    constexpr bool GATED = MODE == MG_GATED, GATHER = MODE != MG_PLAIN;
     constexpr int RM = TM / 16;          // rows per thread
     __shared__ float As[MG_K][TM + 1];
     __shared__ float Ws[MG_K][MG_N + 1];
@@ -300,7 +314,7 @@ moe_expert_gemm_kernel(const T* __restrict__ A, long long lda, const T* __restri
     const int n0 = blockIdx.x * MG_N;
     const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
     const int me = (int)threadIdx.x;
-    if (me < TM) src[me] = me < rows ? (GATED ? sorted_token[r0 + me] : r0 + me) : -1;
+    if (me < TM) src[me] = me < rows ? (GATHER ? sorted_token[r0 + me] : r0 + me) : -1;
     __syncthreads();
     const T* We = W + (size_t)e * (GATED ? 2 : 1) * N * K;
     float acc[RM][4], accu[GATED ? RM : 1][4];
@@ -353,6 +367,8 @@ moe_expert_gemm_kernel(const T* __restrict__ A, long long lda, const T* __restri
                 const float u = fminf(fmaxf(accu[i][j], -limit), limit);
                 const float y = g * (1.0f / (1.0f + expf(-alpha * g))) * (u + up_shift);
                 ((T*)Cv)[(size_t)(r0 + m) * ldc + n] = from_f32<T>(y);
+            } else if (MODE == MG_GELU) {
+                ((T*)Cv)[(size_t)(r0 + m) * ldc + n] = from_f32<T>(gelu_erf(acc[i][j] * (row_scale ? row_scale[r0 + m] : 1.0f)));
             } else {
                 ((float*)Cv)[(size_t)(r0 + m) * ldc + n] = acc[i][j];
             }
@@ -385,12 +401,13 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <int TM, bool GATED>
+template <int TM, int MODE>
 __global__ void __launch_bounds__(128)
 moe_expert_mma_kernel(const __nv_bfloat16* __restrict__ A, long long lda, const __nv_bfloat16* __restrict__ W, void* __restrict__ Cv,
                       long long ldc, int N, int K, const int* __restrict__ sorted_token, const int* __restrict__ tile_expert,
                       const int* __restrict__ tile_row0, const int* __restrict__ tile_rows, const int* __restrict__ meta,
-                      float limit, float alpha, float up_shift) {
+                      float limit, float alpha, float up_shift, const float* __restrict__ row_scale) {
+    constexpr bool GATED = MODE == MG_GATED, GATHER = MODE != MG_PLAIN;
     constexpr int WR = GATED ? 2 * MM_BN : MM_BN, MF = TM / 16;
     __shared__ __align__(16) __nv_bfloat16 As[MM_STAGES][TM][MM_LDS];
     __shared__ __align__(16) __nv_bfloat16 Ws[MM_STAGES][WR][MM_LDS];
@@ -401,7 +418,7 @@ moe_expert_mma_kernel(const __nv_bfloat16* __restrict__ A, long long lda, const 
     const int e = tile_expert[tile], r0 = tile_row0[tile], rows = tile_rows[tile];
     const int n0 = blockIdx.x * MM_BN;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    if (tid < TM) src[tid] = tid < rows ? (GATED ? sorted_token[r0 + tid] : r0 + tid) : -1;
+    if (tid < TM) src[tid] = tid < rows ? (GATHER ? sorted_token[r0 + tid] : r0 + tid) : -1;
     __syncthreads();
     const __nv_bfloat16* We = W + (size_t)e * (GATED ? 2 : 1) * N * K;
     const int KT = (K + MM_BK - 1) / MM_BK;
@@ -474,42 +491,55 @@ moe_expert_mma_kernel(const __nv_bfloat16* __restrict__ A, long long lda, const 
                     const float u = fminf(fmaxf(accu[mi][nf][c], -limit), limit);
                     const float y = g * (1.0f / (1.0f + expf(-alpha * g))) * (u + up_shift);
                     ((__nv_bfloat16*)Cv)[(size_t)(r0 + m) * ldc + n] = __float2bfloat16_rn(y);
+                } else if (MODE == MG_GELU) {
+                    const float y = gelu_erf(acc[mi][nf][c] * (row_scale ? row_scale[r0 + m] : 1.0f));
+                    ((__nv_bfloat16*)Cv)[(size_t)(r0 + m) * ldc + n] = __float2bfloat16_rn(y);
                 } else {
                     ((float*)Cv)[(size_t)(r0 + m) * ldc + n] = acc[mi][nf][c];
                 }
             }
 }
 
-// gated 1: A = the tokens' rows [n, K] (T), W [E, 2 * N, K], C [pairs, N] (T).  gated 0: A [pairs, K] (T), W [E, N, K],
-// C [pairs, N] float.  max_tiles: the grid's height; tm: 16 or 64, the tile height moe_sort was given.
+// mode MG_GATED (1): A = the tokens' rows [n, K] (T), W [E, 2 * N, K], C [pairs, N] (T).  MG_GELU (2): A the tokens' rows, W [E,
+// N, K], C [pairs, N] (T), row_scale float [pairs] or null.  MG_PLAIN (0): A [pairs, K] (T), W [E, N, K], C [pairs, N] float.
+// max_tiles: the grid's height; tm: 16 or 64, the tile height moe_sort was given.
+VCB_EXPORT int vcb_moe_expert_gemm_as(const void* A, long long lda, const void* W, void* C, long long ldc, int N, int K,
+                                      const int* sorted_token, const int* tile_expert, const int* tile_row0, const int* tile_rows,
+                                      const int* meta, int max_tiles, int tm, int mode, float limit, float alpha, float up_shift,
+                                      const float* row_scale, int dtype, void* stream) {
+    if (max_tiles <= 0) return 0;
+    if (!A || !W || !C || N <= 0 || K <= 0 || (tm != 16 && tm != 64) || max_tiles > 65535 || mode < MG_PLAIN || mode > MG_GELU) return VCB_ERR_BAD_ARG;
+    dim3 grid((N + MG_N - 1) / MG_N, max_tiles);
+    cudaStream_t s = (cudaStream_t)stream;
+#define MOE_LIST C, ldc, N, K, sorted_token, tile_expert, tile_row0, tile_rows, meta, limit, alpha, up_shift, row_scale
+#define MOE_MODES(GO, TMV) do { if (mode == MG_GATED) GO(TMV, MG_GATED); else if (mode == MG_GELU) GO(TMV, MG_GELU); else GO(TMV, MG_PLAIN); } while (0)
+    if (dtype == VCB_BF16 && K % 8 == 0 && lda % 8 == 0 && !(((uintptr_t)A | (uintptr_t)W) & 15)) {
+        // the tensor-core form
+#define MOE_MMA(TMV, M) vcb_launch(moe_expert_mma_kernel<TMV, M>, grid, 128, 0, s, (const __nv_bfloat16*)A, lda, (const __nv_bfloat16*)W, MOE_LIST)
+        if (tm == 16) MOE_MODES(MOE_MMA, 16);
+        else MOE_MODES(MOE_MMA, 64);
+#undef MOE_MMA
+        return vcb_last_error();
+    }
+#define MOE_F32(TMV, M) vcb_launch(moe_expert_gemm_kernel<float, TMV, M>, grid, 256, 0, s, (const float*)A, lda, (const float*)W, MOE_LIST)
+#define MOE_BF16(TMV, M) vcb_launch(moe_expert_gemm_kernel<__nv_bfloat16, TMV, M>, grid, 256, 0, s, (const __nv_bfloat16*)A, lda, (const __nv_bfloat16*)W, MOE_LIST)
+    if (dtype == VCB_F32) { if (tm == 16) MOE_MODES(MOE_F32, 16); else MOE_MODES(MOE_F32, 64); }
+    else if (dtype == VCB_BF16) { if (tm == 16) MOE_MODES(MOE_BF16, 16); else MOE_MODES(MOE_BF16, 64); }
+    else return VCB_ERR_BAD_ARG;
+#undef MOE_F32
+#undef MOE_BF16
+#undef MOE_MODES
+#undef MOE_LIST
+    return vcb_last_error();
+}
+
+// Gated experts' first product, or the second product of any.
 VCB_EXPORT int vcb_moe_expert_gemm(const void* A, long long lda, const void* W, void* C, long long ldc, int N, int K,
                                    const int* sorted_token, const int* tile_expert, const int* tile_row0, const int* tile_rows,
                                    const int* meta, int max_tiles, int tm, int gated, float limit, float alpha, float up_shift,
                                    int dtype, void* stream) {
-    if (max_tiles <= 0) return 0;
-    if (!A || !W || !C || N <= 0 || K <= 0 || (tm != 16 && tm != 64) || max_tiles > 65535) return VCB_ERR_BAD_ARG;
-    dim3 grid((N + MG_N - 1) / MG_N, max_tiles);
-    cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == VCB_BF16 && K % 8 == 0 && lda % 8 == 0 && !(((uintptr_t)A | (uintptr_t)W) & 15)) {
-        // the tensor-core form
-#define MOE_MMA(TMV, G) vcb_launch(moe_expert_mma_kernel<TMV, G>, grid, 128, 0, s, (const __nv_bfloat16*)A, lda, (const __nv_bfloat16*)W, C, ldc, N, K, \
-                                   sorted_token, tile_expert, tile_row0, tile_rows, meta, limit, alpha, up_shift)
-        if (tm == 16) { if (gated) MOE_MMA(16, true); else MOE_MMA(16, false); }
-        else { if (gated) MOE_MMA(64, true); else MOE_MMA(64, false); }
-#undef MOE_MMA
-        return vcb_last_error();
-    }
-#define MOE_GO(TT, TMV, G) vcb_launch(moe_expert_gemm_kernel<TT, TMV, G>, grid, 256, 0, s, (const TT*)A, lda, (const TT*)W, C, ldc, N, K, \
-                                      sorted_token, tile_expert, tile_row0, tile_rows, meta, limit, alpha, up_shift)
-    if (dtype == VCB_F32) {
-        if (tm == 16) { if (gated) MOE_GO(float, 16, true); else MOE_GO(float, 16, false); }
-        else { if (gated) MOE_GO(float, 64, true); else MOE_GO(float, 64, false); }
-    } else if (dtype == VCB_BF16) {
-        if (tm == 16) { if (gated) MOE_GO(__nv_bfloat16, 16, true); else MOE_GO(__nv_bfloat16, 16, false); }
-        else { if (gated) MOE_GO(__nv_bfloat16, 64, true); else MOE_GO(__nv_bfloat16, 64, false); }
-    } else return VCB_ERR_BAD_ARG;
-#undef MOE_GO
-    return vcb_last_error();
+    return vcb_moe_expert_gemm_as(A, lda, W, C, ldc, N, K, sorted_token, tile_expert, tile_row0, tile_rows, meta, max_tiles, tm,
+                                  gated ? MG_GATED : MG_PLAIN, limit, alpha, up_shift, nullptr, dtype, stream);
 }
 
 // ------------------------------------------------------------------------------------------ combine
@@ -523,7 +553,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const T* __restr
         float acc = add ? to_f32<T>(add[(size_t)t * lda + i]) : 0.0f;      // what every token takes beside its choices (a shared expert)
         for (int k = 0; k < top; ++k) {
             const int p = pos[(size_t)t * top + k];
-            const float w = wts[(size_t)t * top + k];
+            const float w = wts ? wts[(size_t)t * top + k] : 1.0f;
             acc += w * (p >= 0 ? y[(size_t)p * width + i] : to_f32<T>(h[(size_t)t * ldh + i]));
         }
         out[(size_t)t * width + i] = from_f32<T>(acc);
@@ -533,7 +563,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const T* __restr
 VCB_EXPORT int vcb_moe_combine_add(const float* y, const void* h, long long ldh, const int* pos, const float* wts, void* out,
                                    int n_tokens, int width, int top, const void* add, long long lda, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
-    if (!y || !h || !pos || !wts || !out || width <= 0 || top <= 0) return VCB_ERR_BAD_ARG;
+    if (!y || !h || !pos || !out || width <= 0 || top <= 0) return VCB_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = width >= 1024 ? 256 : 128;
     if (dtype == VCB_F32) vcb_launch(moe_combine_kernel<float>, n_tokens, threads, 0, s, y, (const float*)h, ldh, pos, wts, (float*)out, width, top, (const float*)add, lda);

@@ -99,6 +99,19 @@ _SIGNATURES = {
     "vcb_gate_blocks": [_P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _F, _I, _P],
     "vcb_linear_recurrence": [_P, _P, _L, _P, _L, _P, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _P],
     "vcb_gated_delta_scan": [_P, _P, _P, _L, _L, _L, _P, _L, _P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _P, _I, _P],
+    "vcb_add_tanh_norm": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _F, _I, _P],
+    "vcb_act_rows": [_P, _P, _L, _I, _I, _P],
+    "vcb_state_dual": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+    "vcb_qk_norm_cache_write_temp": [_P, _L, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _I, _P],
+    "vcb_attention_biased_kept": [_P, _P, _P, _P, _L, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _P, _I, _I, _P],
+    "vcb_attention_simt_sink": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _I, _P],
+    "vcb_latent_rope_cache_write_scaled": [_P, _I, _P, _P, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _I, _P, _L, _I, _I, _I, _F, _I, _I, _F, _P, _I, _P],
+    "vcb_gated_group_norm_as": [_P, _L, _P, _L, _P, _I, _P, _L, _I, _I, _I, _I, _I, _F, _I, _P],
+    "vcb_attention_decode_mma_shaped_kept": [_P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _F, _P, _I,
+                                             _P, _P, _L, _I, _I, _I, _P],
+    "vcb_attention_prefill_tc_shaped_kept": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _F, _P, _I, _P, _P, _L, _I, _I, _I, _P],
+    "vcb_moe_sort_weighted": [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P],
+    "vcb_moe_expert_gemm_as": [_P, _L, _P, _P, _L, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _F, _F, _F, _P, _I, _P],
     "vcb_moe_sort": [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P],
     "vcb_moe_expert_gemm": [_P, _L, _P, _P, _L, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _F, _F, _F, _I, _P],
     "vcb_moe_combine": [_P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _P],
@@ -247,6 +260,29 @@ def relu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
                               dtype_code(out.dtype), _stream()), "relu_mul")
 
 
+def add_tanh_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], alpha: torch.Tensor, gain: torch.Tensor, shift: torch.Tensor,
+                  out: torch.Tensor, row_index: Optional[torch.Tensor] = None, mult: float = 1.0) -> None:
+    """out = tanh(alpha * (residual + mult * delta)) * gain + shift; the sum is written back to residual unless rows are gathered.
+    alpha float32 [1], gain and shift float32 [hidden]."""
+    hidden, n_rows = residual.shape[1], out.shape[0]
+    _need(out.shape[1] == hidden and gain.numel() == hidden and shift.numel() == hidden and alpha.numel() == 1, "add_tanh_norm: widths differ")
+    _need(delta is None or (delta.shape == residual.shape and delta.dtype == out.dtype), "add_tanh_norm: delta shape or type differs")
+    _need(n_rows == residual.shape[0] if row_index is None else row_index.numel() == n_rows, "add_tanh_norm: one row read per output row")
+    _check(lib().vcb_add_tanh_norm(_dev(residual, "residual", torch.float32), None if delta is None else _dev(delta, "delta"),
+                                   _dev(alpha, "alpha", torch.float32), _dev(gain, "gain", torch.float32), _dev(shift, "shift", torch.float32),
+                                   _dev(out, "out"), None if row_index is None else _dev(row_index, "row_index", torch.int32), n_rows, hidden,
+                                   float(mult), dtype_code(out.dtype), _stream()), "add_tanh_norm")
+
+
+ROW_ACTS = {"relu_squared": 0, "gelu": 1}      # gelu by its definition, through erf
+
+
+def act_rows(x: torch.Tensor, out: torch.Tensor, act: str) -> None:
+    """out = act(x) element by element, evaluated in float (out may be x)."""
+    _need(x.shape == out.shape and x.dtype == out.dtype and act in ROW_ACTS, f"act_rows: one shape, one type, act one of {sorted(ROW_ACTS)}")
+    _check(lib().vcb_act_rows(_dev(x, "x"), _dev(out, "out"), x.numel(), ROW_ACTS[act], dtype_code(x.dtype), _stream()), "act_rows")
+
+
 def cast_rows(x: torch.Tensor, delta: Optional[torch.Tensor], mult: float, out: torch.Tensor) -> None:
     """out = x + mult * delta (float; ``delta`` None: x itself) rounded to out's type; x float32 [n, width] contiguous,
     delta contiguous of out's type, out rows may be strided.  x is left as it is."""
@@ -306,20 +342,23 @@ SIMT_MAX_HEAD_DIM = 1024
 
 
 def attention_simt(q, cache, out, positions, req_of_token, block_table, *, num_heads: int,
-                   num_kv_heads: int, head_dim: int, page_size: int, window: int, scale: float, planes: int = 2) -> None:
+                   num_kv_heads: int, head_dim: int, page_size: int, window: int, scale: float, planes: int = 2,
+                   sink: Optional[torch.Tensor] = None) -> None:
     """Plain paged attention.  ``planes`` 2: a page holds keys, then values; 1: one plane of rows that serve
-    as key and as value (cached latent rows)."""
+    as key and as value (cached latent rows).  ``sink`` (float32 [heads]): a logit per head that joins the denominator once."""
     n = q.shape[0]
     _need(head_dim <= SIMT_MAX_HEAD_DIM, f"head_dim {head_dim} exceeds {SIMT_MAX_HEAD_DIM}, the largest this attention kernel takes")
     _need(planes in (1, 2), "planes must be 1 or 2")
     _need(q.shape == (n, num_heads * head_dim) and out.shape == q.shape and out.dtype == q.dtype, "q/out shape")
     _need(num_heads % num_kv_heads == 0, "num_heads must be a multiple of num_kv_heads")
     _need(cache.dtype == q.dtype, "cache and q must share a storage type")
-    _check(lib().vcb_attention_simt_planes(
+    _need(sink is None or sink.numel() == num_heads, "attention_simt: one sink per head")
+    _check(lib().vcb_attention_simt_sink(
         _dev(q, "q"), _dev(cache, "cache"), _dev(out, "out"), _dev(positions, "positions", torch.int32),
         _dev(req_of_token, "req_of_token", torch.int32), _dev(block_table, "block_table", torch.int32),
         block_table.shape[1], n, num_heads, num_kv_heads, head_dim, page_size, window, float(scale),
-        cache.shape[0], status_tensor(q.device).data_ptr(), planes, dtype_code(q.dtype), _stream()), "attention_simt")
+        cache.shape[0], status_tensor(q.device).data_ptr(), planes, None if sink is None else _dev(sink, "sink", torch.float32),
+        dtype_code(q.dtype), _stream()), "attention_simt")
 
 
 MMA_HEAD_DIMS = (64, 128)
@@ -342,13 +381,14 @@ def attention_decode_mma(q, cache, out, q_start, ctx_lens, block_table, req_list
                          part_o, part_ml, counters, *, num_heads: int, num_kv_heads: int, head_dim: int, page_size: int,
                          window: int, scale: float, split_tiles=None, planes: int = 2, kv_share: int = 1,
                          cap: float = 0.0, bias_t: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
-                         head_gate: Optional[torch.Tensor] = None, precise_weights: bool = False) -> None:
+                         head_gate: Optional[torch.Tensor] = None, precise_weights: bool = False, keep_first: int = 0) -> None:
     """Split-KV tensor-core attention for requests that bring one token each (bfloat16).  The grid has
     ``nsplit`` columns; without ``split_tiles`` every request's keys are cut into that many equal parts,
     with it (int32 [1] on the device: tiles of DECODE_KEY_TILE keys per split) a request takes as many
     columns as its context needs, so that requests of different lengths keep all CTAs equally busy.
     ``kv_share`` > 1: ``num_kv_heads`` counts groups of query heads of which ``kv_share`` consecutive ones read the
-    same head of the cache (decode_head_groups): each group gets CTAs of its own."""
+    same head of the cache (decode_head_groups): each group gets CTAs of its own.  ``keep_first`` > 0 with a window: the
+    sequence's first tokens are seen wherever the window is."""
     _need(q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
           "attention_decode_mma is a bfloat16 kernel")
     _need(head_dim in MMA_HEAD_DIMS and page_size % 8 == 0,
@@ -360,13 +400,13 @@ def attention_decode_mma(q, cache, out, q_start, ctx_lens, block_table, req_list
               "attention_decode_mma: scratch for the split merge is too small")
     _need(planes in (1, 2), "planes must be 1 or 2")
     _need(kv_share >= 1 and num_kv_heads % kv_share == 0, "attention_decode_mma: kv_share divides num_kv_heads")
-    if cap > 0 or bias_t is not None or sink is not None or head_gate is not None or precise_weights:
+    if cap > 0 or bias_t is not None or sink is not None or head_gate is not None or precise_weights or keep_first:
         # ``precise_weights``: the softmax weights enter the P V product as two bfloat16 terms (16 bits of mantissa)
         # shaped scores: cap * tanh(scale * q.k / cap) + bias_t[head, min(distance, last)]; the epilogue: a sink logit per
         # head in the denominator, the head's output times sigmoid(head_gate[token, head]) (see attention_mma.cu)
         _need(bias_t is None or (bias_t.dim() == 2 and bias_t.shape[0] == num_heads), "attention_decode_mma: bias_t [heads, distances]")
         _epilogue_args(sink, head_gate, q.shape[0], num_heads, "attention_decode_mma")
-        _check(lib().vcb_attention_decode_mma_shaped_planes(
+        _check(lib().vcb_attention_decode_mma_shaped_kept(
             _dev(q, "q"), _dev(cache, "cache"), _dev(out, "out"), _dev(q_start, "q_start", torch.int32),
             _dev(ctx_lens, "ctx_lens", torch.int32), _dev(block_table, "block_table", torch.int32),
             block_table.shape[1], None if req_list is None else _dev(req_list, "req_list", torch.int32),
@@ -377,7 +417,7 @@ def attention_decode_mma(q, cache, out, q_start, ctx_lens, block_table, req_list
             num_heads, num_kv_heads, head_dim, page_size, window, float(scale), cache.shape[0],
             status_tensor(q.device).data_ptr(), kv_share, float(cap),
             None if bias_t is None else _dev(bias_t, "bias_t", torch.float32), 0 if bias_t is None else bias_t.shape[1],
-            *_epilogue_ptrs(sink, head_gate), 1 if precise_weights else 0, planes, _stream()), "attention_decode_mma")
+            *_epilogue_ptrs(sink, head_gate), 1 if precise_weights else 0, planes, int(keep_first), _stream()), "attention_decode_mma")
         return
     _check(lib().vcb_attention_decode_mma_planes(
         _dev(q, "q"), _dev(cache, "cache"), _dev(out, "out"), _dev(q_start, "q_start", torch.int32),
@@ -410,9 +450,11 @@ def attention_prefill_tc(q, cache, out, q_start, ctx_lens, block_table, tile_req
                          num_heads: int, num_kv_heads: int, head_dim: int, page_size: int, window: int,
                          scale: float, planes: int = 2, cap: float = 0.0, bias_t: Optional[torch.Tensor] = None,
                          sink: Optional[torch.Tensor] = None, head_gate: Optional[torch.Tensor] = None,
-                         precise_weights: bool = False) -> None:
+                         precise_weights: bool = False, keep_first: int = 0) -> None:
     """Attention for portions of any length on tcgen05 tensor cores (scores and output tiles in tensor
-    memory); head sizes 64 and 128, bfloat16, pages of a multiple of 8 slots, tiles of 128 packed rows."""
+    memory); head sizes 64 and 128, bfloat16, pages of a multiple of 8 slots, tiles of 128 packed rows.  ``keep_first`` as in
+    attention_decode_mma, with two-term weights only."""
+    _need(not keep_first or precise_weights, "attention_prefill_tc: kept first tokens come with two-term weights")
     _need(q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
           "attention_prefill_tc is a bfloat16 kernel")
     _need(head_dim in TC_ATTENTION_HEAD_DIMS and page_size % 8 == 0,
@@ -420,16 +462,16 @@ def attention_prefill_tc(q, cache, out, q_start, ctx_lens, block_table, tile_req
     n_tiles = tile_req.numel()
     _need(tile_row0.numel() == n_tiles, "one first row per tile")
     _need(planes in (1, 2), "planes must be 1 or 2")
-    if cap > 0 or bias_t is not None or sink is not None or head_gate is not None or precise_weights:
+    if cap > 0 or bias_t is not None or sink is not None or head_gate is not None or precise_weights or keep_first:
         _need(bias_t is None or (bias_t.dim() == 2 and bias_t.shape[0] == num_heads), "attention_prefill_tc: bias_t [heads, distances]")
         _epilogue_args(sink, head_gate, q.shape[0], num_heads, "attention_prefill_tc")
-        _check(lib().vcb_attention_prefill_tc_shaped_planes(
+        _check(lib().vcb_attention_prefill_tc_shaped_kept(
             _dev(q, "q"), _dev(cache, "cache"), _dev(out, "out"), _dev(q_start, "q_start", torch.int32),
             _dev(ctx_lens, "ctx_lens", torch.int32), _dev(block_table, "block_table", torch.int32),
             block_table.shape[1], _dev(tile_req, "tile_req", torch.int32), _dev(tile_row0, "tile_row0", torch.int32),
             n_tiles, num_heads, num_kv_heads, head_dim, page_size, window, float(scale), cache.shape[0],
             status_tensor(q.device).data_ptr(), float(cap), None if bias_t is None else _dev(bias_t, "bias_t", torch.float32),
-            0 if bias_t is None else bias_t.shape[1], *_epilogue_ptrs(sink, head_gate), 1 if precise_weights else 0, planes, _stream()), "attention_prefill_tc")
+            0 if bias_t is None else bias_t.shape[1], *_epilogue_ptrs(sink, head_gate), 1 if precise_weights else 0, planes, int(keep_first), _stream()), "attention_prefill_tc")
         return
     _check(lib().vcb_attention_prefill_tc_planes(
         _dev(q, "q"), _dev(cache, "cache"), _dev(out, "out"), _dev(q_start, "q_start", torch.int32),
@@ -1045,21 +1087,23 @@ def scan_pieces(q_lens):
 
 
 def gated_group_norm(o: torch.Tensor, gate: Optional[torch.Tensor], weight: torch.Tensor, out: torch.Tensor, *, group: int,
-                     eps: float, gate_act: str = "sigmoid") -> None:
-    """out = o / sqrt(mean over each group of ``group`` channels of o^2 + eps) * weight[channel % len(weight)] * act(gate);
+                     eps: float, gate_act: str = "sigmoid", gate_first: bool = False) -> None:
+    """out = o / sqrt(mean over each group of ``group`` channels of o^2 + eps) * weight[channel % len(weight)] * act(gate); with
+    ``gate_first`` the gate comes before the norm, o * act(gate) taking the place of o;
     o float32 [n, C], gate and out rows of the activations' type, act "sigmoid" or "silu"."""
     n, C = o.shape
     _rows(o, "o", torch.float32)
     _rows(out, "out", out.dtype)
     _need(out.shape == o.shape and (C % group == 0) and weight.numel() in (group, C), "gated_group_norm: shapes")
     _need(gate_act in ("sigmoid", "silu"), "gated_group_norm: gate_act is 'sigmoid' or 'silu'")
+    _need(gate is not None or not gate_first, "gated_group_norm: gate_first needs a gate")
     if gate is not None:
         _rows(gate, "gate", out.dtype)
         _need(gate.shape == o.shape, "gated_group_norm: gate like o")
-    _check(lib().vcb_gated_group_norm(o.data_ptr(), o.stride(0), None if gate is None else gate.data_ptr(),
+    _check(lib().vcb_gated_group_norm_as(o.data_ptr(), o.stride(0), None if gate is None else gate.data_ptr(),
                                       0 if gate is None else gate.stride(0), _dev(weight, "weight", torch.float32),
                                       weight.numel(), out.data_ptr(), out.stride(0), n, C, group,
-                                      1 if gate_act == "silu" else 0, float(eps), dtype_code(out.dtype), _stream()),
+                                      1 if gate_act == "silu" else 0, 1 if gate_first else 0, float(eps), dtype_code(out.dtype), _stream()),
            "gated_group_norm")
 
 
@@ -1074,36 +1118,39 @@ def scaled_sum(x: torch.Tensor, y: torch.Tensor, out: torch.Tensor, a: float, b:
 def qk_norm_cache_write(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, wq: Optional[torch.Tensor],
                         wk: Optional[torch.Tensor], q_out: torch.Tensor, cache: torch.Tensor, positions, req_of_token,
                         block_table, *, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int, row: int,
-                        page_size: int, eps: float, write_kv: bool) -> None:
+                        page_size: int, eps: float, write_kv: bool, temperature=None) -> None:
     """A token's row of ``proj`` holds its query projection at ``q_off`` (heads * head_dim), key projection at ``k_off``
     (kv heads * head_dim) and values at ``v_off`` (kv heads * v_head_dim).  Queries and keys are RMS-normed over the whole
     projection with the gains ``wq`` / ``wk`` (None: left as they are); queries go to ``q_out``, keys and values into
-    the token's slot of the cache, whose rows are ``row`` elements wide."""
+    the token's slot of the cache, whose rows are ``row`` elements wide.  ``temperature`` (coef, every): the queries of position
+    p are multiplied by 1 + coef * ln((p + 1) // every + 1)."""
     n = proj.shape[0]
     _rows(proj, "proj", proj.dtype)
+    coef, every = (0.0, 0) if temperature is None else temperature
+    _need(temperature is None or every > 0, "qk_norm_cache_write: the temperature's step must be positive")
     _need(q_out.shape == (n, num_heads * head_dim) and q_out.dtype == proj.dtype and cache.dtype == proj.dtype, "qk_norm_cache_write: types")
     _need(wq is None or wq.numel() == num_heads * head_dim, "qk_norm_cache_write: one query gain per channel")
     _need(wk is None or wk.numel() == num_kv_heads * head_dim, "qk_norm_cache_write: one key gain per channel")
     _need(cache.is_contiguous() and cache.numel() == cache.shape[0] * 2 * num_kv_heads * page_size * row,
           "qk_norm_cache_write: a cache of key and value planes with rows of `row` elements")
-    _check(lib().vcb_qk_norm_cache_write(
+    _check(lib().vcb_qk_norm_cache_write_temp(
         proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, None if wq is None else _dev(wq, "wq", torch.float32),
         None if wk is None else _dev(wk, "wk", torch.float32), _dev(q_out, "q_out"), cache.data_ptr(),
         _dev(positions, "positions", torch.int32), _dev(req_of_token, "req_of_token", torch.int32),
         _dev(block_table, "block_table", torch.int32), block_table.shape[1], n, num_heads, num_kv_heads, head_dim,
-        v_head_dim, row, page_size, cache.shape[0], 1 if write_kv else 0, float(eps), status_tensor(proj.device).data_ptr(),
-        dtype_code(proj.dtype), _stream()), "qk_norm_cache_write")
+        v_head_dim, row, page_size, cache.shape[0], 1 if write_kv else 0, float(eps), float(coef), int(every),
+        status_tensor(proj.device).data_ptr(), dtype_code(proj.dtype), _stream()), "qk_norm_cache_write")
 
 
 def attention_biased(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor], positions,
                      req_of_token, block_table, bias: Optional[torch.Tensor], *, num_heads: int, num_kv_heads: int,
                      head_dim: int, v_head_dim: int, row: int, page_size: int, window: int, scale: float, cap: float,
-                     sink: Optional[torch.Tensor] = None, gate_per_head: bool = False) -> None:
+                     sink: Optional[torch.Tensor] = None, gate_per_head: bool = False, keep_first: int = 0) -> None:
     """Paged attention with  score = cap * tanh(scale * q.k / cap) + bias[min(distance, len(bias) - 1), head]  (cap <= 0: no
     cap; bias float32 [distances, heads] or None), softmax over the keys the window leaves, values of ``v_head_dim``,
     and out *= sigmoid(gate) when a gate is given ([n, heads * v_head_dim] rows, or with ``gate_per_head`` [n, heads]: one
     number per head).  ``sink`` (float32 [heads]): a logit per head that joins the softmax's denominator once, unscaled,
-    and has no value."""
+    and has no value.  ``keep_first`` > 0 with a window: the sequence's first tokens are seen wherever the window is."""
     n = q.shape[0]
     _need(q.shape == (n, num_heads * head_dim) and out.shape == (n, num_heads * v_head_dim) and out.dtype == q.dtype
           and cache.dtype == q.dtype, "attention_biased: shapes or types")
@@ -1114,12 +1161,12 @@ def attention_biased(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, ga
     _need(sink is None or sink.numel() == num_heads, "attention_biased: one sink per head")
     if bias is not None:
         _need(bias.dim() == 2 and bias.shape[1] == num_heads, "attention_biased: bias [distances, heads]")
-    _check(lib().vcb_attention_biased(
+    _check(lib().vcb_attention_biased_kept(
         _dev(q, "q"), _dev(cache, "cache"), _dev(out, "out"), None if gate is None else gate.data_ptr(),
         0 if gate is None else gate.stride(0), _dev(positions, "positions", torch.int32),
         _dev(req_of_token, "req_of_token", torch.int32), _dev(block_table, "block_table", torch.int32), block_table.shape[1],
         None if bias is None else _dev(bias, "bias", torch.float32), 0 if bias is None else bias.shape[0], n, num_heads,
-        num_kv_heads, head_dim, v_head_dim, row, page_size, window, float(scale), float(cap), cache.shape[0],
+        num_kv_heads, head_dim, v_head_dim, row, page_size, window, int(keep_first), float(scale), float(cap), cache.shape[0],
         status_tensor(q.device).data_ptr(), None if sink is None else _dev(sink, "sink", torch.float32),
         1 if gate_per_head else 0, dtype_code(q.dtype), _stream()), "attention_biased")
 
@@ -1199,39 +1246,47 @@ def moe_router(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[tor
     add_launches(1)                # logits and selection
 
 
-def moe_sort(ids: torch.Tensor, n_experts: int, tm: int, sorted_token, pos, tile_expert, tile_row0, tile_rows, meta) -> None:
-    """Groups the (token, choice) pairs of ``ids`` [n, top] by expert (see moe.cu); outputs >= n_experts get pos -1."""
+def moe_sort(ids: torch.Tensor, n_experts: int, tm: int, sorted_token, pos, tile_expert, tile_row0, tile_rows, meta,
+             weights: Optional[torch.Tensor] = None, sorted_weight: Optional[torch.Tensor] = None) -> None:
+    """Groups the (token, choice) pairs of ``ids`` [n, top] by expert (see moe.cu); outputs >= n_experts get pos -1.  With
+    ``weights`` [n, top], ``sorted_weight`` [pairs] receives them in the order of the sorted rows."""
     n, top = ids.shape
+    _need((weights is None) == (sorted_weight is None), "moe_sort: weights and where they go")
+    _need(weights is None or (weights.shape == ids.shape and sorted_weight.numel() >= n * top), "moe_sort: a weight per pair")
+    opt = lambda t, name: None if t is None else _dev(t, name, torch.float32)
     for t, name in ((sorted_token, "sorted_token"), (pos, "pos"), (tile_expert, "tile_expert"), (tile_row0, "tile_row0"),
                     (tile_rows, "tile_rows"), (meta, "meta")):
         _dev(t, name, torch.int32)
     _need(sorted_token.numel() >= n * top and pos.numel() >= n * top, "moe_sort: a row per pair")
     _need(tile_expert.numel() >= moe_max_tiles(n, top, n_experts, tm), "moe_sort: room for every tile")
-    _check(lib().vcb_moe_sort(_dev(ids, "ids", torch.int32), n * top, top, n_experts, tm, sorted_token.data_ptr(), pos.data_ptr(),
+    _check(lib().vcb_moe_sort_weighted(_dev(ids, "ids", torch.int32), opt(weights, "weights"), opt(sorted_weight, "sorted_weight"), n * top, top, n_experts, tm, sorted_token.data_ptr(), pos.data_ptr(),
                               tile_expert.data_ptr(), tile_row0.data_ptr(), tile_rows.data_ptr(), meta.data_ptr(), _stream()),
            "moe_sort")
 
 
 def moe_expert_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, sorted_token, tile_expert, tile_row0, tile_rows, meta,
-                    max_tiles: int, tm: int, *, gated: bool, limit: float = 0.0, alpha: float = 0.0, up_shift: float = 1.0) -> None:
+                    max_tiles: int, tm: int, *, gated: bool, limit: float = 0.0, alpha: float = 0.0, up_shift: float = 1.0,
+                    gelu: bool = False, row_scale: Optional[torch.Tensor] = None) -> None:
     """The experts' products over the tiles of moe_sort.  gated: a [n, K] the tokens' rows, w [E, 2 * N, K] gate rows then
     up rows, out [pairs, N] of the activations' type = g * sigmoid(alpha * g) * (u + up_shift) with g = min(gate, limit),
-    u = clamp(up, -limit, limit) (limit inf, alpha 1, up_shift 0: silu(gate) * up).  Not gated: a [pairs, K] the sorted
-    rows, w [E, N, K], out [pairs, N] float32."""
+    u = clamp(up, -limit, limit) (limit inf, alpha 1, up_shift 0: silu(gate) * up).  ``gelu``: a the tokens'
+    rows, w [E, N, K], out [pairs, N] of the activations' type = gelu(row_scale[row] * sum) (row_scale float32 [pairs] in sorted
+    order, or None).  Neither: a [pairs, K] the sorted rows, w [E, N, K], out [pairs, N] float32."""
+    _need(not (gated and gelu) and (row_scale is None or gelu), "moe_expert_gemm: gated or gelu; a row's factor comes with gelu")
     _rows(a, "a", a.dtype)
     _need(w.dim() == 3 and w.is_contiguous() and w.dtype == a.dtype and w.shape[2] == a.shape[1], "moe_expert_gemm: w [E, N, K]")
     N = w.shape[1] // 2 if gated else w.shape[1]
-    _rows(out, "out", a.dtype if gated else torch.float32)
+    _rows(out, "out", a.dtype if gated or gelu else torch.float32)
     _need(out.shape[1] == N and tm in MOE_TILE_ROWS, "moe_expert_gemm: out [pairs, N]")
-    _check(lib().vcb_moe_expert_gemm(a.data_ptr(), a.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0), N, a.shape[1],
+    _check(lib().vcb_moe_expert_gemm_as(a.data_ptr(), a.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0), N, a.shape[1],
                                      sorted_token.data_ptr(), tile_expert.data_ptr(), tile_row0.data_ptr(), tile_rows.data_ptr(),
-                                     meta.data_ptr(), max_tiles, tm, 1 if gated else 0, float(limit), float(alpha), float(up_shift),
-                                     dtype_code(a.dtype), _stream()), "moe_expert_gemm")
+                                     meta.data_ptr(), max_tiles, tm, 2 if gelu else 1 if gated else 0, float(limit), float(alpha), float(up_shift),
+                                     None if row_scale is None else _dev(row_scale, "row_scale", torch.float32), dtype_code(a.dtype), _stream()), "moe_expert_gemm")
 
 
-def moe_combine(y: torch.Tensor, h: torch.Tensor, pos: torch.Tensor, weights: torch.Tensor, out: torch.Tensor,
+def moe_combine(y: torch.Tensor, h: torch.Tensor, pos: torch.Tensor, weights: Optional[torch.Tensor], out: torch.Tensor,
                 add: Optional[torch.Tensor] = None) -> None:
-    """out[t] = sum_k weights[t, k] * (y[pos[t, k]] if pos[t, k] >= 0 else h[t]) (+ add[t]: what every token takes beside
+    """out[t] = sum_k weights[t, k] (None: 1) * (y[pos[t, k]] if pos[t, k] >= 0 else h[t]) (+ add[t]: what every token takes beside
     its choices, rows of out's type); y float32 [pairs, width]."""
     n, width = out.shape
     _rows(h, "h", out.dtype)
@@ -1240,7 +1295,7 @@ def moe_combine(y: torch.Tensor, h: torch.Tensor, pos: torch.Tensor, weights: to
         _rows(add, "add", out.dtype)
         _need(add.shape == out.shape, "moe_combine: add like out")
     _check(lib().vcb_moe_combine_add(y.data_ptr(), h.data_ptr(), h.stride(0), _dev(pos, "pos", torch.int32),
-                                     _dev(weights, "weights", torch.float32), _dev(out, "out"), n, width, weights.shape[1],
+                                     None if weights is None else _dev(weights, "weights", torch.float32), _dev(out, "out"), n, width, pos.numel() // n,
                                      None if add is None else add.data_ptr(), 0 if add is None else add.stride(0),
                                      dtype_code(out.dtype), _stream()), "moe_combine")
 
@@ -1531,6 +1586,34 @@ def selective_scan(x: torch.Tensor, dt_pre: torch.Tensor, b: torch.Tensor, c: to
                                     n_reqs, max_q_len, I, N, dtype_code(x.dtype), _stream()), "selective_scan")
 
 
+STATE_DUAL_MAX_STATE = 512
+
+
+def state_dual(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, dt_pre: torch.Tensor, dt_bias: torch.Tensor, a_log2: torch.Tensor,
+               d: torch.Tensor, state: torch.Tensor, y: torch.Tensor, q_start, state_slots, n_reqs: int, max_q_len: int, *, num_groups: int,
+               walk: bool = False) -> None:
+    """Per request and head h over the step's tokens, S (float32 [N, P]) read from and left in the request's slot of ``state``
+    [slots, H, N, P]:  dt = softplus(dt_pre + dt_bias);  S <- 2^(dt * a_log2[h]) S + B (dt x)^T;  y = S^T C + d[h] x.
+    x [n, H * P], b and c [n, num_groups * N] (head h reads group h // (H / num_groups)) and dt_pre [n, H] are rows of the
+    activations' type (strided views allowed), y float32 rows.  ``walk``: the token-by-token kernel whatever the portions
+    (csrc/state_dual.cu)."""
+    n, H = dt_pre.shape
+    _need(x.shape[1] % H == 0 and b.shape[1] % num_groups == 0 and H % num_groups == 0, "state_dual: heads and groups")
+    P, N = x.shape[1] // H, b.shape[1] // num_groups
+    for t, name in ((x, "x"), (b, "b"), (c, "c"), (dt_pre, "dt_pre")):
+        _rows(t, name, x.dtype)
+    _rows(y, "y", torch.float32)
+    _need(x.shape[0] == n and y.shape == x.shape and b.shape == c.shape and b.shape[0] == n, "state_dual: shapes")
+    _need(dt_bias.numel() == H and a_log2.numel() == H and d.numel() == H and N <= STATE_DUAL_MAX_STATE,
+          f"state_dual: dt_bias, a_log2 and d [heads], up to {STATE_DUAL_MAX_STATE} state numbers")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, N, P), "state_dual: state float32 [slots, H, N, P]")
+    _check(lib().vcb_state_dual(x.data_ptr(), x.stride(0), b.data_ptr(), b.stride(0), c.data_ptr(), c.stride(0), dt_pre.data_ptr(), dt_pre.stride(0),
+                                _dev(dt_bias, "dt_bias", torch.float32), _dev(a_log2, "a_log2", torch.float32), _dev(d, "d", torch.float32),
+                                state.data_ptr(), y.data_ptr(), y.stride(0), _dev(q_start, "q_start", torch.int32),
+                                _dev(state_slots, "state_slots", torch.int32), n_reqs, int(max_q_len), H, num_groups, N, P, 1 if walk else 0,
+                                dtype_code(x.dtype), _stream()), "state_dual")
+
+
 def general_delta_work(n: int, num_heads: int, head_dim: int, v_head_dim: int) -> int:
     """Floats of the prepared inputs of ``n`` tokens (csrc/general_delta.cu, gd_work_row)."""
     pad = lambda d: (d + 3) // 4 * 4
@@ -1665,10 +1748,11 @@ def rows_rmsnorm(x: torch.Tensor, gain: torch.Tensor, out: torch.Tensor, eps: fl
 
 def latent_rope_cache_write(raw: torch.Tensor, gain: torch.Tensor, q: Optional[torch.Tensor], inv_freq: torch.Tensor, positions,
                             req_of_token, block_table, cache: torch.Tensor, *, rank: int, num_heads: int, q_stride: int, q_off: int,
-                            pairing: int, page_size: int, eps: float, write_kv: bool = True) -> None:
+                            pairing: int, page_size: int, eps: float, write_kv: bool = True, magnitude: float = 1.0) -> None:
     """``raw`` [n, rank + rot] (rows may be strided): the latent's columns, RMS-normed with ``gain``, and the ``rot`` =
     2 * len(inv_freq) columns of a key part that all heads share, turned by the token's position (pair j: coordinates
-    (2j, 2j + 1) with ``pairing`` 1, (j, j + rot / 2) with 0; angle position * inv_freq[j] in float32), go into the token's
+    (2j, 2j + 1) with ``pairing`` 1, (j, j + rot / 2) with 0; angle position * inv_freq[j] in float32; cosine and sine times
+    ``magnitude``), go into the token's
     slot of a one-plane cache [pages, page_size * (rank + rot)] (kv_pos layout).  ``q`` [n, heads * q_stride] is turned in
     place on the ``rot`` columns that start at ``q_off`` inside every head."""
     n = raw.shape[0]
@@ -1680,13 +1764,13 @@ def latent_rope_cache_write(raw: torch.Tensor, gain: torch.Tensor, q: Optional[t
     if q is not None:
         _need(q.dtype == raw.dtype and q.shape == (n, num_heads * q_stride) and q.stride(1) == 1 and q_off + rot <= q_stride,
               "latent_rope_cache_write: q [n, heads * q_stride] with the rotated part inside a head")
-    _check(lib().vcb_latent_rope_cache_write(
+    _check(lib().vcb_latent_rope_cache_write_scaled(
         raw.data_ptr(), raw.stride(0), _dev(gain, "gain", torch.float32), None if q is None else q.data_ptr(),
         0 if q is None else q.stride(0), num_heads, q_stride, q_off, _dev(inv_freq, "inv_freq", torch.float32), rot, int(pairing),
         _dev(positions, "positions", torch.int32), _dev(req_of_token, "req_of_token", torch.int32),
         _dev(block_table, "block_table", torch.int32), block_table.shape[1], cache.data_ptr(), page_size * (rank + rot), n, rank,
-        page_size, float(eps), cache.shape[0], 1 if write_kv else 0, status_tensor(raw.device).data_ptr(), dtype_code(raw.dtype),
-        _stream()), "latent_rope_cache_write")
+        page_size, float(eps), cache.shape[0], 1 if write_kv else 0, float(magnitude), status_tensor(raw.device).data_ptr(),
+        dtype_code(raw.dtype), _stream()), "latent_rope_cache_write")
 
 
 TALKING_MAX_HEADS = 32

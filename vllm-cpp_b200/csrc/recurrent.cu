@@ -319,25 +319,28 @@ VCB_EXPORT int vcb_decayed_state_join(const float* qp, long long ldqp, float* pi
 
 // ------------------------------------------------------------- norm over groups of channels, times a gate
 // One CTA per token.  o: float [n, C]; groups of `group` consecutive channels are normed apart,
-// out = o / sqrt(mean_group(o^2) + eps) * w[channel % wlen] * act(gate), act 0: sigmoid, 1: silu.
+// out = o / sqrt(mean_group(o^2) + eps) * w[channel % wlen] * act(gate), act 0: sigmoid, 1: silu.  `first`: the gate comes
+// before the norm instead, o * act(gate) is normed.
 // One group (group == C): the CTA reduces together; several: a warp per group.
 template <typename T>
 __global__ void gated_group_norm_kernel(const float* __restrict__ o, long long ldo, const T* __restrict__ gate, long long ldg,
                                         const float* __restrict__ w, int wlen, T* __restrict__ out, long long ldout,
-                                        int C, int group, int act, float eps) {
+                                        int C, int group, int act, int first, float eps) {
     __shared__ float scratch[33];
     pdl_start();
     const float* orow = o + (size_t)blockIdx.x * ldo;
     const T* grow = gate ? gate + (size_t)blockIdx.x * ldg : nullptr;
     T* dst = out + (size_t)blockIdx.x * ldout;
+    auto gated = [&](int i) { const float g = to_f32<T>(grow[i]); return act ? silu_f(g) : sigmoid_f(g); };
+    auto value = [&](int i) { return grow && first ? orow[i] * gated(i) : orow[i]; };
     if (group >= C) {
         float ss = 0.0f;
-        for (int i = threadIdx.x; i < C; i += blockDim.x) ss += orow[i] * orow[i];
+        for (int i = threadIdx.x; i < C; i += blockDim.x) { const float v = value(i); ss += v * v; }
         ss = block_sum(ss, scratch);
         const float r = 1.0f / sqrtf(ss / (float)C + eps);
         for (int i = threadIdx.x; i < C; i += blockDim.x) {
-            float y = orow[i] * r * w[i % wlen];
-            if (grow) { const float g = to_f32<T>(grow[i]); y *= act ? silu_f(g) : sigmoid_f(g); }
+            float y = value(i) * r * w[i % wlen];
+            if (grow && !first) y *= gated(i);
             dst[i] = from_f32<T>(y);
         }
         return;
@@ -346,12 +349,12 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ o, long long l
     for (int g0 = warp * group; g0 < C; g0 += nwarps * group) {
         const int len = min(group, C - g0);
         float ss = 0.0f;
-        for (int i = lane; i < len; i += 32) ss += orow[g0 + i] * orow[g0 + i];
+        for (int i = lane; i < len; i += 32) { const float v = value(g0 + i); ss += v * v; }
         ss = warp_sum(ss);
         const float r = 1.0f / sqrtf(ss / (float)len + eps);
         for (int i = lane; i < len; i += 32) {
-            float y = orow[g0 + i] * r * w[(g0 + i) % wlen];
-            if (grow) { const float g = to_f32<T>(grow[g0 + i]); y *= act ? silu_f(g) : sigmoid_f(g); }
+            float y = value(g0 + i) * r * w[(g0 + i) % wlen];
+            if (grow && !first) y *= gated(g0 + i);
             dst[g0 + i] = from_f32<T>(y);
         }
     }
@@ -361,23 +364,31 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ o, long long l
 // thread at a time (16-byte loads of o and the gain, 8-byte loads and stores of the gate and the result).
 __global__ void gated_group_norm_bf16x4_kernel(const float* __restrict__ o, long long ldo, const __nv_bfloat16* __restrict__ gate, long long ldg,
                                                const float* __restrict__ w, int wlen, __nv_bfloat16* __restrict__ out, long long ldout,
-                                               int C, int group, int act, float eps) {
+                                               int C, int group, int act, int first, float eps) {
     __shared__ float scratch[33];
     pdl_start();
     const float* orow = o + (size_t)blockIdx.x * ldo;
     const __nv_bfloat16* grow = gate ? gate + (size_t)blockIdx.x * ldg : nullptr;
     __nv_bfloat16* dst = out + (size_t)blockIdx.x * ldout;
+    auto gates = [&](int i, float (&y)[4]) {                      // y *= act(gate) on channels i .. i + 3
+        const uint2 raw = *reinterpret_cast<const uint2*>(grow + i);
+        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        const float2 a0 = __bfloat1622float2(p[0]), a1 = __bfloat1622float2(p[1]);
+        const float gs[4] = {a0.x, a0.y, a1.x, a1.y};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[e] *= act ? silu_f(gs[e]) : sigmoid_f(gs[e]);
+    };
+    auto value = [&](int i) {                                     // what is normed
+        const float4 v = *reinterpret_cast<const float4*>(orow + i);
+        if (!grow || !first) return v;
+        float y[4] = {v.x, v.y, v.z, v.w};
+        gates(i, y);
+        return make_float4(y[0], y[1], y[2], y[3]);
+    };
     auto finish = [&](int i, float r, const float4& v) {          // channels i .. i + 3, whose values are v
         const float4 g = *reinterpret_cast<const float4*>(w + i % wlen);
         float y[4] = {v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w};
-        if (grow) {
-            const uint2 raw = *reinterpret_cast<const uint2*>(grow + i);
-            const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
-            const float2 a0 = __bfloat1622float2(p[0]), a1 = __bfloat1622float2(p[1]);
-            const float gs[4] = {a0.x, a0.y, a1.x, a1.y};
-#pragma unroll
-            for (int e = 0; e < 4; ++e) y[e] *= act ? silu_f(gs[e]) : sigmoid_f(gs[e]);
-        }
+        if (grow && !first) gates(i, y);
         uint2 packed;
         __nv_bfloat162* q = reinterpret_cast<__nv_bfloat162*>(&packed);
         q[0] = __floats2bfloat162_rn(y[0], y[1]);
@@ -387,12 +398,12 @@ __global__ void gated_group_norm_bf16x4_kernel(const float* __restrict__ o, long
     if (group >= C) {
         float ss = 0.0f;
         for (int i = threadIdx.x * 4; i < C; i += blockDim.x * 4) {
-            const float4 v = *reinterpret_cast<const float4*>(orow + i);
+            const float4 v = value(i);
             ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
         }
         ss = block_sum(ss, scratch);
         const float r = 1.0f / sqrtf(ss / (float)C + eps);
-        for (int i = threadIdx.x * 4; i < C; i += blockDim.x * 4) finish(i, r, *reinterpret_cast<const float4*>(orow + i));
+        for (int i = threadIdx.x * 4; i < C; i += blockDim.x * 4) finish(i, r, value(i));
         return;
     }
     // with few tokens a row's groups are dealt to gridDim.y blocks, so that every warp has one round of work
@@ -403,8 +414,8 @@ __global__ void gated_group_norm_bf16x4_kernel(const float* __restrict__ o, long
             const int g1 = g0 + nwarps * group;
             const bool in0 = lane * 4 < group, in1 = in0 && g1 < C;
             const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            const float4 v0 = in0 ? *reinterpret_cast<const float4*>(orow + g0 + lane * 4) : zero;
-            const float4 v1 = in1 ? *reinterpret_cast<const float4*>(orow + g1 + lane * 4) : zero;
+            const float4 v0 = in0 ? value(g0 + lane * 4) : zero;
+            const float4 v1 = in1 ? value(g1 + lane * 4) : zero;
             const float s0 = warp_sum(v0.x * v0.x + v0.y * v0.y + v0.z * v0.z + v0.w * v0.w);
             const float s1 = warp_sum(v1.x * v1.x + v1.y * v1.y + v1.z * v1.z + v1.w * v1.w);
             if (in0) finish(g0 + lane * 4, 1.0f / sqrtf(s0 / (float)group + eps), v0);
@@ -415,20 +426,20 @@ __global__ void gated_group_norm_bf16x4_kernel(const float* __restrict__ o, long
     for (int g0 = warp * group; g0 < C; g0 += nwarps * group) {
         float ss = 0.0f;
         for (int i = lane * 4; i < group; i += 128) {
-            const float4 v = *reinterpret_cast<const float4*>(orow + g0 + i);
+            const float4 v = value(g0 + i);
             ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
         }
         ss = warp_sum(ss);
         const float r = 1.0f / sqrtf(ss / (float)group + eps);
-        for (int i = lane * 4; i < group; i += 128) finish(g0 + i, r, *reinterpret_cast<const float4*>(orow + g0 + i));
+        for (int i = lane * 4; i < group; i += 128) finish(g0 + i, r, value(g0 + i));
     }
 }
 
-VCB_EXPORT int vcb_gated_group_norm(const float* o, long long ldo, const void* gate, long long ldg, const float* w, int wlen,
-                                    void* out, long long ldout, int n_tokens, int C, int group, int act, float eps,
+VCB_EXPORT int vcb_gated_group_norm_as(const float* o, long long ldo, const void* gate, long long ldg, const float* w, int wlen,
+                                    void* out, long long ldout, int n_tokens, int C, int group, int act, int first, float eps,
                                     int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
-    if (!o || !w || !out || C <= 0 || group <= 0 || wlen <= 0) return VCB_ERR_BAD_ARG;
+    if (!o || !w || !out || (first && !gate) || C <= 0 || group <= 0 || wlen <= 0) return VCB_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = C >= 2048 ? 512 : C >= 512 ? 256 : 128;
     const uintptr_t addrs = (uintptr_t)o | (uintptr_t)w;
@@ -442,18 +453,25 @@ VCB_EXPORT int vcb_gated_group_norm(const float* o, long long ldo, const void* g
             if (split > 8) split = 8;
         }
         vcb_launch(gated_group_norm_bf16x4_kernel, dim3(n_tokens, split), th, 0, s, o, ldo, (const __nv_bfloat16*)gate, ldg, w, wlen, (__nv_bfloat16*)out,
-                   ldout, C, group, act, eps);
+                   ldout, C, group, act, first, eps);
         return vcb_last_error();
     }
     if (dtype == VCB_F32)
         vcb_launch(gated_group_norm_kernel<float>, n_tokens, threads, 0, s, o, ldo, (const float*)gate, ldg, w, wlen, (float*)out,
-                   ldout, C, group, act, eps);
+                   ldout, C, group, act, first, eps);
     else if (dtype == VCB_BF16)
         vcb_launch(gated_group_norm_kernel<__nv_bfloat16>, n_tokens, threads, 0, s, o, ldo, (const __nv_bfloat16*)gate, ldg, w, wlen,
-                   (__nv_bfloat16*)out, ldout, C, group, act, eps);
+                   (__nv_bfloat16*)out, ldout, C, group, act, first, eps);
     else
         return VCB_ERR_BAD_ARG;
     return vcb_last_error();
+}
+
+// The gate after the norm.
+VCB_EXPORT int vcb_gated_group_norm(const float* o, long long ldo, const void* gate, long long ldg, const float* w, int wlen,
+                                    void* out, long long ldout, int n_tokens, int C, int group, int act, float eps,
+                                    int dtype, void* stream) {
+    return vcb_gated_group_norm_as(o, ldo, gate, ldg, w, wlen, out, ldout, n_tokens, C, group, act, 0, eps, dtype, stream);
 }
 
 // ------------------------------------------------------------- two mixers side by side

@@ -1,2 +1,2 @@
 """Architectures known to the registry."""
-from . import gipinex, kasuvik, lutodra, qwen2, retodra, rolesun  # noqa: F401
+from . import gipinex, kasuvik, lutodra, qwen2, retodra, rolesun, rufisun  # noqa: F401

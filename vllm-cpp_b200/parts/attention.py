@@ -33,9 +33,11 @@ class PagedAttentionKernels(Mixer):
     work lists, the kernels' scratch and the choice of kernel.  A subclass sets ``nh`` (query heads),
     ``nkv`` (heads of the cache), ``d`` (width of a cached row), ``window``, ``scale``, ``dtype`` and
     ``planes`` (PagedKVSpec.planes: 2 for keys and values, 1 for rows that are both); ``pool`` > 0 with a window: beside
-    the window's tokens a row per block of ``pool`` tokens that lies before it, in pages of its own (``attend``'s ``blocks``)."""
+    the window's tokens a row per block of ``pool`` tokens that lies before it, in pages of its own (``attend``'s ``blocks``);
+    ``keep_first`` > 0 with a window: beside the window's tokens the sequence's first ones (PagedKVSpec.keep_first)."""
     planes = 2
     pool = 0
+    keep_first = 0
 
     # -- work lists and kernel choice
     def _tensor_core_path(self) -> bool:
@@ -86,6 +88,8 @@ class PagedAttentionKernels(Mixer):
             n = -(-hi // tile) - lo // tile                     # key tiles of every request
             if self.pool:
                 n = n + -(-(lo // self.pool) // tile)           # and those of the blocks before its window
+            elif self.keep_first:
+                n = n + -(-np.minimum(lo, self.keep_first) // tile)     # and those of the kept tokens before its window
             slots = self.decode_slots(len(n))
             low, high = max(1, -(-int(n.sum()) // slots)), int(n.max())
             while low < high:                                   # smallest count whose splits fit the slots
@@ -127,7 +131,7 @@ class PagedAttentionKernels(Mixer):
             ops.zeroed_ints("attn_tickets", n_reqs * self.decode_groups(), device)
 
     def _splits_key(self):
-        return f"attn_splits_kv{self.decode_groups()}_w{self.window}" + (f"_p{self.pool}" if self.pool else "")
+        return f"attn_splits_kv{self.decode_groups()}_w{self.window}" + (f"_p{self.pool}" if self.pool else "") + (f"_k{self.keep_first}" if self.keep_first else "")
 
     def score_shaping(self) -> dict:
         """What the tensor-core kernels do to a score beyond the scale: ``cap`` (cap * tanh(score / cap)) and ``bias_t``
@@ -143,6 +147,8 @@ class PagedAttentionKernels(Mixer):
                       window=self.window, scale=self.scale, planes=self.planes, **self.score_shaping())
             if head_gate is not None:
                 kw["head_gate"] = head_gate
+            if self.keep_first and self.window:
+                kw["keep_first"] = self.keep_first
             pooled = ()
             if blocks is not None:
                 kw = {name: kw[name] for name in ("num_heads", "num_kv_heads", "head_dim", "page_size", "window", "scale")}
@@ -155,7 +161,7 @@ class PagedAttentionKernels(Mixer):
                     # the device once, from the longest context's power-of-two bucket
                     longest = step.split_len or step.max_total_len
                     if self.window > 0 and not self.pool:
-                        longest = min(longest, self.window + 64)
+                        longest = min(longest, self.window + 64 + self.keep_first)
                     nsplit = max(1, min(-(-longest // 64), 2 * ops.sm_count() // (step.n_reqs * self.decode_groups()),
                                         ops.DECODE_MAX_SPLITS))
                     split_tiles = None
@@ -185,7 +191,8 @@ class PagedAttentionKernels(Mixer):
             raise ValueError("attend: the plain kernel has no gate; a mixer with one calls its own kernel")
         ops.attention_simt(q, cache.pages, attn, step.positions, step.req_of_token, block_table,
                            num_heads=self.nh, num_kv_heads=self.nkv, head_dim=self.d,
-                           page_size=cache.page_size, window=self.window, scale=self.scale, planes=self.planes)
+                           page_size=cache.page_size, window=self.window, scale=self.scale, planes=self.planes,
+                           sink=self.score_shaping().get("sink"))
 
 
 @register_mixer("attention")
@@ -206,6 +213,8 @@ class PagedAttention(PagedAttentionKernels):
         self.qkv_bias, self.window = bool(qkv_bias), int(window)
         self.dtype, self.device = dtype, device
         self.position = build_part(POSITION_ENCODINGS, "position encoding", position, dtype=dtype, device=device)
+        if getattr(self.position, "magnitude", 1.0) != 1.0:
+            raise ValueError("attention: a rotation whose cosine and sine carry a factor is not built")
         # 1/sqrtf(d) in float, as src/layers/attention.cpp:126 computes it
         self.scale = float(np.float32(1.0) / np.sqrt(np.float32(head_dim)))
         self.w_qkv = None

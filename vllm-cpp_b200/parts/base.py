@@ -58,13 +58,16 @@ class PagedKVSpec:
     ``stride`` > 1: a row for every ``stride`` tokens instead of one per token, written once the last of them is there (a
     summary of a block of tokens): a request of n tokens holds n // stride rows.  ``keep_block`` > 1 (with a window): the
     tokens of the block of ``keep_block`` tokens that is not complete yet are kept although the window may have passed
-    them, because the block's summary is made of them."""
+    them, because the block's summary is made of them.
+    ``keep_first`` > 0 (with a window): the sequence's first ``keep_first`` tokens are read wherever the window is, and their
+    pages are never given back."""
     num_kv_heads: int
     head_dim: int
     window: int = 0
     planes: int = 2
     stride: int = 1
     keep_block: int = 1
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

@@ -11,7 +11,13 @@ rows are spread evenly over the logarithm of the distance up to ``bias_reach``, 
 ``bias_reach`` on uses the last row:  bucket(n) = n  for n < B // 2,  else
 min(B - 1, B // 2 + floor(ln(n / (B // 2)) / ln(bias_reach / (B // 2)) * (B - B // 2))).  At load the table is
 expanded to one row per distance (up to the window, or to ``bias_reach``, where it becomes constant), so the
-kernel looks a distance up directly.  ``cap`` 0 switches the cap off, ``window`` 0 the window.
+kernel looks a distance up directly.  ``cap`` 0 switches the cap off, ``window`` 0 the window, ``bias_reach`` None the bias and its table.
+
+``keep_first`` > 0 (with a window): the sequence's first tokens are seen wherever the window is, under their true distances; their
+pages stay.  ``sink``: a learned logit per head (tensor "sink") that joins the softmax's denominator once, neither scaled nor
+capped nor biased, with no key and no value.  ``temperature`` (coef, every): the queries of position p are multiplied by
+1 + coef * ln((p + 1) // every + 1), in float before they are rounded.  ``precise_weights``: the softmax weights enter the
+tensor-core kernels' product with the values as two bfloat16 terms.
 
 The cache holds the normed keys and the values in rows of max(head_dim, v_head_dim) elements
 (PagedKVSpec.head_dim); with a window, pages behind it are given back.  q, k, v and the gate are one product.
@@ -23,7 +29,7 @@ The reference's attention (src/layers/attention.cpp) has rotation and none of th
 from __future__ import annotations
 
 import math
-from typing import Dict
+from typing import Dict, Optional
 
 import numpy as np
 import torch
@@ -50,19 +56,26 @@ def distance_buckets(rows: int, reach: float, count: int) -> np.ndarray:
 @register_mixer("biased_window_attention")
 class BiasedWindowAttention(PagedAttentionKernels):
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int, scale: float,
-                 softcap: float, window: int, bias_reach: float, eps: float, dtype, device, qk_norm: bool = True,
-                 output_gate: bool = True):
+                 softcap: float, window: int, bias_reach: Optional[float], eps: float, dtype, device, qk_norm: bool = True,
+                 output_gate: bool = True, keep_first: int = 0, sink: bool = False, temperature=None, precise_weights: bool = False):
         if min(hidden_size, num_heads, num_kv_heads, head_dim, v_head_dim) <= 0 or num_heads % num_kv_heads:
             raise ValueError(f"biased_window_attention: {num_heads} heads cannot share {num_kv_heads} kv heads")
         if v_head_dim > 256 or head_dim > 1024:
             raise ValueError("biased_window_attention: head sizes up to 1024 (keys) and 256 (values)")
-        if window < 0 or softcap < 0 or not eps > 0 or not bias_reach > 0:
+        if window < 0 or softcap < 0 or not eps > 0 or (bias_reach is not None and not bias_reach > 0):
             raise ValueError("biased_window_attention: window and softcap must not be negative, eps and bias_reach positive")
+        if keep_first < 0 or (temperature is not None and not int(temperature[1]) > 0):
+            raise ValueError("biased_window_attention: keep_first must not be negative, the temperature's step positive")
+        if keep_first and window and not precise_weights:
+            raise ValueError("biased_window_attention: kept first tokens are built with two-term weights")
         self.hidden, self.nh, self.nkv, self.dk, self.dv = hidden_size, num_heads, num_kv_heads, head_dim, v_head_dim
         self.row = max(head_dim, v_head_dim)
         self.d = self.row              # a cached row's width, as the paged attention kernels see it
-        self.scale, self.cap, self.window, self.reach, self.eps = float(scale), float(softcap), int(window), float(bias_reach), float(eps)
+        self.scale, self.cap, self.window, self.reach, self.eps = float(scale), float(softcap), int(window), bias_reach, float(eps)
         self.qk_norm, self.output_gate = bool(qk_norm), bool(output_gate)
+        self.keep_first = int(keep_first) if window else 0              # without a window everything is seen anyway
+        self.has_sink, self.precise_weights, self.sink = bool(sink), bool(precise_weights), None
+        self.temperature = None if temperature is None else (float(temperature[0]), int(temperature[1]))
         self.dtype, self.device = dtype, device
         self.w_in = self.w_o = self.w_qn = self.w_kn = self.bias = self.bias_t = None
 
@@ -72,7 +85,10 @@ class BiasedWindowAttention(PagedAttentionKernels):
         if self.qk_norm:
             specs["q.norm"] = ParamSpec((q,), "gain")
             specs["k.norm"] = ParamSpec((kk,), "gain")
-        specs["rel"] = ParamSpec((-1, self.nh), "bias", default_shape=(DEFAULT_BIAS_ROWS, self.nh))
+        if self.reach is not None:
+            specs["rel"] = ParamSpec((-1, self.nh), "bias", default_shape=(DEFAULT_BIAS_ROWS, self.nh))
+        if self.has_sink:
+            specs["sink"] = ParamSpec((self.nh,), "bias")
         if self.output_gate:
             specs["g"] = ParamSpec((self.nh * self.dv, self.hidden))
         specs["o"] = ParamSpec((self.hidden, self.nh * self.dv))
@@ -84,31 +100,36 @@ class BiasedWindowAttention(PagedAttentionKernels):
         self.w_o = tensors["o"].contiguous()
         if self.qk_norm:
             self.w_qn, self.w_kn = tensors["q.norm"].contiguous(), tensors["k.norm"].contiguous()
-        rel = tensors["rel"].to(torch.float32)
+        if self.has_sink:
+            self.sink = tensors["sink"].contiguous()
+        if self.reach is not None:
+            self._expand_bias(tensors["rel"].to(torch.float32))
+        if self.dk == self.dv:
+            self.warn_if_plain()
+
+    def _expand_bias(self, rel):
         B = int(rel.shape[0])
         if B < 2 or self.reach <= B // 2:
             raise ValueError(f"biased_window_attention: a bias table of {B} rows cannot reach distance {self.reach}")
         # one row per distance; from ceil(bias_reach) on every distance reads the last row of the table
         count = int(math.ceil(self.reach)) + 1
-        if self.window > 0:
+        if self.window > 0 and not self.keep_first:              # kept tokens may lie at any distance
             count = min(count, self.window)
         idx = torch.from_numpy(distance_buckets(B, self.reach, count)).to(rel.device)
         self.bias = rel.index_select(0, idx).contiguous()           # [distances, heads]
         self.bias_t = self.bias.t().contiguous()                    # [heads, distances], for the tensor-core kernels
-        if self.dk == self.dv:
-            self.warn_if_plain()
 
     def _tensor_core_path(self) -> bool:
         return self.dk == self.dv and super()._tensor_core_path()
 
     def score_shaping(self):
-        return {"cap": self.cap, "bias_t": self.bias_t}
+        return dict({"sink": self.sink} if self.has_sink else {}, cap=self.cap, bias_t=self.bias_t, precise_weights=self.precise_weights)
 
     def product_weights(self):
-        return [(self.w_in, 0), (self.w_o, 0)]
+        return [(w, 0) for w in (self.w_in, self.w_o) if w is not None]
 
     def cache_spec(self):
-        return PagedKVSpec(self.nkv, self.row, self.window)
+        return PagedKVSpec(self.nkv, self.row, self.window, keep_first=self.keep_first)
 
     def in_width(self) -> int:
         return self.nh * self.dk + self.nkv * (self.dk + self.dv) + (self.nh * self.dv if self.output_gate else 0)
@@ -118,10 +139,16 @@ class BiasedWindowAttention(PagedAttentionKernels):
                 + workspace_piece((n_tokens, self.nh * self.dv), self.dtype))
 
     def forward(self, x, out, step, cache, writes_cache, ws):
-        n = x.shape[0]
         mark = ws.mark()
-        proj = ws.take((n, self.in_width()), self.dtype)
+        proj = ws.take((x.shape[0], self.in_width()), self.dtype)
         ops.linear(x, self.w_in, proj)
+        self.forward_projected(proj, out, step, cache, writes_cache, ws)
+        ws.release(mark)
+
+    def forward_projected(self, proj, out, step, cache, writes_cache, ws):
+        """``forward`` from the rows of the input product on (a mixer that shares its input product calls this)."""
+        n = proj.shape[0]
+        mark = ws.mark()
         q_off, k_off = 0, self.nh * self.dk
         v_off = k_off + self.nkv * self.dk
         g_off = v_off + self.nkv * self.dv
@@ -131,15 +158,15 @@ class BiasedWindowAttention(PagedAttentionKernels):
                      page_size=cache.page_size)
         q = ws.take((n, self.nh * self.dk), self.dtype)
         ops.qk_norm_cache_write(proj, q_off, k_off, v_off, self.w_qn, self.w_kn, q, pages, step.positions, step.req_of_token,
-                                block_table, eps=self.eps, write_kv=writes_cache, **sizes)
+                                block_table, eps=self.eps, write_kv=writes_cache, temperature=self.temperature, **sizes)
         attn = ws.take((n, self.nh * self.dv), self.dtype)
-        gate = proj[:, g_off:] if self.output_gate else None
+        gate = proj[:, g_off: self.in_width()] if self.output_gate else None
         if self._tensor_core_path() and cache.page_size % 8 == 0:
             self.attend(q, attn, step, cache, block_table)
             if gate is not None:
                 ops.sigmoid_gate(attn, gate)
         else:
             ops.attention_biased(q, pages, attn, gate, step.positions, step.req_of_token, block_table, self.bias,
-                                 window=self.window, scale=self.scale, cap=self.cap, **sizes)
+                                 window=self.window, scale=self.scale, cap=self.cap, sink=self.sink, keep_first=self.keep_first, **sizes)
         ops.linear(attn, self.w_o, out)
         ws.release(mark)

@@ -135,12 +135,15 @@ class RotaryLatentAttention(PagedAttentionKernels):
     Only [c | rot(kr)] is cached, one row of kv_rank + rot_dim per token (PagedKVSpec.planes = 1): the plain query part is
     moved into the latent space and the rotated part rides along, both by one per-head product with the block matrix
     [[Wuk_h^T, 0], [0, I]], so that attention is multi-query attention over the cached rows; its result leaves the latent
-    space by Wuv_h (zero columns where the rotated part sat), with the gate in that product's epilogue."""
+    space by Wuv_h (zero columns where the rotated part sat), with the gate in that product's epilogue.  A position encoding whose
+    cosine and sine carry a factor (``magnitude``) turns both parts with it.  ``sink``: a learned logit per head (tensor "sink") that
+    joins the softmax's denominator once, unscaled, with no key and no value."""
     planes = 1
     GATES = ("head", "channel", "none")
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, kv_rank: int, q_rank: int,
-                 scale: float, eps: float, position: PartSpec, dtype, device, gate: str = "head", window: int = 0):
+                 scale: float, eps: float, position: PartSpec, dtype, device, gate: str = "head", window: int = 0,
+                 sink: bool = False):
         if min(hidden_size, num_heads, head_dim, v_head_dim, kv_rank) <= 0 or q_rank < 0 or rot_dim < 0 or rot_dim % 2:
             raise ValueError("rotary_latent_attention: sizes must be positive, rot_dim even")
         if kv_rank + rot_dim > ops.SIMT_MAX_HEAD_DIM:
@@ -153,18 +156,20 @@ class RotaryLatentAttention(PagedAttentionKernels):
         self.scale, self.window, self.eps, self.gate = float(scale), int(window), float(eps), gate
         self.dtype, self.device = dtype, device
         self.position = build_part(POSITION_ENCODINGS, "position encoding", position, dtype=dtype, device=device)
-        self.pairing, self.inv_freq = 0, None
+        self.pairing, self.inv_freq, self.magnitude = 0, None, 1.0
+        self.has_sink, self.sink = bool(sink), None
         if rot_dim:
             fused = self.position.fused()
             if fused is None or fused["rotary_dim"] != rot_dim or not hasattr(self.position, "inv_freq"):
                 raise ValueError("rotary_latent_attention: the position encoding must rotate rot_dim coordinates with given frequencies")
             self.pairing, self.inv_freq = int(fused["pairing"]), self.position.inv_freq
+            self.magnitude = float(getattr(self.position, "magnitude", 1.0))
         self.w_in = self.w_uq = self.w_qn = self.w_c = self.w_qk = self.w_uv = self.w_o = None
 
     # -- tensors
     def score_shaping(self):
         # attention weights are wanted in 32-bit: the tensor-core kernels take them as two bfloat16 terms
-        return {"precise_weights": True}
+        return dict({"sink": self.sink} if self.has_sink else {}, precise_weights=True)
 
     def gate_rows(self) -> int:
         return {"head": self.heads, "channel": self.heads * self.vd, "none": 0}[self.gate]
@@ -181,6 +186,8 @@ class RotaryLatentAttention(PagedAttentionKernels):
                       "uk": ParamSpec((h * self.qk, self.rank)), "uv": ParamSpec((h * self.vd, self.rank))})
         if self.gate != "none":
             specs["g"] = ParamSpec((self.gate_rows(), self.hidden))
+        if self.has_sink:
+            specs["sink"] = ParamSpec((self.heads,), "bias")
         specs["o"] = ParamSpec((self.hidden, h * self.vd))
         return specs
 
@@ -201,6 +208,8 @@ class RotaryLatentAttention(PagedAttentionKernels):
         w_uv[:, :, :self.rank] = tensors["uv"].unflatten(0, (h, self.vd))
         self.w_uv = w_uv.contiguous()
         self.w_o = tensors["o"].contiguous()
+        if self.has_sink:
+            self.sink = tensors["sink"].contiguous()
         self._no_freq = torch.zeros(0, dtype=torch.float32, device=self.w_c.device)
         self.warn_if_plain()
 
@@ -243,7 +252,8 @@ class RotaryLatentAttention(PagedAttentionKernels):
         inv_freq = self.inv_freq if self.rot else self._no_freq
         ops.latent_rope_cache_write(proj[:, q0:g0], self.w_c, q if self.rot else None, inv_freq, step.positions, step.req_of_token,
                                     block_table, pages, rank=self.rank, num_heads=h, q_stride=qd, q_off=self.qk,
-                                    pairing=self.pairing, page_size=cache.page_size, eps=self.eps, write_kv=writes_cache)
+                                    pairing=self.pairing, page_size=cache.page_size, eps=self.eps, write_kv=writes_cache,
+                                    magnitude=self.magnitude)
         q_lat = ws.take((n, h * self.d), self.dtype)
         ops.headwise_linear(q, self.w_qk, q_lat)
         o_lat = ws.take((n, h * self.d), self.dtype)

@@ -102,3 +102,38 @@ class GatedMLP(FeedForward):
             (ops.relu_mul if self.activation == "relu" else ops.silu_mul)(gate_up, act)
         ops.linear(act, self.w_down, out, fuse=fuse)
         ws.release(mark)
+
+
+@register_feed_forward("two_layer_mlp")
+class TwoLayerMLP(FeedForward):
+    """Feed-forward without a gate: down( act(up(x)) ), no biases.  ``activation`` "relu_squared" is max(z, 0)^2, "gelu" is
+    z Phi(z) by its definition (through erf)."""
+
+    def __init__(self, hidden_size: int, intermediate_size: int, activation: str, dtype, device, tensor_names=("up", "down")):
+        if activation not in ops.ROW_ACTS:
+            raise ValueError(f"two_layer_mlp: activation {activation!r} is not built (known: {sorted(ops.ROW_ACTS)})")
+        self.hidden, self.inter, self.activation, self.names = hidden_size, intermediate_size, activation, tuple(tensor_names)
+        self.dtype, self.device = dtype, device
+        self.w_up = None          # [inter, hidden]
+        self.w_down = None        # [hidden, inter]
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        up, down = self.names
+        return {up: ParamSpec((self.inter, self.hidden)), down: ParamSpec((self.hidden, self.inter))}
+
+    def load_params(self, tensors):
+        self.w_up, self.w_down = (tensors[n].contiguous() for n in self.names)
+
+    def product_weights(self):
+        return [(self.w_up, 0), (self.w_down, 0)]
+
+    def workspace_bytes(self, n_tokens, n_reqs):
+        return workspace_piece((n_tokens, self.inter), self.dtype)
+
+    def forward(self, x, out, step, ws):
+        mark = ws.mark()
+        act = ws.take((x.shape[0], self.inter), self.dtype)
+        ops.linear(x, self.w_up, act)
+        ops.act_rows(act, act, self.activation)
+        ops.linear(act, self.w_down, out)
+        ws.release(mark)

@@ -24,7 +24,7 @@ from .base import BLOCKS, FAMILIES, NORMS, ParamSpec, StepContext, Workspace, Sc
 from . import (attention as _attention, biased_attention as _biased, block as _block, gate as _gate,  # noqa: F401
                latent_attention as _latent, linear_attention as _linear, mlp as _mlp, moe as _moe, norm as _norm,
                gated_recurrence as _gated_recurrence, general_delta as _general_delta, parallel as _parallel, pooled_attention as _pooled,
-               position as _position, scale as _scale, selective_state as _selective, shift as _shift, sink_attention as _sink_attention, streams as _streams, talking_attention as _talking)
+               position as _position, scale as _scale, selective_state as _selective, shift as _shift, sink_attention as _sink_attention, state_dual as _state_dual, streams as _streams, talking_attention as _talking)
 
 TORCH_DTYPES = {"bfloat16": torch.bfloat16, "float32": torch.float32}
 

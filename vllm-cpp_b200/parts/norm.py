@@ -114,6 +114,32 @@ class LayerNorm(Norm):
         ops.stream_norm(x, self._one, self.weight, self.bias, out, self.eps, row_index, self.out_scale)
 
 
+@register_norm("tanh")
+class TanhNorm(Norm):
+    """A norm without statistics: y = tanh(alpha * x) * w + b, alpha one learned number, w and b a number per coordinate, in
+    float32.  ``tensor_name`` is the local name of the gain ("": the slot's prefix itself); slope and shift are that name plus
+    ``alpha_suffix`` and ``bias_suffix``."""
+
+    def __init__(self, size: int, dtype, device, tensor_name: str = "weight", alpha_suffix: str = ".alpha", bias_suffix: str = ".b"):
+        if size <= 0:
+            raise ValueError(f"tanh norm: size {size} must be positive")
+        self.size, self.tensor_name = size, tensor_name
+        self.alpha_name, self.bias_name = tensor_name + alpha_suffix, tensor_name + bias_suffix
+        self.alpha: Optional[torch.Tensor] = None          # float32 [1]
+        self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        return {self.tensor_name: ParamSpec((self.size,), "gain"), self.alpha_name: ParamSpec((), "gain"), self.bias_name: ParamSpec((self.size,), "bias")}
+
+    def load_params(self, tensors):
+        self.weight, self.bias = tensors[self.tensor_name].contiguous(), tensors[self.bias_name].contiguous()
+        self.alpha = tensors[self.alpha_name].reshape(1).to(torch.float32).contiguous()
+
+    def forward(self, residual, delta, out, row_index=None, mult=1.0):
+        ops.add_tanh_norm(residual, delta, self.alpha, self.weight, self.bias, out, row_index, mult)
+
+
 @register_norm("none")
 class NoNorm(Norm):
     """Fills the norm slot of a sublayer that a layer does not have."""

@@ -51,6 +51,8 @@ class PooledWindowAttention(PagedAttentionKernels):
         fused = self.position.fused()
         if fused is None or (fused["rotary_dim"] and (fused["pairing"] != 1 or not hasattr(self.position, "inv_freq"))):
             raise ValueError("pooled_window_attention: positions enter by a rotation of interleaved pairs with given frequencies, or not at all")
+        if getattr(self.position, "magnitude", 1.0) != 1.0:
+            raise ValueError("pooled_window_attention: a rotation whose cosine and sine carry a factor is not built")
         self.rot = int(fused["rotary_dim"])
         if self.rot > head_dim:
             raise ValueError(f"pooled_window_attention: {self.rot} rotated coordinates in heads of {head_dim}")

@@ -41,6 +41,8 @@ class RotaryEmbedding(PositionEncoding):
         denom = np.power(np.float64(np.float32(theta)), exponent.astype(np.float64)).astype(np.float32)
         self.denom = torch.from_numpy(denom).to(device)
 
+    magnitude = 1.0          # factor of cosine and sine
+
     def fused(self) -> Optional[dict]:
         return {"rotary_dim": self.rotary_dim, "pairing": PAIRINGS[self.pairing], "denom": self.denom}
 
@@ -57,10 +59,25 @@ def rescale_by_wavelength(freq: np.ndarray, factor: float, low: float, high: flo
     return np.where(wavelength < original / high, freq, np.where(wavelength > original / low, freq / factor, between))
 
 
+def stretch_by_ramp(freq: np.ndarray, theta: float, factor: float, original: float, fast: float, slow: float) -> np.ndarray:
+    """Frequencies (float64, f_i = theta^(-2i / dims)) rescaled by how often they turn within ``original`` positions: those that turn
+    more than ``fast`` times stay, those below ``slow`` are divided by ``factor``, with a linear ramp over the index i between the two
+    borders (rounded outwards to whole indices, and kept inside 0 .. dims - 1)."""
+    if not (factor > 0 and original > 0 and fast > 0 and slow > 0 and theta > 1):
+        raise ValueError(f"frequency scaling: factor {factor}, original {original}, fast {fast}, slow {slow}, base {theta}")
+    dims = 2 * len(freq)
+    border = lambda turns: dims * np.log(original / (2.0 * np.pi * turns)) / (2.0 * np.log(theta))
+    lo, hi = max(np.floor(border(fast)), 0.0), min(np.ceil(border(slow)), dims - 1.0)
+    ramp = np.clip((np.arange(len(freq)) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return freq / factor * ramp + freq * (1.0 - ramp)
+
+
 @register_position_encoding("scaled_rope")
 class ScaledRotaryEmbedding(RotaryEmbedding):
     """"rope" whose frequencies f_i = theta^(-2i / rotary_dim) are rescaled by wavelength (``scaling``: None, or
-    {"factor", "low", "high", "original"}; rescale_by_wavelength).  The frequencies are computed in double and rounded
+    {"factor", "low", "high", "original"}; rescale_by_wavelength) or by a ramp over their index ({"factor", "fast", "slow",
+    "original"}; stretch_by_ramp), in which case cosine and sine are also multiplied by ``magnitude`` = 0.1 ln(factor) + 1 (a mixer
+    whose kernel has no such factor refuses an encoding with a magnitude other than 1).  The frequencies are computed in double and rounded
     once; ``inv_freq`` (float32 [rotary_dim / 2]) is what a kernel multiplies a position by, ``denom`` its reciprocal
     for kernels that divide."""
 
@@ -68,7 +85,14 @@ class ScaledRotaryEmbedding(RotaryEmbedding):
         super().__init__(theta, rotary_dim, pairing, dtype=dtype, device=device)
         i = np.arange(rotary_dim // 2, dtype=np.float64)
         freq = np.power(float(theta), -2.0 * i / rotary_dim)
-        if scaling is not None:
+        self.magnitude = 1.0
+        if scaling is not None and "fast" in scaling:
+            missing = [k for k in ("factor", "fast", "slow", "original") if k not in scaling]
+            if missing:
+                raise ValueError(f"scaled_rope: scaling lacks {missing}")
+            freq = stretch_by_ramp(freq, float(theta), *(float(scaling[k]) for k in ("factor", "original", "fast", "slow")))
+            self.magnitude = 0.1 * float(np.log(float(scaling["factor"]))) + 1.0
+        elif scaling is not None:
             missing = [k for k in ("factor", "low", "high", "original") if k not in scaling]
             if missing:
                 raise ValueError(f"scaled_rope: scaling lacks {missing}")

@@ -50,6 +50,8 @@ class SinkAttention(PagedAttentionKernels):
         fused = self.position.fused()
         if fused is None or (fused["rotary_dim"] and (fused["pairing"] != 0 or not hasattr(self.position, "inv_freq"))):
             raise ValueError("sink_attention: positions enter by a rotation of half-split pairs with given frequencies, or not at all")
+        if getattr(self.position, "magnitude", 1.0) != 1.0:
+            raise ValueError("sink_attention: a rotation whose cosine and sine carry a factor is not built")
         self.rot = int(fused["rotary_dim"])
         if self.rot > head_dim:
             raise ValueError(f"sink_attention: {self.rot} rotated coordinates in heads of {head_dim}")
