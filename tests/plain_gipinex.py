@@ -81,7 +81,7 @@ def write_model_folder(path, cfg, weights, store="F32"):
             raw = (((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype("<u2")).tobytes()
         else:
             raw = a.astype("<f4").tobytes()
-        header[name] = {"dtype": store, "shape": list(a.shape), "data_offsets": [at, at + len(raw)]}
+        header[name] = {"dtype": store, "shape": list(np.shape(w)), "data_offsets": [at, at + len(raw)]}
         blobs.append(raw)
         at += len(raw)
     text = json.dumps(header).encode()

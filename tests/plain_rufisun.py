@@ -27,7 +27,7 @@ from scipy.special import erf
 from plain_kasuvik import perturbed, product, rms, rounded_like_bf16, short_conv, sigmoid, silu, softplus  # noqa: F401
 from plain_gipinex import read_model_folder, read_safetensors, round_to_bf16, write_model_folder  # noqa: F401
 
-BIAS_ROWS = 32          # rows of the distance-bias table that random_weights makes
+BIAS_ROWS = 20          # rows of the distance-bias table that random_weights makes
 
 
 # ------------------------------------------------------------- shapes and random weights

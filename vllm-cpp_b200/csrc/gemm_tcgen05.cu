@@ -84,9 +84,22 @@ struct GemmArgs {
     // Tile t holds gate rows 64 t .. and, in its upper half, the matching up rows;
     // out[token, 64 t + r] = act(gate) * up, act silu or relu (the kernel's parameter).
     int gated;
+    // EPI_TANH_NORM (with residual and gain): out = bfloat16(tanh(alpha * residual) * gain + shift), a norm without statistics
+    const float* shift;          // [rows_p]
+    const float* alpha;          // [1]
 };
 
-template <bool RELU> __device__ __forceinline__ float gate_activation(float z) { return RELU ? fmaxf(z, 0.0f) : z / (1.0f + expf(-z)); }
+// What the epilogue does beside scaling and storing (a template parameter of the kernel: a choice at run time costs every other
+// product of a decode step).  Gated products: silu or relu of the gate.  Others: the square of relu, gelu by its definition, or the
+// end of a residual branch with a norm that needs no statistics.
+enum { EPI_SILU = 0, EPI_RELU = 1, EPI_RELU_SQUARED = 2, EPI_GELU = 3, EPI_TANH_NORM = 4 };
+
+template <int EPI> __device__ __forceinline__ float gate_activation(float z) { return EPI == EPI_RELU ? fmaxf(z, 0.0f) : z / (1.0f + expf(-z)); }
+template <int EPI> __device__ __forceinline__ float product_activation(float z) {
+    if (EPI == EPI_RELU_SQUARED) { const float r = fmaxf(z, 0.0f); return r * r; }
+    if (EPI == EPI_GELU) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f));
+    return z;
+}
 
 // The segments of one CTA's run of (tile, slab) units.
 struct Segments {
@@ -210,7 +223,7 @@ struct Units {
     }
 };
 
-template <int BN, int STAGES, bool RELU>
+template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant__ CUtensorMap map_q, GemmArgs a) {
     constexpr int Q_BYTES = BN * BK * 2;
@@ -379,7 +392,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
                             const float f = a.scale_sumsq ? rstd_s[j] : 1.0f;
                             const float z = v[g8 + e] * f, u = xch[r * 8 + e] * f;
                             reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)j * a.ldc + feature] =
-                                __float2bfloat16_rn(gate_activation<RELU>(z) * u);
+                                __float2bfloat16_rn(gate_activation<EPI>(z) * u);
                         }
                     }
                     asm volatile("bar.sync 1, 128;" ::: "memory");   // the halves are read before the next group overwrites them
@@ -389,6 +402,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
             const bool row_ok = i < a.rows_p;
             if (a.residual) {                       // swapped, one tile of tokens: j = c + e is the token
                 float x[NE];
+                [[maybe_unused]] float slope = 0.0f, shift = 0.0f;
+                if constexpr (EPI == EPI_TANH_NORM) {
+                    slope = __ldg(a.alpha);
+                    shift = row_ok ? __ldg(a.shift + i) : 0.0f;
+                }
 #pragma unroll
                 for (int e = 0; e < NE; ++e) {      // all loads first: the stores below would order them
                     const int j = q0 + c + e;
@@ -402,8 +420,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
                     if (row_ok) {
                         x[e] += a.scale_sumsq ? v[e] * rstd_s[j] : v[e];
                         a.residual[(size_t)j * a.ldr + i] = x[e];
-                        reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)j * a.ldc + i] = __float2bfloat16_rn(x[e] * g);
+                        reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)j * a.ldc + i] =
+                            __float2bfloat16_rn(EPI == EPI_TANH_NORM ? fmaf(tanhf(slope * x[e]), g, shift) : x[e] * g);
                     }
+                    if constexpr (EPI == EPI_TANH_NORM) continue;
                     float sq = x[e] * x[e];
 #pragma unroll
                     for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
@@ -417,7 +437,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
                 const int j = q0 + c + e;
                 if (j >= a.rows_q) break;
                 const size_t idx = a.swapped ? (size_t)j * a.ldc + i : (size_t)i * a.ldc + j;
-                const float x = a.scale_sumsq ? v[e] * rstd_s[j] : v[e];
+                const float x = product_activation<EPI>(a.scale_sumsq ? v[e] * rstd_s[j] : v[e]);
                 if (a.out_f32) reinterpret_cast<float*>(a.out)[idx] = x;
                 else reinterpret_cast<__nv_bfloat16*>(a.out)[idx] = __float2bfloat16_rn(x);
             }
@@ -481,7 +501,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
                                 const float z = (is_gate ? __uint_as_float(lo[e]) : from_gate[e * 64 + half_row]) * f;
                                 const float u = (is_gate ? from_up[e * 64 + half_row] : __uint_as_float(hi[e])) * f;
                                 reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)j * a.ldc + feature] =
-                                    __float2bfloat16_rn(gate_activation<RELU>(z) * u);
+                                    __float2bfloat16_rn(gate_activation<EPI>(z) * u);
                             }
                         }
                         asm volatile("bar.sync 1, 128;" ::: "memory");   // read before the next round overwrites
@@ -657,22 +677,29 @@ int make_map(CUtensorMap* map, const void* base, int rows, int k, int ld, int bo
     return r == CUDA_SUCCESS ? 0 : VCB_ERR_BAD_ARG;
 }
 
-template <int BN, int STAGES, bool RELU>
+template <int BN, int STAGES, int EPI>
 int launch_as(const CUtensorMap& mp, const CUtensorMap& mq, const GemmArgs& a, int ctas, cudaStream_t s) {
     // stages, 1 KB to align them, barriers with the epilogue's factor and exchange areas (2 KB, 8 KB for wide tiles)
     constexpr size_t smem = (size_t)STAGES * (P_BYTES + BN * BK * 2) + 1024 + (BN >= 32 ? 9216 : 3072);
     static unsigned long long configured = 0;
-    if (int e = vcb_allow_dynamic_smem(gemm_tcgen05_kernel<BN, STAGES, RELU>, (int)smem, &configured)) return e;
-    vcb_launch(gemm_tcgen05_kernel<BN, STAGES, RELU>, ctas, GEMM_THREADS, smem, s, mp, mq, a);
+    if (int e = vcb_allow_dynamic_smem(gemm_tcgen05_kernel<BN, STAGES, EPI>, (int)smem, &configured)) return e;
+    vcb_launch(gemm_tcgen05_kernel<BN, STAGES, EPI>, ctas, GEMM_THREADS, smem, s, mp, mq, a);
     return vcb_last_error();
 }
 
-// relu: the activation of a gated product (tiles of up to 128 columns); other products do not look at it
+// epi other than EPI_SILU: tiles of up to 128 columns
 template <int BN, int STAGES>
-int launch(const CUtensorMap& mp, const CUtensorMap& mq, const GemmArgs& a, int ctas, bool relu, cudaStream_t s) {
-    if constexpr (BN <= 128)
-        if (relu) return launch_as<BN, STAGES, true>(mp, mq, a, ctas, s);
-    return launch_as<BN, STAGES, false>(mp, mq, a, ctas, s);
+int launch(const CUtensorMap& mp, const CUtensorMap& mq, const GemmArgs& a, int ctas, int epi, cudaStream_t s) {
+    if constexpr (BN <= 128) {
+        switch (epi) {
+            case EPI_RELU: return launch_as<BN, STAGES, EPI_RELU>(mp, mq, a, ctas, s);
+            case EPI_RELU_SQUARED: return launch_as<BN, STAGES, EPI_RELU_SQUARED>(mp, mq, a, ctas, s);
+            case EPI_GELU: return launch_as<BN, STAGES, EPI_GELU>(mp, mq, a, ctas, s);
+            case EPI_TANH_NORM: return launch_as<BN, STAGES, EPI_TANH_NORM>(mp, mq, a, ctas, s);
+            default: break;
+        }
+    }
+    return launch_as<BN, STAGES, EPI_SILU>(mp, mq, a, ctas, s);
 }
 
 }  // namespace
@@ -741,14 +768,17 @@ VCB_EXPORT int vcb_tile_weights(const void* w, int rows, int k, int ld, int gate
 //       residual += result; out (bfloat16) = residual * gain; sumsq_out = partial sums over the features
 //       of residual^2 for every token.
 //   gated > 0: p_tiled is a gated image (vcb_tile_weights) of a [2 gated, k] matrix, rows_p = 2 gated;
-//       out (bfloat16, [rows_q][>= gated]) = act(gate) * up with gated_act 0: silu, 1: relu.
-VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused_act(const void* p, int rows_p, int ldp, const void* p_tiled, const void* q,
+//       out (bfloat16, [rows_q][>= gated]) = act(gate) * up with epi EPI_SILU or EPI_RELU;
+//   not gated, epi EPI_RELU_SQUARED or EPI_GELU (rows_q <= bn <= 128): out = act(result);
+//   epi EPI_TANH_NORM with residual and gain (sumsq_out not used): residual += result, out (bfloat16) =
+//       tanh(alpha * residual) * gain + shift, shift [rows_p] and alpha [1] float.
+VCB_EXPORT int vcb_gemm_bf16_tcgen05_epilogue(const void* p, int rows_p, int ldp, const void* p_tiled, const void* q,
                                            int rows_q, int ldq, int k, void* out, int ldc, int out_f32, int swapped,
                                            int bn, int max_ctas, float* partial, int* tickets, int n_tickets,
                                            int* status, const float* scale_sumsq, int scale_parts, int scale_ld,
                                            int scale_width, float scale_eps, float* residual, int ldr,
-                                           const float* gain, float* sumsq_out, int sumsq_ld, int gated, int gated_act,
-                                           void* stream) {
+                                           const float* gain, float* sumsq_out, int sumsq_ld, int gated, int epi,
+                                           const float* shift, const float* alpha, void* stream) {
     if (rows_p <= 0 || rows_q <= 0) return 0;
     if (k <= 0 || max_ctas < 1 || !status || !partial || !tickets) return VCB_ERR_BAD_ARG;
     // TMA needs 16-byte aligned bases and row strides
@@ -756,15 +786,18 @@ VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused_act(const void* p, int rows_p, int ld
     if (!p_tiled && ((ldp % 8) || ((uintptr_t)p & 15))) return VCB_ERR_UNSUPPORTED;
     if (bn != 16 && bn != 32 && bn != 64 && bn != 128 && bn != 256) return VCB_ERR_BAD_ARG;
     if (gated) {
-        if (gated < 0 || gated_act < 0 || gated_act > 1 || rows_p != 2 * gated || !p_tiled || !swapped || rows_q > bn || bn > 128 || out_f32 || residual ||
+        if (gated < 0 || (epi != EPI_SILU && epi != EPI_RELU) || rows_p != 2 * gated || !p_tiled || !swapped || rows_q > bn || bn > 128 || out_f32 || residual ||
             ldc < gated)
             return VCB_ERR_BAD_ARG;
         rows_p = 128 * ((gated + 63) / 64);       // rows of the image
     }
+    if (epi < EPI_SILU || epi > EPI_TANH_NORM || (epi == EPI_RELU && !gated)) return VCB_ERR_BAD_ARG;
+    if (epi > EPI_RELU && (gated || !swapped || rows_q > bn || bn > 128 || out_f32)) return VCB_ERR_UNSUPPORTED;
+    if (epi == EPI_TANH_NORM ? (!residual || !shift || !alpha) : epi > EPI_RELU && residual) return VCB_ERR_BAD_ARG;
     if (scale_sumsq || residual) {
         if (!swapped || rows_q > bn || bn > 128) return VCB_ERR_UNSUPPORTED;
         if (scale_sumsq && (scale_parts < 1 || scale_ld < rows_q || scale_width < 1)) return VCB_ERR_BAD_ARG;
-        if (residual && (!gain || !sumsq_out || out_f32 || ldr < rows_p || sumsq_ld < rows_q)) return VCB_ERR_BAD_ARG;
+        if (residual && (!gain || out_f32 || ldr < rows_p || (epi != EPI_TANH_NORM && (!sumsq_out || sumsq_ld < rows_q)))) return VCB_ERR_BAD_ARG;
     }
     const int k_slabs = (k + BK - 1) / BK;
     const int tiles_p = (rows_p + BM - 1) / BM, tiles_q = (rows_q + bn - 1) / bn;
@@ -782,16 +815,29 @@ VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused_act(const void* p, int rows_p, int ld
     GemmArgs a{out, partial, tickets, status, (const uint8_t*)p_tiled, ldc, out_f32, swapped, rows_p, rows_q,
                k_slabs, tiles_p, per, (int)total,
                scale_sumsq, scale_parts, scale_ld, scale_sumsq ? 1.0f / (float)scale_width : 0.0f, scale_eps,
-               residual, gain, sumsq_out, ldr, sumsq_ld, gated};
-    const bool relu = gated && gated_act == 1;
+               residual, gain, sumsq_out, ldr, sumsq_ld, gated, shift, alpha};
     cudaStream_t s = (cudaStream_t)stream;
     switch (bn) {
-        case 16: return launch<16, 6>(mp, mq, a, ctas, relu, s);
-        case 32: return launch<32, 5>(mp, mq, a, ctas, relu, s);
-        case 64: return max_ctas > vcb_sm_count() ? launch<64, 4>(mp, mq, a, ctas, relu, s) : launch<64, 8>(mp, mq, a, ctas, relu, s);
-        case 128: return launch<128, 6>(mp, mq, a, ctas, relu, s);
-        default: return launch<256, 4>(mp, mq, a, ctas, relu, s);
+        case 16: return launch<16, 6>(mp, mq, a, ctas, epi, s);
+        case 32: return launch<32, 5>(mp, mq, a, ctas, epi, s);
+        case 64: return max_ctas > vcb_sm_count() ? launch<64, 4>(mp, mq, a, ctas, epi, s) : launch<64, 8>(mp, mq, a, ctas, epi, s);
+        case 128: return launch<128, 6>(mp, mq, a, ctas, epi, s);
+        default: return launch<256, 4>(mp, mq, a, ctas, epi, s);
     }
+}
+
+// The same with the gated forms' activations alone.
+VCB_EXPORT int vcb_gemm_bf16_tcgen05_fused_act(const void* p, int rows_p, int ldp, const void* p_tiled, const void* q,
+                                           int rows_q, int ldq, int k, void* out, int ldc, int out_f32, int swapped,
+                                           int bn, int max_ctas, float* partial, int* tickets, int n_tickets,
+                                           int* status, const float* scale_sumsq, int scale_parts, int scale_ld,
+                                           int scale_width, float scale_eps, float* residual, int ldr,
+                                           const float* gain, float* sumsq_out, int sumsq_ld, int gated, int gated_act,
+                                           void* stream) {
+    return vcb_gemm_bf16_tcgen05_epilogue(p, rows_p, ldp, p_tiled, q, rows_q, ldq, k, out, ldc, out_f32, swapped, bn, max_ctas,
+                                          partial, tickets, n_tickets, status, scale_sumsq, scale_parts, scale_ld, scale_width,
+                                          scale_eps, residual, ldr, gain, sumsq_out, sumsq_ld, gated, gated && gated_act == 1 ? EPI_RELU : EPI_SILU,
+                                          nullptr, nullptr, stream);
 }
 
 // The same with silu in the gated form.

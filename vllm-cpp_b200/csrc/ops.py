@@ -43,6 +43,8 @@ _SIGNATURES = {
                                     _P, _I, _I, _I, _F, _P, _I, _P, _P, _I, _I, _P],
     "vcb_gemm_bf16_tcgen05_fused_act": [_P, _I, _I, _P, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P,
                                         _P, _I, _I, _I, _F, _P, _I, _P, _P, _I, _I, _I, _P],
+    "vcb_gemm_bf16_tcgen05_epilogue": [_P, _I, _I, _P, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P,
+                                       _P, _I, _I, _I, _F, _P, _I, _P, _P, _I, _I, _I, _P, _P, _P],
     "vcb_tile_weights": [_P, _I, _I, _I, _I, _P, _P],
     "vcb_repetition_penalty": [_P, _I, _P, _P, _P, _I, _I, _P],
     "vcb_sample": [_P, _I, _I, _P, _P, _P, _I, _P],
@@ -99,7 +101,7 @@ _SIGNATURES = {
     "vcb_gate_blocks": [_P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _F, _I, _P],
     "vcb_linear_recurrence": [_P, _P, _L, _P, _L, _P, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _P],
     "vcb_gated_delta_scan": [_P, _P, _P, _L, _L, _L, _P, _L, _P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _P, _I, _P],
-    "vcb_add_tanh_norm": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _F, _I, _P],
+    "vcb_add_tanh_norm": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _F, _F, _I, _P],
     "vcb_act_rows": [_P, _P, _L, _I, _I, _P],
     "vcb_state_dual": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "vcb_qk_norm_cache_write_temp": [_P, _L, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _I, _P],
@@ -261,17 +263,19 @@ def relu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
 
 
 def add_tanh_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], alpha: torch.Tensor, gain: torch.Tensor, shift: torch.Tensor,
-                  out: torch.Tensor, row_index: Optional[torch.Tensor] = None, mult: float = 1.0) -> None:
-    """out = tanh(alpha * (residual + mult * delta)) * gain + shift; the sum is written back to residual unless rows are gathered.
-    alpha float32 [1], gain and shift float32 [hidden]."""
+                  out: torch.Tensor, row_index: Optional[torch.Tensor] = None, mult: float = 1.0, delta2: Optional[torch.Tensor] = None,
+                  mult2: float = 0.0) -> None:
+    """out = tanh(alpha * (residual + mult * delta + mult2 * delta2)) * gain + shift; the sum is written back to residual unless rows
+    are gathered.  alpha float32 [1], gain and shift float32 [hidden]; delta2 (with a delta only) like delta."""
     hidden, n_rows = residual.shape[1], out.shape[0]
     _need(out.shape[1] == hidden and gain.numel() == hidden and shift.numel() == hidden and alpha.numel() == 1, "add_tanh_norm: widths differ")
     _need(delta is None or (delta.shape == residual.shape and delta.dtype == out.dtype), "add_tanh_norm: delta shape or type differs")
     _need(n_rows == residual.shape[0] if row_index is None else row_index.numel() == n_rows, "add_tanh_norm: one row read per output row")
+    _need(delta2 is None or (delta is not None and delta2.shape == delta.shape and delta2.dtype == delta.dtype), "add_tanh_norm: delta2 like delta")
     _check(lib().vcb_add_tanh_norm(_dev(residual, "residual", torch.float32), None if delta is None else _dev(delta, "delta"),
-                                   _dev(alpha, "alpha", torch.float32), _dev(gain, "gain", torch.float32), _dev(shift, "shift", torch.float32),
+                                   None if delta2 is None else _dev(delta2, "delta2"), _dev(alpha, "alpha", torch.float32), _dev(gain, "gain", torch.float32), _dev(shift, "shift", torch.float32),
                                    _dev(out, "out"), None if row_index is None else _dev(row_index, "row_index", torch.int32), n_rows, hidden,
-                                   float(mult), dtype_code(out.dtype), _stream()), "add_tanh_norm")
+                                   float(mult), float(mult2), dtype_code(out.dtype), _stream()), "add_tanh_norm")
 
 
 ROW_ACTS = {"relu_squared": 0, "gelu": 1}      # gelu by its definition, through erf
@@ -601,6 +605,15 @@ class ResidualNorm:
         return RowScale(self.sumsq, sumsq_parts(self.residual.shape[1]), self.residual.shape[1], self.eps)
 
 
+class ResidualTanhNorm:
+    """Asks a product to end a residual branch before a norm that needs no statistics: residual (float32 [tokens, features]) +=
+    result; out = bfloat16(tanh(alpha * residual) * gain + shift), the finished input of the sublayer that follows."""
+    __slots__ = ("residual", "alpha", "gain", "shift")
+
+    def __init__(self, residual: torch.Tensor, alpha: torch.Tensor, gain: torch.Tensor, shift: torch.Tensor):
+        self.residual, self.alpha, self.gain, self.shift = residual, alpha, gain, shift
+
+
 def sumsq_parts(features: int) -> int:
     """Partial sums a ResidualNorm product leaves per token: one per epilogue warp of every 128-row tile."""
     return 4 * (-(-features // 128))
@@ -608,11 +621,11 @@ def sumsq_parts(features: int) -> int:
 
 def gemm_bf16_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan=None, max_ctas: Optional[int] = None,
                       use_tiled: bool = True, x_scale: Optional[RowScale] = None,
-                      fuse: Optional[ResidualNorm] = None, gated: bool = False, gate_act: str = "silu") -> None:
+                      fuse=None, gated: bool = False, gate_act: str = "silu", act: Optional[str] = None) -> None:
     """out = x @ w^T on tcgen05 tensor cores fed by TMA (see gemm_tcgen05.cu); out bfloat16 or float32.
     When the weights are the 128-row operand and tile_weights(w) has been made, the image is used
     (``use_tiled`` False forces the tensor-map path).  ``x_scale`` and ``fuse`` (up to 128 tokens):
-    see RowScale and ResidualNorm.  ``gated``: w is a gate-and-up matrix [2 * inter, k] with a gated
+    see RowScale and ResidualNorm (or ResidualTanhNorm).  ``act`` (up to 128 tokens; a name of ROW_ACTS): out = act(x @ w^T).  ``gated``: w is a gate-and-up matrix [2 * inter, k] with a gated
     image (tile_weights(w, inter)) and out [tokens, inter] = act(x gate^T) * (x up^T), act "silu" or "relu"."""
     m, k = x.shape
     n = w.shape[0]
@@ -631,15 +644,27 @@ def gemm_bf16_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan=
               "gemm_bf16_tcgen05: sums of squares must be float32 [parts, tokens]")
         sc = (x_scale.sumsq.data_ptr(), x_scale.parts, x_scale.sumsq.stride(0), x_scale.width, x_scale.eps)
     fu = (None, 0, None, None, 0)
+    epi, extra = (GATE_ACTS[gate_act] if gated else 0), (None, None)
+    if act is not None:
+        _need(swapped and m <= bn <= 128 and out.dtype == torch.bfloat16 and fuse is None and not gated and act in PRODUCT_ACTS,
+              f"gemm_bf16_tcgen05: an activation ({sorted(PRODUCT_ACTS)}) needs the few-token form and a bfloat16 result")
+        epi = PRODUCT_ACTS[act]
     if fuse is not None:
         _need(swapped and m <= bn <= 128 and out.dtype == torch.bfloat16,
               "gemm_bf16_tcgen05: a fused residual needs the few-token form and a bfloat16 result")
-        r, g, ss = fuse.residual, fuse.gain, fuse.sumsq
+        r, g = fuse.residual, fuse.gain
         _need(r.dtype == torch.float32 and r.shape == (m, n) and r.stride(1) == 1 and g.dtype == torch.float32
               and g.shape == (n,) and g.is_contiguous(), "gemm_bf16_tcgen05: residual float32 [tokens, features], gain float32 [features]")
-        _need(ss.dtype == torch.float32 and ss.dim() == 2 and ss.stride(1) == 1 and ss.shape[0] >= sumsq_parts(n)
-              and ss.shape[1] >= m, "gemm_bf16_tcgen05: sums of squares must be float32 [sumsq_parts(features), tokens]")
-        fu = (r.data_ptr(), r.stride(0), g.data_ptr(), ss.data_ptr(), ss.stride(0))
+        if isinstance(fuse, ResidualTanhNorm):
+            _need(fuse.shift.dtype == torch.float32 and fuse.shift.shape == (n,) and fuse.shift.is_contiguous() and fuse.alpha.dtype == torch.float32
+                  and fuse.alpha.numel() == 1, "gemm_bf16_tcgen05: shift float32 [features], alpha float32 [1]")
+            fu = (r.data_ptr(), r.stride(0), g.data_ptr(), None, 0)
+            epi, extra = EPI_TANH_NORM, (fuse.shift.data_ptr(), fuse.alpha.data_ptr())
+        else:
+            ss = fuse.sumsq
+            _need(ss.dtype == torch.float32 and ss.dim() == 2 and ss.stride(1) == 1 and ss.shape[0] >= sumsq_parts(n)
+                  and ss.shape[1] >= m, "gemm_bf16_tcgen05: sums of squares must be float32 [sumsq_parts(features), tokens]")
+            fu = (r.data_ptr(), r.stride(0), g.data_ptr(), ss.data_ptr(), ss.stride(0))
     p, q = (w, x) if swapped else (x, w)
     tiled = tiled_weights_of(w, gated) if (swapped and use_tiled) else None
     if gated:
@@ -655,16 +680,18 @@ def gemm_bf16_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan=
         max_ctas = _cta_choice.get((n, k, bn, bool(gated), fuse is not None), 2 * sms if bn in (32, 64) else sms)
     partial = scratch("gemm_partial", sms * 2 * 256 * 128, out.device)
     tickets = zeroed_ints("gemm_tickets", GEMM_MAX_TICKETS, out.device)
-    _check(lib().vcb_gemm_bf16_tcgen05_fused_act(p.data_ptr(), p.shape[0], p.stride(0),
+    _check(lib().vcb_gemm_bf16_tcgen05_epilogue(p.data_ptr(), p.shape[0], p.stride(0),
                                              None if tiled is None else tiled.data_ptr(),
                                              q.data_ptr(), q.shape[0], q.stride(0), k,
                                              out.data_ptr(), out.stride(0), 1 if out.dtype == torch.float32 else 0,
                                              1 if swapped else 0, bn, min(max_ctas, 2 * sms), partial.data_ptr(),
                                              tickets.data_ptr(), GEMM_MAX_TICKETS, status_tensor(out.device).data_ptr(),
-                                             *sc, *fu, n // 2 if gated else 0, GATE_ACTS[gate_act], _stream()), "gemm_bf16_tcgen05")
+                                             *sc, *fu, n // 2 if gated else 0, epi, *extra, _stream()), "gemm_bf16_tcgen05")
 
 
 GATE_ACTS = {"silu": 0, "relu": 1}      # activations of the gated product's epilogue
+PRODUCT_ACTS = {"relu_squared": 2, "gelu": 3}      # activations of a plain product's epilogue
+EPI_TANH_NORM = 4
 
 TCGEN05_MAX_TOKENS = 128      # up to here the engine's own tcgen05 product may run; above, the library's
 _tcgen05_linear = True
@@ -898,7 +925,7 @@ def linear_fuses_norm(tokens: int, w: torch.Tensor, out_dtype=torch.bfloat16) ->
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_scale: Optional[RowScale] = None,
-           fuse: Optional[ResidualNorm] = None) -> None:
+           fuse=None) -> None:
     """out = x @ w^T.  float32: the engine's own FMA kernel.  bfloat16 with up to TCGEN05_MAX_TOKENS
     rows (decode steps, short portions): the engine's tcgen05 + TMA kernel with the weights on the
     128-row side of the tile, where the measurement at load found it faster than the library (and always
@@ -916,6 +943,16 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_scale: Optiona
         return
     _need(x_scale is None and fuse is None, "linear: the library product fuses no norm; ask linear_fuses_norm first")
     _library_mm(x, w, out)
+
+
+def linear_act(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str) -> None:
+    """out = act(x @ w^T), act a name of ROW_ACTS: in the product's epilogue where ``linear`` would run this library's tcgen05
+    product, else as a kernel after it."""
+    if x.dtype == torch.bfloat16 and linear_fuses_norm(x.shape[0], w) and _tcgen05_ok(x, w, out):
+        gemm_bf16_tcgen05(x, w, out, act=act)
+        return
+    linear(x, w, out)
+    act_rows(out, out, act)
 
 
 def linear_gated_fuses(tokens: int, w: torch.Tensor) -> bool:

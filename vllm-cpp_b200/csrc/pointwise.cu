@@ -1,8 +1,8 @@
 // Kernels that treat every coordinate by itself:
 //
-//   add_tanh_norm_kernel   the norm without statistics: x += mult * delta, out = tanh(alpha * x) * gain + shift.  The sum is
-//                          written back to the float residual stream; nothing about a row needs the whole row, so a CTA takes
-//                          any run of coordinates.
+//   add_tanh_norm_kernel   the norm without statistics: x += mult * delta (+ mult2 * delta2: two
+//                          mixers' results), out = tanh(alpha * x) * gain + shift.  The sum is written back to the float
+//                          residual stream; nothing about a row needs the whole row, so a CTA takes any run of coordinates.
 //   act_rows_kernel        the activation between the two matrices of a feed-forward without a gate: the square of relu, or
 //                          gelu by its definition z Phi(z), Phi through erf.
 //
@@ -56,8 +56,9 @@ template <> struct PwVec<__nv_bfloat16, 8> {
 // Grid-stride over vectors of V coordinates; the row and column of a vector advance with the stride.
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
-add_tanh_norm_kernel(float* __restrict__ residual, const T* __restrict__ delta, const float* __restrict__ alpha, const float* __restrict__ gain,
-                     const float* __restrict__ shift, T* __restrict__ out, const int* __restrict__ row_index, int n_rows, int hidden, float mult) {
+add_tanh_norm_kernel(float* __restrict__ residual, const T* __restrict__ delta, const T* __restrict__ delta2, const float* __restrict__ alpha,
+                     const float* __restrict__ gain, const float* __restrict__ shift, T* __restrict__ out, const int* __restrict__ row_index,
+                     int n_rows, int hidden, float mult, float mult2) {
     const int vpr = hidden / V;                          // vectors per row
     const float slope = *alpha;
     pdl_start();
@@ -74,6 +75,11 @@ add_tanh_norm_kernel(float* __restrict__ residual, const T* __restrict__ delta, 
             PwVec<T, V>::load(delta + row * hidden + c, d);
 #pragma unroll
             for (int i = 0; i < V; ++i) x[i] = fmaf(mult, d[i], x[i]);
+            if (delta2) {
+                PwVec<T, V>::load(delta2 + row * hidden + c, d);
+#pragma unroll
+                for (int i = 0; i < V; ++i) x[i] = fmaf(mult2, d[i], x[i]);
+            }
             if (!row_index) PwVec<float, V>::store(residual + row * hidden + c, x);
         }
 #pragma unroll
@@ -83,28 +89,28 @@ add_tanh_norm_kernel(float* __restrict__ residual, const T* __restrict__ delta, 
 }
 
 template <typename T, int V>
-static int launch_tanh_norm(float* residual, const void* delta, const float* alpha, const float* gain, const float* shift, void* out,
-                            const int* row_index, int n_rows, int hidden, float mult, cudaStream_t s) {
+static int launch_tanh_norm(float* residual, const void* delta, const void* delta2, const float* alpha, const float* gain, const float* shift, void* out,
+                            const int* row_index, int n_rows, int hidden, float mult, float mult2, cudaStream_t s) {
     const long long want = ((long long)n_rows * (hidden / V) + 255) / 256, cap = (long long)vcb_sm_count() * 16;
-    vcb_launch(add_tanh_norm_kernel<T, V>, (int)(want < cap ? want : cap), 256, 0, s, residual, (const T*)delta, alpha, gain, shift, (T*)out,
-               row_index, n_rows, hidden, mult);
+    vcb_launch(add_tanh_norm_kernel<T, V>, (int)(want < cap ? want : cap), 256, 0, s, residual, (const T*)delta, (const T*)delta2, alpha, gain,
+               shift, (T*)out, row_index, n_rows, hidden, mult, mult2);
     return vcb_last_error();
 }
 
 // alpha: float [1].  row_index (may be null): output row o reads row row_index[o], and nothing is written back.
-VCB_EXPORT int vcb_add_tanh_norm(float* residual, const void* delta, const float* alpha, const float* gain, const float* shift, void* out,
-                                 const int* row_index, int n_rows, int hidden, float mult, int dtype, void* stream) {
+VCB_EXPORT int vcb_add_tanh_norm(float* residual, const void* delta, const void* delta2, const float* alpha, const float* gain, const float* shift,
+                                 void* out, const int* row_index, int n_rows, int hidden, float mult, float mult2, int dtype, void* stream) {
     if (n_rows <= 0) return 0;
-    if (!residual || !alpha || !gain || !shift || !out || hidden <= 0) return VCB_ERR_BAD_ARG;
+    if (!residual || (delta2 && !delta) || !alpha || !gain || !shift || !out || hidden <= 0) return VCB_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
-    const bool aligned = !(((uintptr_t)residual | (uintptr_t)delta | (uintptr_t)gain | (uintptr_t)shift | (uintptr_t)out) & 15);
+    const bool aligned = !(((uintptr_t)residual | (uintptr_t)delta | (uintptr_t)delta2 | (uintptr_t)gain | (uintptr_t)shift | (uintptr_t)out) & 15);
     if (dtype == VCB_F32) {
-        if (aligned && hidden % 4 == 0) return launch_tanh_norm<float, 4>(residual, delta, alpha, gain, shift, out, row_index, n_rows, hidden, mult, s);
-        return launch_tanh_norm<float, 1>(residual, delta, alpha, gain, shift, out, row_index, n_rows, hidden, mult, s);
+        if (aligned && hidden % 4 == 0) return launch_tanh_norm<float, 4>(residual, delta, delta2, alpha, gain, shift, out, row_index, n_rows, hidden, mult, mult2, s);
+        return launch_tanh_norm<float, 1>(residual, delta, delta2, alpha, gain, shift, out, row_index, n_rows, hidden, mult, mult2, s);
     }
     if (dtype != VCB_BF16) return VCB_ERR_BAD_ARG;
-    if (aligned && hidden % 8 == 0) return launch_tanh_norm<__nv_bfloat16, 8>(residual, delta, alpha, gain, shift, out, row_index, n_rows, hidden, mult, s);
-    return launch_tanh_norm<__nv_bfloat16, 1>(residual, delta, alpha, gain, shift, out, row_index, n_rows, hidden, mult, s);
+    if (aligned && hidden % 8 == 0) return launch_tanh_norm<__nv_bfloat16, 8>(residual, delta, delta2, alpha, gain, shift, out, row_index, n_rows, hidden, mult, mult2, s);
+    return launch_tanh_norm<__nv_bfloat16, 1>(residual, delta, delta2, alpha, gain, shift, out, row_index, n_rows, hidden, mult, mult2, s);
 }
 
 // ------------------------------------------------------------------------------------- activations

@@ -89,10 +89,10 @@ __global__ void __launch_bounds__(512) state_dual_walk_kernel(DualArgs a) {
             bs[i] = n < a.N ? to_f32<T>(bp[(size_t)(t0 + t) * a.ldb + n]) : 0.0f;
             cs[i] = n < a.N ? to_f32<T>(cp[(size_t)(t0 + t) * a.ldc + n]) : 0.0f;
         }
-        if (tid < tc) {
-            const float dt = sd_softplus(to_f32<T>(((const T*)a.dt_pre)[(size_t)(t0 + tid) * a.lddt + h]) + bias);
-            ts[2 * tid] = exp2f(a2 * dt);
-            ts[2 * tid + 1] = dt;
+        for (int t = tid; t < tc; t += nthreads) {
+            const float dt = sd_softplus(to_f32<T>(((const T*)a.dt_pre)[(size_t)(t0 + t) * a.lddt + h]) + bias);
+            ts[2 * t] = exp2f(a2 * dt);
+            ts[2 * t + 1] = dt;
         }
         __syncthreads();
         for (int t = 0; t < tc; ++t) {

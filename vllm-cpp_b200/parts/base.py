@@ -278,6 +278,12 @@ class Norm(Part):
         (see ops.ResidualNorm, ops.RowScale), and no norm kernel runs.  None: the norm runs by itself."""
         return None
 
+    def end_of_branch(self, residual: torch.Tensor):
+        """What to hand, as ``fuse``, to the product that ends the residual branch before this norm, if the norm is one whose result
+        that product can finish itself, coordinate by coordinate (ops.ResidualTanhNorm); None if it needs the whole row or a kernel
+        of its own."""
+        return None
+
 
 class Mixer(Part):
     """Mixes information between the tokens of a request (attention here)."""
@@ -290,6 +296,11 @@ class Mixer(Part):
         """True if, for a step of ``n_tokens``, ``forward`` accepts ``x_scale`` (an ops.RowScale its first
         product applies to x) and ``fuse`` (an ops.ResidualNorm its last product performs instead of
         writing ``out`` plainly).  The block passes those keywords only after a yes."""
+        return False
+
+    def ends_branch(self, n_tokens: int) -> bool:
+        """True if, for a step of ``n_tokens``, ``forward`` accepts ``fuse`` (what Norm.end_of_branch gave), which its last product
+        performs instead of writing ``out`` plainly."""
         return False
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext, cache, writes_cache: bool,
@@ -332,6 +343,10 @@ class Scale(Part):
 class FeedForward(Part):
     def fuses_norm(self, n_tokens: int) -> bool:
         """As Mixer.fuses_norm."""
+        return False
+
+    def ends_branch(self, n_tokens: int) -> bool:
+        """As Mixer.ends_branch."""
         return False
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, step: StepContext, ws: Workspace) -> None:
@@ -410,6 +425,11 @@ class Block:
         """(gain, eps) of the norm this block starts with if, for a step of ``n_tokens``, the block can
         take its input as ``delta`` = residual * gain with the rows' factor still to be applied
         (``pending`` an ops.RowScale); None if it wants the residual stream as it is."""
+        return None
+
+    def accepts_end_of_branch(self, n_tokens: int, residual: torch.Tensor):
+        """What the norm this block starts with hands to the product before it (Norm.end_of_branch) if the block takes its input
+        finished (``pending`` a NormedInput); None if it runs its own norm."""
         return None
 
     def accepts_normed(self, n_tokens: int):

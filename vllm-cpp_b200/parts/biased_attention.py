@@ -138,14 +138,17 @@ class BiasedWindowAttention(PagedAttentionKernels):
         return (workspace_piece((n_tokens, self.in_width()), self.dtype) + workspace_piece((n_tokens, self.nh * self.dk), self.dtype)
                 + workspace_piece((n_tokens, self.nh * self.dv), self.dtype))
 
-    def forward(self, x, out, step, cache, writes_cache, ws):
+    def ends_branch(self, n_tokens):
+        return ops.linear_fuses_norm(n_tokens, self.w_o)
+
+    def forward(self, x, out, step, cache, writes_cache, ws, fuse=None):
         mark = ws.mark()
         proj = ws.take((x.shape[0], self.in_width()), self.dtype)
         ops.linear(x, self.w_in, proj)
-        self.forward_projected(proj, out, step, cache, writes_cache, ws)
+        self.forward_projected(proj, out, step, cache, writes_cache, ws, fuse)
         ws.release(mark)
 
-    def forward_projected(self, proj, out, step, cache, writes_cache, ws):
+    def forward_projected(self, proj, out, step, cache, writes_cache, ws, fuse=None):
         """``forward`` from the rows of the input product on (a mixer that shares its input product calls this)."""
         n = proj.shape[0]
         mark = ws.mark()
@@ -168,5 +171,5 @@ class BiasedWindowAttention(PagedAttentionKernels):
         else:
             ops.attention_biased(q, pages, attn, gate, step.positions, step.req_of_token, block_table, self.bias,
                                  window=self.window, scale=self.scale, cap=self.cap, sink=self.sink, keep_first=self.keep_first, **sizes)
-        ops.linear(attn, self.w_o, out)
+        ops.linear(attn, self.w_o, out, fuse=fuse)
         ws.release(mark)

@@ -10,7 +10,9 @@ split (``Norm.split``), no norm kernel runs: the product that ends the branch be
 norm adds its result to the residual stream, multiplies by the gain and leaves the rows'
 sums of squares, and the product after the norm applies the factor (ops.ResidualNorm,
 ops.RowScale).  That holds for the norm inside the layer and for the one the next layer
-starts with.
+starts with.  A norm that needs no statistics (``Norm.end_of_branch``) is finished by the product
+before it, and the product after it reads its input as it is; where the mixer is two mixers whose
+results are added (``plain_scales``), the norm's own kernel adds both.
 """
 from __future__ import annotations
 
@@ -41,9 +43,35 @@ class PreNormBlock(Block):
         return self.mixer_norm.split() if self.mixer.fuses_norm(n_tokens) else None
 
     def workspace_bytes(self, n_tokens, n_reqs, hidden, dtype):
-        own = 2 * workspace_piece((n_tokens, hidden), dtype) \
+        own = (3 if self._pair_scales() else 2) * workspace_piece((n_tokens, hidden), dtype) \
             + workspace_piece((ops.sumsq_parts(hidden), n_tokens), torch.float32)
         return own + super().workspace_bytes(n_tokens, n_reqs, hidden, dtype)
+
+    def accepts_end_of_branch(self, n_tokens, residual):
+        # (a layer of a mixer alone writes its result where its finished input would lie)
+        return self.mixer_norm.end_of_branch(residual) if self.mult == 1.0 and self.has_ff else None
+
+    def _end_for(self, next_block, part, residual):
+        """What ``part``'s last product does for the norm the next block starts with, or None."""
+        if next_block is None or self.mult != 1.0 or not part.ends_branch(residual.shape[0]):
+            return None
+        return next_block.accepts_end_of_branch(residual.shape[0], residual)
+
+    def _pair_scales(self):
+        """The factors of the mixer's two results where the norm after it joins them itself."""
+        if not self.has_ff or self.mult != 1.0 or not hasattr(self.feed_forward_norm, "forward_pair"):
+            return None
+        offer = getattr(self.mixer, "plain_scales", None)
+        return offer() if offer else None
+
+    def _run_feed_forward(self, h, delta, residual, step, ws, next_block):
+        """The feed-forward on its normed input, its result left in ``delta`` or finished for the next block."""
+        end = self._end_for(next_block, self.feed_forward, residual)
+        if end is None:
+            self.feed_forward.forward(h, delta, step, ws)
+            return self._left()
+        self.feed_forward.forward(h, delta, step, ws, fuse=end)
+        return NormedInput()
 
     def forward(self, residual, delta, pending, step, cache, writes_cache, ws, next_block=None, carry=None):
         mark = ws.mark()
@@ -52,22 +80,39 @@ class PreNormBlock(Block):
         mixed = ws.take((n, hidden), delta.dtype)
         if isinstance(pending, ops.RowScale):
             x, scale_kw = delta, {"x_scale": pending}
+        elif isinstance(pending, NormedInput):
+            x, scale_kw = delta, {}
         else:
             came = pending_mult(pending)               # norms of other makes know no factor; they are asked only for one
             self.mixer_norm.forward(residual, delta if pending else None, h, **({} if came == 1.0 else {"mult": came}))
             x, scale_kw = h, {}
         if not self.has_ff:
-            self.mixer.forward(x, delta, step, cache, writes_cache, ws, **scale_kw)
+            end = self._end_for(next_block, self.mixer, residual)
+            self.mixer.forward(x, delta, step, cache, writes_cache, ws, **({"fuse": end} if end is not None else {}), **scale_kw)
             ws.release(mark)
-            return self._left()
+            return self._left() if end is None else NormedInput()
+        scales = self._pair_scales()
+        if scales is not None:
+            other = ws.take((n, hidden), delta.dtype)
+            self.mixer.forward_pair(x, mixed, other, step, cache, writes_cache, ws)
+            self.feed_forward_norm.forward_pair(residual, mixed, other, h, *scales)
+            pending = self._run_feed_forward(h, delta, residual, step, ws, next_block)
+            ws.release(mark)
+            return pending
+        end = self.feed_forward_norm.end_of_branch(residual) if self.mult == 1.0 and self.mixer.ends_branch(n) else None
+        if end is not None:
+            self.mixer.forward(x, mixed, step, cache, writes_cache, ws, fuse=end, **scale_kw)
+            pending = self._run_feed_forward(mixed, delta, residual, step, ws, next_block)
+            ws.release(mark)
+            return pending
         inner = self.feed_forward_norm.split()
         if (self.mult != 1.0 or inner is None or carry is None
                 or not (self.mixer.fuses_norm(n) and self.feed_forward.fuses_norm(n))):
             self.mixer.forward(x, mixed, step, cache, writes_cache, ws, **scale_kw)
             self.feed_forward_norm.forward(residual, mixed, h, **({} if self.mult == 1.0 else {"mult": self.mult}))
-            self.feed_forward.forward(h, delta, step, ws)
+            pending = self._run_feed_forward(h, delta, residual, step, ws, next_block)
             ws.release(mark)
-            return self._left()
+            return pending
         # the mixer's last product ends its branch: residual += ..., mixed = residual * gain
         sumsq = ws.take((ops.sumsq_parts(hidden), n), torch.float32)
         ends = ops.ResidualNorm(residual, inner[0], sumsq, inner[1])

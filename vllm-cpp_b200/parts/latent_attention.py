@@ -233,7 +233,10 @@ class RotaryLatentAttention(PagedAttentionKernels):
                 + workspace_piece((n_tokens, h * self.vd), self.dtype))
 
     # -- run
-    def forward(self, x, out, step, cache, writes_cache, ws):
+    def ends_branch(self, n_tokens):
+        return ops.linear_fuses_norm(n_tokens, self.w_o)
+
+    def forward(self, x, out, step, cache, writes_cache, ws, fuse=None):
         n, h, qd = x.shape[0], self.heads, self.qk + self.rot
         mark = ws.mark()
         proj = ws.take((n, self.w_rows()), self.dtype)
@@ -261,5 +264,5 @@ class RotaryLatentAttention(PagedAttentionKernels):
         o = ws.take((n, h * self.vd), self.dtype)
         gate = proj[:, g0:] if self.gate != "none" else None
         ops.headwise_linear(o_lat, self.w_uv, o, gate=gate, gate_per_head=self.gate == "head")
-        ops.linear(o, self.w_o, out)
+        ops.linear(o, self.w_o, out, fuse=fuse)
         ws.release(mark)

@@ -130,10 +130,12 @@ class TwoLayerMLP(FeedForward):
     def workspace_bytes(self, n_tokens, n_reqs):
         return workspace_piece((n_tokens, self.inter), self.dtype)
 
-    def forward(self, x, out, step, ws):
+    def ends_branch(self, n_tokens):
+        return ops.linear_fuses_norm(n_tokens, self.w_down)
+
+    def forward(self, x, out, step, ws, fuse=None):
         mark = ws.mark()
         act = ws.take((x.shape[0], self.inter), self.dtype)
-        ops.linear(x, self.w_up, act)
-        ops.act_rows(act, act, self.activation)
-        ops.linear(act, self.w_down, out)
+        ops.linear_act(x, self.w_up, act, self.activation)           # few tokens: product and activation in one kernel
+        ops.linear(act, self.w_down, out, fuse=fuse)
         ws.release(mark)

@@ -136,8 +136,15 @@ class TanhNorm(Norm):
         self.weight, self.bias = tensors[self.tensor_name].contiguous(), tensors[self.bias_name].contiguous()
         self.alpha = tensors[self.alpha_name].reshape(1).to(torch.float32).contiguous()
 
+    def end_of_branch(self, residual):
+        return ops.ResidualTanhNorm(residual, self.alpha, self.weight, self.bias)
+
     def forward(self, residual, delta, out, row_index=None, mult=1.0):
         ops.add_tanh_norm(residual, delta, self.alpha, self.weight, self.bias, out, row_index, mult)
+
+    def forward_pair(self, residual, a, b, out, mult_a, mult_b):
+        """residual += mult_a * a + mult_b * b, then the norm: the results of two mixers side by side, joined here."""
+        ops.add_tanh_norm(residual, a, self.alpha, self.weight, self.bias, out, None, mult_a, b, mult_b)
 
 
 @register_norm("none")

@@ -76,6 +76,11 @@ class ParallelMixers(Mixer):
             return None
         return self.w_left, self.w_right, self.left_scale, self.right_scale, self.result_eps
 
+    def plain_scales(self):
+        """(left scale, right scale) if the two results are added as they are, for an arrangement whose norm kernel joins them
+        itself; None if they are normed first."""
+        return (self.left_scale, self.right_scale) if self.result_eps is None else None
+
     def forward_pair(self, x, a, b, step, cache, writes_cache, ws):
         """The two members' results as they are."""
         if self.w_in is None:
