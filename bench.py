@@ -714,7 +714,7 @@ def decode_step_bytes(model, cache, batch, context):
     el = model.embed.element_size()
     for spec in flatten_specs(model.cache_specs()):
         if isinstance(spec, PagedKVSpec):
-            keys = min(context, spec.window) if spec.window else context // spec.stride
+            keys = min(context, spec.window + spec.keep_first) if spec.window else context // spec.stride
             total += batch * keys * spec.planes * spec.num_kv_heads * spec.head_dim * el
         elif isinstance(spec, StateSpec):
             n = 4
@@ -1642,6 +1642,247 @@ def kasuvik_attention_kernels(z, add, rnd):
                     bytes_=batch * keys * 2 * nkv * d * 2)
 
 
+# ------------------------------------------------------------------- the Rufisun design beside Retodra
+# Layer sizes that resemble real models'.  Rufisun: attention over a window and the first tokens with a dense feed-forward, latent
+# attention with routed experts, attention beside a state space in its dual form with routed experts, attention with routed experts.
+# Retodra (gated linear attention with dense feed-forwards in turn with windowed, capped and biased attention beside lightning
+# attention with routed experts) at equal width, heads, kv heads, head size, window, feed-forward widths and experts is the nearest
+# model the engine has.
+RUFISUN_SIZES = {"2k": dict(width=2048, heads=16, kv_heads=4, dim=128, ff=8192, experts=16, top=2, expert_ff=2048, layers=4, groups=4),
+                 "4k": dict(width=4096, heads=32, kv_heads=8, dim=128, ff=14336, experts=32, top=4, expert_ff=2048, layers=4, groups=8)}
+RUFISUN_VOCAB, RUFISUN_CONTEXT, RUFISUN_PROMPT, RUFISUN_WINDOW, RUFISUN_KEEP = 32000, 2048, 2048, 1024, 16
+RUFISUN_STATE, RUFISUN_VDIM = 128, 64
+
+
+def rufisun_config(size):
+    z = RUFISUN_SIZES[size]
+    w, h, d = z["width"], z["heads"], z["dim"]
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}, "shared": {"ff": z["expert_ff"]}}
+    heads = {"heads": h, "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5}
+    att = {"type": "attention", "mixer": dict(heads, bias_max=float(RUFISUN_WINDOW), mask={"size": RUFISUN_WINDOW, "keep_first": RUFISUN_KEEP})}
+    lat = {"type": "latent_attention", "mixer": {"heads": h, "dim": 96, "rot_dim": 32, "vdim": 96, "kv_rank": 96, "q_rank": 3 * w // 8, "scale": 128 ** -0.5,
+                                                 "rot": {"base": 1e4, "dims": 32, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    par = {"type": "parallel", "mixer": {
+        "left": dict(heads, softcap=30.0, q_temp={"coef": 0.1, "every": 1024}), "left_scale": 1.0, "right_scale": 1.0,
+        "right": {"heads": 2 * w // RUFISUN_VDIM, "vdim": RUFISUN_VDIM, "state": RUFISUN_STATE, "groups": z["groups"], "conv": 4, "norm_groups": z["groups"]}}}
+    layers = [dict(att, mlp=dense), dict(lat, mlp=moe), dict(par, mlp=moe), dict(att, mlp=moe)]
+    return {"architecture": "Rufisun", "vocab": RUFISUN_VOCAB, "width": w, "norm": {"eps": 1e-6}, "layers": [layers[i % 4] for i in range(z["layers"])]}
+
+
+def run_rufisun(a) -> int:
+    """Prefill and decode throughput of the Rufisun design beside Retodra at equal layer sizes (random weights, synthetic cache
+    contents), and the design's own kernels alone beside the like kernels of the engine's other models with their share of the
+    measured peaks.  One JSON line."""
+    import numpy as np
+    peaks = load_peaks()
+    steps, warmup = max(1, a.steps), max(3, a.warmup)
+    rng = np.random.default_rng(0)
+    sampler = ClockSampler()
+    sampler.start()
+    sampler.mark("decode")
+    out = {"metric": "prefill and decode tok/s of Rufisun beside Retodra at equal layer sizes (bf16, random weights)",
+           "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic", "sizes": {}, "peaks": peaks}
+    sizes = a.rufisun.split(",") if a.rufisun != "all" else sorted(RUFISUN_SIZES)
+    for size in sizes:
+        args = (steps, warmup, rng, peaks, RUFISUN_VOCAB, RUFISUN_CONTEXT, RUFISUN_PROMPT)
+        out["sizes"][size] = {"layers": RUFISUN_SIZES[size], "rufisun": measure_design(rufisun_config(size), (8, 64), *args),
+                              "retodra": measure_design(dict(retodra_configs(size)[0], vocab=RUFISUN_VOCAB), (8, 64), *args)}
+    if not a.skip_points:
+        out["kernels"] = rufisun_kernels(RUFISUN_SIZES[sizes[-1]], peaks)
+    out["clocks"] = sampler.stop()
+    big = out["sizes"][sizes[-1]]
+    out.update(value=big["rufisun"]["decode"]["8"]["tok_s"], unit=f"tokens/s (Rufisun, {sizes[-1]}-wide layers, batch 8)",
+               higher_is_better=True, gpu_launches=big["rufisun"]["decode"]["8"]["launches_per_step"] * steps,
+               config={"sizes": RUFISUN_SIZES, "context": RUFISUN_CONTEXT, "prompt": RUFISUN_PROMPT, "window": RUFISUN_WINDOW, "keep_first": RUFISUN_KEEP,
+                       "state": RUFISUN_STATE, "l2": "a step's weights exceed the 126 MB of L2"})
+    print(json.dumps(out))
+    return 0
+
+
+def rufisun_kernels(z, peaks):
+    """The design's own kernels alone at one layer size, each beside the like kernel of another model of the engine:
+    [{kernel, like, us, GB/s or TFLOP/s, share of the measured peak}, ...] (CUDA graphs on rotating buffers)."""
+    import torch
+    from vllm_cpp_b200.csrc import ops
+    h, bf, dev = z["width"], torch.bfloat16, "cuda"
+    rows = []
+
+    def rnd(*shape, dtype=bf, scale=1.0):
+        return (torch.randn(*shape, device=dev) * scale).to(dtype)
+
+    def add(name, like, fn, copies, bytes_=0, flops=0, peak=None):
+        us = ops.time_in_graph(fn, reps=max(4, copies))
+        rate = bytes_ / us / 1e3 if bytes_ else flops / us / 1e6
+        row = {"kernel": name, "like": like, "us": round(us, 2), ("gb_s" if bytes_ else "tflop_s"): round(rate, 1)}
+        if bytes_ or peak != "none":
+            row["of_peak"] = round(rate / (peaks["hbm_gbs"] if bytes_ else peaks["bf16_tflops"]), 4)
+        rows.append(row)
+
+    alpha, gain, ff = torch.full((1,), 0.5, device=dev), torch.ones(h, device=dev), z["ff"]
+    # ---- rows
+    for t in (64, 2048):
+        c = 6 if t == 64 else 3
+        x = [rnd(t, h, dtype=torch.float32) for _ in range(c)]
+        ya, yb, o1 = ([rnd(t, h) for _ in range(c)] for _ in range(3))
+        add(f"addition + norm by tanh, {t} tokens", "", lambda i: ops.add_tanh_norm(x[i % c], ya[i % c], alpha, gain, gain, o1[i % c]), c, bytes_=t * h * 12)
+        add(f"Qwen2: addition + RMS norm, {t} tokens", "like the one above", lambda i: ops.add_rmsnorm(x[i % c], ya[i % c], gain, o1[i % c], 1e-6), c, bytes_=t * h * 12)
+        add(f"two results joined + addition + norm by tanh, {t} tokens", "", lambda i: ops.add_tanh_norm(
+            x[i % c], ya[i % c], alpha, gain, gain, o1[i % c], None, 0.5, yb[i % c], 0.5), c, bytes_=t * h * 14)
+        add(f"Kasuvik: two results normed and joined + post norm + addition + next norm, {t} tokens", "like the one above", lambda i: ops.pair_norm(
+            ya[i % c], yb[i % c], gain, gain, 0.5, 0.5, 1e-6, o1[i % c], x=x[i % c], gain=gain, eps=1e-6, next_gain=gain, next_eps=1e-6), c, bytes_=t * h * 14)
+        gu, act = [rnd(t, 2 * ff) for _ in range(c)], torch.empty(t, ff, dtype=bf, device=dev)
+        up = [g[:, :ff].contiguous() for g in gu]
+        for name in ("relu_squared", "gelu"):
+            add(f"{name}, width {ff}, {t} tokens", "", lambda i: ops.act_rows(up[i % c], act, name), c, bytes_=t * ff * 4)
+        add(f"Qwen2: silu(gate) * up, width {ff}, {t} tokens", "like the two above", lambda i: ops.silu_mul(gu[i % c], act), c, bytes_=t * ff * 6)
+        I = 2 * h
+        yf, zz, w = [rnd(t, I, dtype=torch.float32) for _ in range(c)], [rnd(t, I) for _ in range(c)], torch.ones(I, device=dev)
+        out = torch.empty(t, I, dtype=bf, device=dev)
+        for first in (True, False):
+            add(f"{'' if first else 'Retodra: '}gate {'before' if first else 'after'} the norm, {I} channels in {z['groups']} parts, {t} tokens",
+                "" if first else "like the one above", lambda i: ops.gated_group_norm(
+                    yf[i % c], zz[i % c], w, out, group=I // z["groups"], eps=1e-6, gate_act="silu", gate_first=first), c, bytes_=t * I * 8)
+        del x, ya, yb, o1, gu, up, yf, zz
+    # ---- products of a decode step with what their epilogues do, and the experts' products
+    for t in (8, 64):
+        c = 4
+        xs, res, out = rnd(t, h), rnd(t, h, dtype=torch.float32), torch.empty(t, h, dtype=bf, device=dev)
+        up, down = [rnd(ff, h, scale=0.02) for _ in range(c)], [rnd(h, ff, scale=0.02) for _ in range(c)]
+        both = [rnd(2 * ff, h, scale=0.02) for _ in range(c)]
+        for m in up + down:
+            ops.tile_weights(m)
+        for m in both:
+            ops.tile_weights(m, ff)
+        act, wide = torch.empty(t, ff, dtype=bf, device=dev), rnd(t, ff)
+        sumsq = torch.empty(ops.sumsq_parts(h), t, device=dev)
+        add(f"up product [{ff}, {h}] + square of relu, {t} tokens", "", lambda i: ops.gemm_bf16_tcgen05(xs, up[i % c], act, act="relu_squared"), c, bytes_=ff * h * 2)
+        add(f"Qwen2: gate-and-up product [{2 * ff}, {h}] + silu, {t} tokens", "like the one above",
+            lambda i: ops.gemm_bf16_tcgen05(xs, both[i % c], act, gated=True), c, bytes_=2 * ff * h * 2)
+        add(f"down product [{h}, {ff}] + addition + norm by tanh, {t} tokens", "", lambda i: ops.gemm_bf16_tcgen05(
+            wide, down[i % c], out, fuse=ops.ResidualTanhNorm(res, alpha, gain, gain)), c, bytes_=ff * h * 2)
+        add(f"Qwen2: down product [{h}, {ff}] + addition + sums of squares, {t} tokens", "like the one above", lambda i: ops.gemm_bf16_tcgen05(
+            wide, down[i % c], out, fuse=ops.ResidualNorm(res, gain, sumsq, 1e-6)), c, bytes_=ff * h * 2)
+        del up, down, both
+    E, top, ef = z["experts"], z["top"], z["expert_ff"]
+    w1, w2 = rnd(E, ef, h, scale=0.02), rnd(E, 2 * ef, h, scale=0.02)
+    for t in (8, 64, 2048):
+        tm, pairs = ops.moe_tile_rows(t, top, E), t * top
+        tiles = ops.moe_max_tiles(t, top, E, tm)
+        ids = torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(t)]).to(torch.int32).contiguous()
+        ints = [torch.empty(n, dtype=torch.int32, device=dev) for n in (pairs, pairs, tiles, tiles, tiles, 4)]
+        wts, rs = torch.rand(t, top, device=dev), torch.empty(pairs, device=dev)
+        ops.moe_sort(ids, E, tm, *ints, wts, rs)
+        st, _, te, t0, tr, meta = ints
+        xs, act = rnd(t, h), torch.empty(pairs, ef, dtype=bf, device=dev)
+        used = int(torch.unique(ids).numel())
+        size = (lambda n: dict(bytes_=used * n * h * 2)) if t <= 64 else (lambda n: dict(flops=2.0 * pairs * n * h))
+        add(f"experts' first product + gelu of the weighted input, {E} of {ef}, top {top}, {t} tokens", "", lambda i: ops.moe_expert_gemm(
+            xs, w1, act, st, te, t0, tr, meta, tiles, tm, gated=False, gelu=True, row_scale=rs), 4, **size(ef))
+        add(f"Lutodra: experts' gate-and-up product + silu, {E} of {ef}, top {top}, {t} tokens", "like the one above", lambda i: ops.moe_expert_gemm(
+            xs, w2, act, st, te, t0, tr, meta, tiles, tm, gated=True, limit=float("inf"), alpha=1.0, up_shift=0.0), 4, **size(2 * ef))
+    del w1, w2
+    # ---- the state space: single tokens of a batch, then a prompt
+    N, P, G = RUFISUN_STATE, RUFISUN_VDIM, z["groups"]
+    H, J = 2 * h // P, 4
+    I, C = 2 * h, 2 * h + 2 * G * N
+    for n_reqs, per in ((8, 1), (64, 1), (1, RUFISUN_PROMPT)):
+        t, c = n_reqs * per, 3
+        what = f"decode, batch {n_reqs}" if per == 1 else f"prompt of {per}"
+        q_start = torch.arange(0, t + 1, per, dtype=torch.int32, device=dev)
+        slots = torch.arange(n_reqs, dtype=torch.int32, device=dev)
+        row, dt, y = [rnd(t, C) for _ in range(c)], rnd(t, H), torch.empty(t, I, device=dev)
+        one, a2 = torch.ones(H, device=dev), -torch.rand(H, device=dev) - 0.05
+        st = [torch.zeros(n_reqs, H, N, P, device=dev) for _ in range(c)]
+        size = dict(bytes_=n_reqs * H * N * P * 8 + t * (C + 2 * I) * 2) if per == 1 else dict(flops=4.0 * t * H * N * P, peak="none")
+        add(f"state space in its dual form, {H} heads of {N} x {P}, {what}", "", lambda i: ops.state_dual(
+            row[i % c][:, :I], row[i % c][:, I:I + G * N], row[i % c][:, I + G * N:], dt, one, a2, one, st[i % c], y, q_start, slots, n_reqs, per, num_groups=G),
+            c, **size)
+        q, k, v = rnd(t, H * N), rnd(t, H * N), rnd(t, I)
+        pieces = None
+        if per > 1:
+            starts, per_req = ops.scan_pieces([per])
+            count = len(starts) - 1
+            pieces = {"start": torch.from_numpy(starts).to(dev), "req": torch.from_numpy(per_req).to(dev), "slots": torch.arange(count, dtype=torch.int32, device=dev),
+                      "count": count, "state": torch.empty(count, H, N, P, device=dev), "qp": torch.empty(t, H * N, device=dev), "dtot": torch.empty(count, H, N, device=dev)}
+        size = dict(bytes_=n_reqs * H * N * P * 8 + t * (2 * H * N + 3 * I) * 2) if per == 1 else dict(flops=4.0 * t * H * N * P, peak="none")
+        add(f"Retodra: decaying matrix state, {H} heads of {N} x {P}, {what}", "like the one above", lambda i: ops.decayed_state_scan(
+            q, k, v, st[i % c], y, q_start, slots, n_reqs, num_heads=H, decay_const=one, pieces=pieces), c, **size)
+        taps, bias, window, u = rnd(C, J, dtype=torch.float32), torch.zeros(C, device=dev), torch.zeros(n_reqs, J - 1, C, device=dev), torch.empty(t, C, dtype=bf, device=dev)
+        add(f"causal convolution of {J} taps + silu, {C} channels, {what}", "Kasuvik runs the same kernel", lambda i: ops.causal_conv(
+            row[i % c], taps, window, u, q_start, slots, n_reqs, per, bias=bias, act="silu"), c, bytes_=t * C * 4 + 2 * n_reqs * (J - 1) * C * 4)
+        del row, dt, y, st, q, k, v, pieces
+    rufisun_attention_kernels(z, add, rnd)
+    ops.check_status()
+    return rows
+
+
+def rufisun_attention_kernels(z, add, rnd):
+    """Cache writes with growing queries, attention over a window and kept first tokens (distance bias, sink, two-term weights),
+    capped attention with a sink, and latent attention with a sink, beside the like kernels of Retodra, Lutodra and Gipinex."""
+    import numpy as np
+    import torch
+    from vllm_cpp_b200.config.model_spec import PartSpec
+    from vllm_cpp_b200.csrc import ops
+    from vllm_cpp_b200.engine.runner import HostStep
+    from vllm_cpp_b200.parts.attention import PagedAttention
+    h, nh, nkv, d, page, bf, dev = z["width"], z["heads"], z["kv_heads"], z["dim"], 16, torch.bfloat16, "cuda"
+    W, keep, T = RUFISUN_WINDOW, RUFISUN_KEEP, RUFISUN_PROMPT
+    ints = lambda a: torch.tensor(np.asarray(a), dtype=torch.int32, device=dev)
+    bias, sink = rnd(nh, W + 1, dtype=torch.float32), torch.zeros(nh, device=dev)
+    sizes = dict(num_heads=nh, num_kv_heads=nkv, head_dim=d, v_head_dim=d, row=d, page_size=page)
+    C = (nh + 2 * nkv) * d
+    for n_reqs, per in ((64, 1), (1, T)):
+        t, c = n_reqs * per, 3
+        ctx = RUFISUN_CONTEXT if per == 1 else 0
+        blocks = (ctx + per) // page + 1
+        bt = ints(np.arange(n_reqs * blocks)).view(n_reqs, blocks)
+        pages = rnd(n_reqs * blocks, 2 * nkv * page * d)
+        proj, q = [rnd(t, C) for _ in range(c)], torch.empty(t, nh * d, dtype=bf, device=dev)
+        pos, req = ints(np.tile(np.arange(ctx, ctx + per), n_reqs)), ints(np.repeat(np.arange(n_reqs), per))
+        gq, gk = torch.ones(nh * d, device=dev), torch.ones(nkv * d, device=dev)
+        for temp, name, like in (((0.1, 1024), "growing queries + cache write", ""), (None, "Retodra: query and key norms + cache write", "like the one above")):
+            add(f"{name}, {t} {'single tokens' if per == 1 else 'tokens'}", like, lambda i: ops.qk_norm_cache_write(
+                proj[i % c], 0, nh * d, (nh + nkv) * d, None if temp else gq, None if temp else gk, q, pages, pos, req, bt, eps=1e-6, write_kv=True,
+                temperature=temp, **sizes), c, bytes_=t * C * 4)
+    forms = [("attention, window and kept tokens, distance bias, sink, two-term weights", "", dict(window=W, bias_t=bias, sink=sink, precise_weights=True, keep_first=keep), 2),
+             ("Retodra: attention, window, capped and biased scores, two-term weights", "like the one above", dict(window=W, bias_t=bias, cap=30.0, precise_weights=True), 2),
+             ("attention, all tokens, capped scores, sink, two-term weights", "", dict(window=0, cap=30.0, sink=sink, precise_weights=True), 2),
+             ("Lutodra: attention, all tokens, sink, two-term weights", "like the one above", dict(window=0, sink=sink, precise_weights=True), 2),
+             ("attention over latent rows of 128, sink, two-term weights", "", dict(window=0, sink=sink, precise_weights=True), 1),
+             ("Gipinex: attention over latent rows of 128, two-term weights", "like the one above", dict(window=0, precise_weights=True), 1)]
+    for name, like, kw, planes in forms:
+        kvh = nkv if planes == 2 else 1
+        G, row = nh // kvh, d if planes == 2 else 128
+        n_pages = T // page + 2
+        q_start, ctx, bt = ints([0, T]), ints([0]), ints(np.arange(n_pages)).view(1, -1)
+        n_tiles = -(-T * G // ops.TC_ATTENTION_TILE_ROWS)
+        tile_req, tile_row0 = ints(np.zeros(n_tiles)), ints((np.arange(n_tiles) * ops.TC_ATTENTION_TILE_ROWS)[::-1].copy())
+        q, o, kv = rnd(T, nh * row), torch.empty(T, nh * row, dtype=bf, device=dev), rnd(n_pages, planes, kvh, page * row, scale=0.5)
+        w = kw["window"]
+        seen = sum(min(i + 1, w + min(kw.get("keep_first", 0), max(0, i + 1 - w))) if w else i + 1 for i in range(T))
+        add(f"{name}, prompt of {T}", like, lambda i: ops.attention_prefill_tc(
+            q, kv, o, q_start, ctx, bt, tile_req, tile_row0, num_heads=nh, num_kv_heads=kvh, head_dim=row, page_size=page, scale=row ** -0.5, planes=planes, **kw),
+            4, flops=4.0 * nh * row * seen)
+        part = PagedAttention(h, nh, kvh, row, True, False, w, PartSpec("none"), bf, dev)
+        part.keep_first = kw.get("keep_first", 0)
+        for batch in (8, 64):
+            contexts, blocks = [RUFISUN_CONTEXT - 1] * batch, -(-RUFISUN_CONTEXT // page)
+            bt, q_start, ctx = ints(np.arange(batch * blocks)).view(batch, blocks), ints(np.arange(batch + 1)), ints(contexts)
+            q, o = rnd(batch, nh * row), torch.empty(batch, nh * row, dtype=bf, device=dev)
+            kv = rnd(batch * blocks + 1, planes, kvh, page * row, scale=0.5)
+            share = ops.decode_head_groups(nh, kvh)
+            host = HostStep([1] * batch, contexts, page)
+            tiles = ints(part.step_arrays()[part._splits_key()](host))
+            ns = host.shapes[part._splits_key()]
+            scratch = (torch.empty(batch * nh * ns * row, device=dev), torch.empty(batch * nh * ns * 2, device=dev),
+                       torch.zeros(batch * kvh * share, dtype=torch.int32, device=dev))
+            keys = min(RUFISUN_CONTEXT, w + kw.get("keep_first", 0)) if w else RUFISUN_CONTEXT
+            add(f"{name}, decode, batch {batch}, context {RUFISUN_CONTEXT}", like, lambda i: ops.attention_decode_mma(
+                q, kv, o, q_start, ctx, bt, None, batch, ns, *scratch, num_heads=nh, num_kv_heads=kvh * share, head_dim=row, page_size=page,
+                scale=row ** -0.5, split_tiles=tiles, kv_share=share, planes=planes, **kw), 4, bytes_=batch * keys * planes * kvh * row * 2)
+
+
 def unavailable(why: str) -> int:
     print(json.dumps({"impl": "reference", "unavailable": " ".join(str(why).split())[:600]}))
     return 0
@@ -1797,6 +2038,9 @@ def main() -> int:
                     help="instead of the benchmark's workload: prefill and decode throughput of the Kasuvik design beside Retodra "
                          "with dense feed-forwards at equal layer sizes, and the design's kernels alone: 'all' or a comma list of "
                          + ",".join(sorted(KASUVIK_SIZES)))
+    ap.add_argument("--rufisun", default="", metavar="SIZES",
+                    help="instead of the benchmark's workload: prefill and decode throughput of the Rufisun design beside Retodra "
+                         "at equal layer sizes, and the design's kernels alone: 'all' or a comma list of " + ",".join(sorted(RUFISUN_SIZES)))
     ap.add_argument("--retodra", default="", metavar="SIZES",
                     help="instead of the benchmark's workload: prefill and decode throughput of the Retodra design beside Qwen2 "
                          f"at equal layer sizes ({','.join(sorted(RETODRA_SIZES))} or 'all'), and the design's kernels alone "
@@ -1842,6 +2086,8 @@ def main() -> int:
         return run_gipinex(a)
     if a.kasuvik:
         return run_kasuvik(a)
+    if a.rufisun:
+        return run_rufisun(a)
     if a.mix:
         return run_mix(cfg, a)
     if a.kernels:
